@@ -1,4 +1,4 @@
-// Resident decode engine behind the tenzo.h ABI (and its additive extension, tenzo_ext.h).
+// The BitNet model of the resident decode engine behind the tenzo.h ABI (and its additive extension, tenzo_ext.h).
 //
 // Mirrors TenzoEngineImpl of the reference (src/runtime/TenzoEngine.cpp:1215-1838): embedding ->
 // num_layers x forward_layer -> (generate only) logits + sampler, with the sequence length
@@ -14,7 +14,6 @@
 //   tl1_gemv  post_norm + quant + [gate|up] rows, relu(g)^2*u           [:1594-1620]
 //   tl1_gemv  ffn_sub_norm + quant + down rows, x = h1 + .              [:1622-1628]
 #include <cuda_runtime.h>
-#include <nvtx3/nvToolsExt.h>
 
 #include <cmath>
 #include <cstdio>
@@ -46,33 +45,6 @@ void rope_tables_host(int max_seq, int head_dim, float theta, float* cs, float* 
             cs[(size_t)p * half + i] = std::cos(ang);
             sn[(size_t)p * half + i] = std::sin(ang);
         }
-}
-
-
-thread_local std::string g_last_error;
-void set_error(const std::string& m) { g_last_error = m; }
-
-#define TZ_KERNEL(expr)                                                                         \
-    do {                                                                                        \
-        int _r = (expr);                                                                        \
-        if (_r > 0) throw CudaError((cudaError_t)_r, #expr);                                    \
-        if (_r < 0) throw std::runtime_error(std::string(#expr) + " rejected its arguments");   \
-    } while (0)
-
-__global__ void advance_kernel(int* pos, int* tokens, const int* next, int batch, int feed_back, int vocab) {
-    const int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < batch) {
-        pos[i] += 1;
-        if (feed_back) {
-            const int t = next[i];
-            tokens[i] = (t >= 0 && t < vocab) ? t : 0;
-        }
-    }
-}
-
-__global__ void record_tokens_kernel(const int* next, int* history, int step, int batch) {
-    const int i = blockIdx.x * blockDim.x + threadIdx.x;
-    if (i < batch) history[(size_t)step * batch + i] = next[i];
 }
 
 // Chunked prefill: rotate and quantise the K rows, quantise the V rows of M consecutive tokens of one sequence and
@@ -142,23 +114,10 @@ __global__ void kv_fill_kernel(int8_t* k, int8_t* v, float* sk, float* sv, size_
     }
 }
 
-static int env_flag(const char* name, int dflt) {
-    const char* s = std::getenv(name);
-    return s ? std::atoi(s) : dflt;
-}
-
-// Named ranges around the engine's public operations for timeline tools (the reference marks nothing; its only
-// instrumentation is the wall-clock tok/s of its CLI). Off unless TENZO_NVTX=1: a range push is a call into the tools
-// interface on every token.
-struct NvtxRange {
-    bool on;
-    explicit NvtxRange(const char* name) : on(env_flag("TENZO_NVTX", 0) != 0) { if (on) nvtxRangePushA(name); }
-    ~NvtxRange() { if (on) nvtxRangePop(); }
-};
-
 // A constructor that throws never runs the destructor, so what it had acquired by then (stream, events, device and
 // pinned memory) is released here before the exception leaves.
-Engine::Engine(const tenzo_config_t& c, const tenzo_ext_options_t& o) : cfg(c) {
+Engine::Engine(const tenzo_config_t& c, const tenzo_ext_options_t& o) {
+    cfg = c;
     try {
         init(c, o);
     } catch (...) {
@@ -168,10 +127,7 @@ Engine::Engine(const tenzo_config_t& c, const tenzo_ext_options_t& o) : cfg(c) {
 }
 
 void Engine::init(const tenzo_config_t& c, const tenzo_ext_options_t& o) {
-    batch = o.batch > 0 ? o.batch : 1;
     rope_theta = o.rope_theta > 0.0f ? o.rope_theta : 10000.0f;   // TenzoEngine.cpp:456
-    use_graph = o.use_graph >= 0 ? o.use_graph : env_flag("TENZO_CUDA_GRAPH", 1);
-    use_pdl = o.use_pdl >= 0 ? o.use_pdl : env_flag("TENZO_CUDA_PDL", 1);
     persistent = o.persistent >= 0 ? o.persistent : env_flag("TENZO_PERSISTENT", 0);
     attention_mode = o.attention_mode >= 0 ? o.attention_mode : env_flag("TENZO_ATTENTION_MODE", 0);
     if (attention_mode != 0 && attention_mode != 1) throw std::invalid_argument("attention_mode must be 0 or 1");
@@ -193,29 +149,15 @@ void Engine::init(const tenzo_config_t& c, const tenzo_ext_options_t& o) {
     if (g != 1 && g != 2 && g != 4 && g != 8) throw std::invalid_argument("query group size must be 1, 2, 4 or 8");
     if (h > 16384 || ffn > 16384) throw std::invalid_argument("hidden_size and ffn_dim are limited to 16384");
 
-    TZ_CUDA(cudaGetDevice(&device));
-    TZ_CUDA(cudaStreamCreateWithFlags(&stream, cudaStreamNonBlocking));
-    TZ_CUDA(cudaEventCreate(&ev0));
-    TZ_CUDA(cudaEventCreate(&ev1));
-
+    init_core(o.batch, o.use_graph, o.use_pdl);
+    init_core_buffers();
     layers.resize(L);
     const size_t B = batch;
-    auto dalloc = [&](size_t bytes) -> void* {
-        void* p = nullptr;
-        TZ_CUDA(cudaMalloc(&p, bytes ? bytes : 16));
-        TZ_CUDA(cudaMemsetAsync(p, 0, bytes ? bytes : 16, stream));
-        owned.push_back(p);
-        return p;
-    };
-    d_tokens = (int*)dalloc(B * 4);
-    d_pos = (int*)dalloc(B * 4);
-    d_next = (int*)dalloc(B * 4);
     b_x = (float*)dalloc(B * h * 4);
     b_qkv = (float*)dalloc(B * (qd + 2 * kvd) * 4);
     b_attn = (float*)dalloc(B * qd * 4);
     b_h1 = (float*)dalloc(B * h * 4);
     b_act = (float*)dalloc(B * ffn * 4);
-    b_logits = (float*)dalloc(B * V * 4);
 
     kv_rows_per_seq = (size_t)L * cfg.num_kv_heads * cfg.max_seq_len;
     if (paged) {
@@ -257,35 +199,15 @@ void Engine::init(const tenzo_config_t& c, const tenzo_ext_options_t& o) {
         persistent = 0;                                   // the one-kernel form has only the exact-order attention
     }
 
-    TZ_CUDA(cudaMallocHost(&h_pin, (3 * B + 16) * sizeof(int)));
-    h_tokens = h_pin;
-    h_pos = h_pin + B;
-    h_next = h_pin + 2 * B;
-    seq_len.assign(batch, 0);
     TZ_CUDA(cudaStreamSynchronize(stream));
 }
 
-// Everything the engine owns, safe to call on a partly constructed object (the constructor calls it when it throws).
 void Engine::release_all() {
     if (stream) cudaStreamSynchronize(stream);
-    for (auto& kv : graphs) cudaGraphExecDestroy(kv.second);
-    graphs.clear();
-    for (void* p : owned) cudaFree(p);
-    owned.clear();
-    if (h_pin) cudaFreeHost(h_pin);
-    if (h_table) cudaFreeHost(h_table);
-    if (h_cand) cudaFreeHost(h_cand);
     if (pc_host) cudaFreeHost(pc_host);
-    h_pin = nullptr; h_table = nullptr; h_cand = nullptr; pc_host = nullptr;
+    pc_host = nullptr;
     free_prefill_rows();
-    if (d_sample_past) cudaFree(d_sample_past);
-    if (d_history) cudaFree(d_history);
-    d_sample_past = nullptr; d_history = nullptr;
-    if (ev0) cudaEventDestroy(ev0);
-    if (ev1) cudaEventDestroy(ev1);
-    if (stream) cudaStreamDestroy(stream);
-    ev0 = ev1 = nullptr;
-    stream = nullptr;
+    release_core();
 }
 
 Engine::~Engine() { release_all(); }
@@ -299,62 +221,12 @@ void Engine::free_prefill_rows() {
     pf_cap = 0;
 }
 
-void Engine::reserve_blocks(int s, int len) {
-    if (!paged) return;
-    while (n_blocks[s] * kBlock < len) {
-        if (free_blocks.empty()) throw std::out_of_range("the KV block pool is exhausted");   // the reference would reuse block 0 (:302)
-        h_table[(size_t)s * table_stride + n_blocks[s]] = free_blocks.back();   // TenzoEngine.h:136-141
-        free_blocks.pop_back();
-        n_blocks[s] += 1;
-        table_dirty = true;
-    }
-}
-
-void Engine::release_blocks(int s, int len) {
-    if (!paged) return;
-    const int keep = (len + kBlock - 1) / kBlock;
-    if (n_blocks[s] <= keep) return;
-    TZ_CUDA(cudaStreamSynchronize(stream));               // no step in flight may still read the entries given back
-    while (n_blocks[s] > keep) {
-        n_blocks[s] -= 1;
-        free_blocks.push_back(h_table[(size_t)s * table_stride + n_blocks[s]]);   // TenzoEngine.h:143-147
-    }
-}
-
-// Entries are only ever added between two synchronising calls (reset_kv, release_blocks), so a copy still queued
-// behind earlier steps may carry newer entries without harm: those steps do not read them.
-void Engine::prepare_kv(int extra) {
-    if (!paged) return;
-    for (int s = 0; s < batch; ++s) reserve_blocks(s, seq_len[s] + extra);
-    if (table_dirty) {
-        TZ_CUDA(cudaMemcpyAsync(d_table, h_table, (size_t)batch * table_stride * sizeof(int), cudaMemcpyHostToDevice, stream));
-        table_dirty = false;
-    }
-}
-
-void Engine::reset_kv() {                                  // TenzoEngine.cpp:242-246
-    for (auto& n : seq_len) n = 0;
-    if (!paged) return;
-    TZ_CUDA(cudaStreamSynchronize(stream));
-    free_blocks.clear();
-    for (int i = total_blocks - 1; i >= 0; --i) free_blocks.push_back(i);
-    n_blocks.assign(batch, 0);
-}
-
 size_t Engine::kv_row(int s, int layer, int kvh, int t) const {
     if (paged) {
         const size_t blk = (size_t)h_table[(size_t)s * table_stride + t / kBlock];
         return ((blk * L + layer) * cfg.num_kv_heads + kvh) * kBlock + (size_t)(t % kBlock);
     }
     return (size_t)s * kv_rows_per_seq + ((size_t)layer * cfg.num_kv_heads + kvh) * cfg.max_seq_len + t;
-}
-
-void* Engine::upload(const void* host, size_t bytes) {
-    void* p = nullptr;
-    TZ_CUDA(cudaMalloc(&p, bytes));
-    owned.push_back(p);
-    TZ_CUDA(cudaMemcpy(p, host, bytes, cudaMemcpyHostToDevice));
-    return p;
 }
 
 void Engine::set_layer(int l, const tenzo_layer_weights_t& w) {
@@ -413,11 +285,10 @@ void Engine::set_lm_head(const int8_t* w, const float* scales) {
 
 void Engine::invalidate_graphs() {
     pc_built = false;                      // the persistent kernel's layer table is rebuilt from the new pointers
-    if (graphs.empty()) return;
-    cudaStreamSynchronize(stream);
-    for (auto& kv : graphs) cudaGraphExecDestroy(kv.second);
-    graphs.clear();
+    EngineCore::invalidate_graphs();
 }
+
+void Engine::enqueue_layer(int l, int max_len) { enqueue_layer(l, max_len, false); }
 
 void Engine::enqueue_layer(int l, int max_len, bool gemv_only) {
     const LayerDev& d = layers[l];
@@ -499,25 +370,16 @@ void Engine::enqueue_step(bool with_logits, bool feed_back, int max_len) {
                                         d_next, lm_scratch, use_pdl, stream));
         launches += batch >= 16 && h % 128 == 0 ? 3 : 2;   // (quantiser +) LM head + argmax finish
     }
-    advance_kernel<<<(batch + 127) / 128, 128, 0, stream>>>(d_pos, d_tokens, d_next, batch, feed_back ? 1 : 0, V);
-    TZ_CUDA(cudaGetLastError());
-    launches += 1;
+    enqueue_advance(feed_back);
 }
-
-static int bucket_for(int len, int max_seq);
 
 // Chunked prefill of one sequence: M prompt tokens go through every layer together - the TL1 layers as GEMMs over the
 // M rows, the K/V rows appended first, then causal attention as M independent queries over the same cache (token i sees
 // keys 0..pos0+i). Row i of every product is the same arithmetic as feeding token i alone, so the cache and the state
 // after the chunk are bit-identical to M calls of prefill().
-void Engine::prefill_chunk(const int* tokens, int M) {
-    NvtxRange range("tenzo.prefill_chunk");
+void Engine::chunk_rows(int, const int* tokens, int M) {
     if (batch != 1) throw std::invalid_argument("chunked prefill is for single-sequence engines");
-    if (M <= 0) return;
     if (!lm_w) throw std::runtime_error("LM head / embedding was never set");
-    if (seq_len[0] + M > cfg.max_seq_len) throw std::out_of_range("KV cache is full (max_seq_len reached)");
-    for (int i = 0; i < M; ++i)
-        if (tokens[i] < 0 || tokens[i] >= V) throw std::out_of_range("token id outside [0, vocab_size)");
     if (M > pf_cap) {
         // Free first, forget the old pointers, and claim the new capacity only once every allocation has succeeded: a
         // failed cudaMalloc must leave the engine with no rows rather than with freed ones.
@@ -544,7 +406,6 @@ void Engine::prefill_chunk(const int* tokens, int M) {
     for (int i = 0; i < M; ++i) hp[i] = pos0 + i;
     TZ_CUDA(cudaMemcpyAsync(pf_tokens, tokens, (size_t)M * 4, cudaMemcpyHostToDevice, stream));
     TZ_CUDA(cudaMemcpyAsync(pf_pos, hp.data(), (size_t)M * 4, cudaMemcpyHostToDevice, stream));
-    TZ_CUDA(cudaEventRecord(ev0, stream));
     TZ_KERNEL(tenzo_cuda_embedding_i8(lm_w, lm_scales, h, pf_tokens, M, pf_x, h, V, stream));
     launches += 1;
     const int gemv_kernels = M > 1 ? 2 : 1;
@@ -598,71 +459,33 @@ void Engine::prefill_chunk(const int* tokens, int M) {
     }
     // the engine's single-token state after the chunk: residual stream of the last token, position
     TZ_CUDA(cudaMemcpyAsync(b_x, pf_x + (size_t)(M - 1) * h, (size_t)h * 4, cudaMemcpyDeviceToDevice, stream));
-    TZ_CUDA(cudaEventRecord(ev1, stream));
-    TZ_CUDA(cudaStreamSynchronize(stream));
+    TZ_CUDA(cudaStreamSynchronize(stream));            // the staged positions and tokens are host memory of this call
     seq_len[0] += M;
-    check_device_status(false);
 }
 
-static int bucket_for(int len, int max_seq) {
-    int b = 256;
-    while (b < len) b <<= 1;
-    return b < max_seq ? b : max_seq;
+void Engine::rows_logits(const int* want, int n_want, float* host) {
+    for (int i = 0; i < n_want; ++i) {
+        TZ_KERNEL(tenzo_cuda_lm_head_i8(pf_x + (size_t)want[i] * h, final_norm, 1, 1e-5f, lm_w, lm_scales, V, h, 1, h, b_logits, nullptr,
+                                        d_next, lm_scratch, 0, stream));
+        launches += 2;
+        TZ_CUDA(cudaMemcpyAsync(host + (size_t)i * V, b_logits, (size_t)V * 4, cudaMemcpyDeviceToHost, stream));
+    }
+    TZ_CUDA(cudaStreamSynchronize(stream));
 }
 
-// One step for all sequences. The graph key is (with_logits, feed_back, attention bucket).
-void Engine::run_step(bool with_logits, bool feed_back) {
-    int longest = 0;
-    for (int s = 0; s < batch; ++s) {
-        if (seq_len[s] + 1 > cfg.max_seq_len) throw std::out_of_range("KV cache is full (max_seq_len reached)");
-        longest = seq_len[s] + 1 > longest ? seq_len[s] + 1 : longest;
+const float* Engine::buffer(int which, int seq, size_t* n) {
+    const size_t qkv = (size_t)qd + 2 * kvd;
+    switch (which) {
+        case TENZO_BUF_X: *n = h; return b_x + (size_t)seq * h;
+        case TENZO_BUF_Q: *n = qd; return b_qkv + seq * qkv;
+        case TENZO_BUF_K: *n = kvd; return b_qkv + seq * qkv + qd;
+        case TENZO_BUF_V: *n = kvd; return b_qkv + seq * qkv + qd + kvd;
+        case TENZO_BUF_ATTN_OUT: *n = qd; return b_attn + (size_t)seq * qd;
+        case TENZO_BUF_H1: *n = h; return b_h1 + (size_t)seq * h;
+        case TENZO_BUF_ACT: *n = ffn; return b_act + (size_t)seq * ffn;
+        case TENZO_BUF_LOGITS: *n = V; return b_logits + (size_t)seq * V;
+        default: throw std::invalid_argument("unknown buffer id");
     }
-    const int max_len = bucket_for(longest, cfg.max_seq_len);
-    prepare_kv(1);
-    if (pc_usable() && longest <= pc_score_cap(max_len)) {
-        pc_step(with_logits, feed_back, max_len);
-    } else if (!use_graph) {
-        enqueue_step(with_logits, feed_back, max_len);
-    } else {
-        const int key = (with_logits ? 1 : 0) | (feed_back ? 2 : 0) | (max_len << 2);
-        auto it = graphs.find(key);
-        if (it == graphs.end()) {
-            const unsigned long long before = launches;
-            cudaGraph_t graph = nullptr;
-            TZ_CUDA(cudaStreamBeginCapture(stream, cudaStreamCaptureModeThreadLocal));
-            try {
-                enqueue_step(with_logits, feed_back, max_len);
-            } catch (...) {
-                cudaStreamEndCapture(stream, &graph);
-                if (graph) cudaGraphDestroy(graph);
-                launches = before;
-                throw;
-            }
-            TZ_CUDA(cudaStreamEndCapture(stream, &graph));
-            cudaGraphExec_t exec = nullptr;
-            cudaError_t e = cudaGraphInstantiate(&exec, graph, 0);
-            cudaGraphDestroy(graph);
-            if (e != cudaSuccess) throw CudaError(e, "cudaGraphInstantiate");
-            graph_kernels[key] = launches - before;
-            launches = before;
-            it = graphs.emplace(key, exec).first;
-        }
-        TZ_CUDA(cudaGraphLaunch(it->second, stream));
-        launches += graph_kernels[key];
-    }
-    for (int s = 0; s < batch; ++s) seq_len[s] += 1;   // :1831-1835, once per token
-}
-
-void Engine::push_state(const int* tokens) {
-    for (int s = 0; s < batch; ++s) {
-        if (tokens) {
-            if (tokens[s] < 0 || tokens[s] >= V) throw std::out_of_range("token id outside [0, vocab_size)");
-            h_tokens[s] = tokens[s];
-        }
-        h_pos[s] = seq_len[s];
-    }
-    if (tokens) TZ_CUDA(cudaMemcpyAsync(d_tokens, h_tokens, (size_t)batch * 4, cudaMemcpyHostToDevice, stream));
-    TZ_CUDA(cudaMemcpyAsync(d_pos, h_pos, (size_t)batch * 4, cudaMemcpyHostToDevice, stream));
 }
 
 // The TL1 kernel's waits on asynchronous copies are bounded; a give-up is reported here instead of
@@ -677,18 +500,7 @@ void Engine::check_device_status(bool force) {
     if (tenzo_cuda_tl1_gemv_take_timeouts() > 0) throw std::runtime_error("a TL1 kernel gave up waiting for its weight copy; results are invalid");
 }
 
-void Engine::prefill(const int* tokens) {
-    NvtxRange range("tenzo.prefill_token");
-    push_state(tokens);
-    TZ_CUDA(cudaEventRecord(ev0, stream));
-    run_step(false, false);
-    TZ_CUDA(cudaEventRecord(ev1, stream));
-    TZ_CUDA(cudaStreamSynchronize(stream));
-    pc_check();
-}
-
 void Engine::generate(const int* cur, int* out) {
-    NvtxRange range("tenzo.generate_step");
     if (pc_usable() && seq_len[0] + 1 <= pc_score_cap(bucket_for(seq_len[0] + 1, cfg.max_seq_len))) {
         // persistent kernel: token and position travel as kernel arguments, the result comes back through a mapped
         // host word - no copies in either direction
@@ -709,37 +521,7 @@ void Engine::generate(const int* cur, int* out) {
         out[0] = pc_host[1];
         return;
     }
-    push_state(cur);
-    TZ_CUDA(cudaEventRecord(ev0, stream));
-    run_step(true, false);
-    TZ_CUDA(cudaEventRecord(ev1, stream));
-    TZ_CUDA(cudaMemcpyAsync(h_next, d_next, (size_t)batch * 4, cudaMemcpyDeviceToHost, stream));
-    TZ_CUDA(cudaStreamSynchronize(stream));
-    check_device_status(false);
-    for (int s = 0; s < batch; ++s) out[s] = h_next[s];
-}
-
-void Engine::decode_greedy(const int* first, int n_steps, int* out) {
-    NvtxRange range("tenzo.decode_greedy");
-    if (n_steps <= 0) return;
-    if ((size_t)n_steps * batch > history_cap) {
-        if (d_history) cudaFree(d_history);
-        d_history = nullptr;
-        TZ_CUDA(cudaMalloc((void**)&d_history, (size_t)n_steps * batch * 4));
-        history_cap = (size_t)n_steps * batch;
-    }
-    push_state(first);
-    TZ_CUDA(cudaEventRecord(ev0, stream));
-    for (int i = 0; i < n_steps; ++i) {
-        run_step(true, true);
-        record_tokens_kernel<<<(batch + 127) / 128, 128, 0, stream>>>(d_next, d_history, i, batch);
-        launches += 1;
-    }
-    TZ_CUDA(cudaEventRecord(ev1, stream));
-    TZ_CUDA(cudaMemcpyAsync(out, d_history, (size_t)n_steps * batch * 4, cudaMemcpyDeviceToHost, stream));
-    TZ_CUDA(cudaStreamSynchronize(stream));
-    pc_check();
-    check_device_status(true);
+    EngineCore::generate(cur, out);
 }
 
 void Engine::kv_fill(int len, unsigned long long seed) {
@@ -843,6 +625,12 @@ bool Engine::pc_usable() {
     return true;
 }
 
+bool Engine::direct_step(bool with_logits, bool feed_back, int max_len, int longest) {
+    if (!pc_usable() || longest > pc_score_cap(max_len)) return false;
+    pc_step(with_logits, feed_back, max_len);
+    return true;
+}
+
 void Engine::pc_step(bool with_logits, bool feed_back, int max_len) {
     PcParams p;
     std::memset(&p, 0, sizeof p);
@@ -888,95 +676,6 @@ void Engine::pc_check() {
     static const char* what[] = {"", "a grid-wide barrier", "a weight copy", "a value-cache copy", "a position inside its bounds"};
     throw std::runtime_error(std::string("the persistent decode kernel gave up waiting for ") + (code >= 1 && code <= 4 ? what[code] : "something") +
                              "; results of that step are invalid");
-}
-
-float Engine::last_ms() {
-    float ms = 0.0f;
-    if (cudaEventElapsedTime(&ms, ev0, ev1) != cudaSuccess) return -1.0f;
-    return ms;
-}
-
-// The reference sampler (TenzoEngine.cpp:1722-1807) on host logits, for the stochastic path and
-// for greedy decoding with a repetition penalty. Candidate order follows std::pair<float,int>.
-// The reference's streaming top-k, softmax, top-p and draw (TenzoEngine.cpp:1745-1806) over pairs in ascending index order.
-int sample_pairs(const float* vals, const int* idxs, int n_in, const tenzo_sampling_params_t& p, float r_in) {
-    if (n_in <= 0) return 0;
-    if (p.temperature <= 0.0f) {                          // first maximum (:1746-1755)
-        int best = 0;
-        for (int i = 1; i < n_in; ++i)
-            if (vals[i] > vals[best]) best = i;
-        return idxs ? idxs[best] : best;
-    }
-    const int top_k = p.top_k < 1 ? 1 : (p.top_k > 64 ? 64 : p.top_k);
-    float cl[64];
-    int ci[64], n = 0;
-    for (int j = 0; j < n_in; ++j) {                      // sorted insert = the min-heap of (value, index) pairs, :1760-1768
-        const float l = vals[j];
-        const int i = idxs ? idxs[j] : j;
-        if (n == top_k) {
-            if (!(l > cl[n - 1])) continue;
-            --n;
-        }
-        int q = n;
-        while (q > 0 && (cl[q - 1] < l || (!(l < cl[q - 1]) && ci[q - 1] < i))) { cl[q] = cl[q - 1]; ci[q] = ci[q - 1]; --q; }
-        cl[q] = l; ci[q] = i; ++n;
-    }
-    float probs[64], sum = 0.0f;
-    for (int i = 0; i < n; ++i) { probs[i] = std::exp((cl[i] - cl[0]) / p.temperature); sum += probs[i]; }
-    for (int i = 0; i < n; ++i) probs[i] /= sum;
-    float cum = 0.0f;
-    int cut = n;
-    for (int i = 0; i < n; ++i) { cum += probs[i]; if (cum >= p.top_p) { cut = i + 1; break; } }
-    float sub = 0.0f;
-    for (int i = 0; i < cut; ++i) sub += probs[i];
-    for (int i = 0; i < cut; ++i) probs[i] /= sub;
-    const float r = r_in >= 0.0f ? r_in : static_cast<float>(std::rand()) / static_cast<float>(RAND_MAX);   // :1800, process-global rand()
-    float acc = 0.0f;
-    for (int i = 0; i < cut; ++i) { acc += probs[i]; if (r <= acc) return ci[i]; }
-    return ci[0];
-}
-
-// Penalty, k-th-largest selection and candidate compaction on the device (sampler.cu), the rest on the host.
-int Engine::sample(const tenzo_sampling_params_t& p, const int* past, int n_past) {
-    if (batch != 1) throw std::invalid_argument("sampling with parameters is per sequence");
-    if (p.repetition_penalty != 1.0f && past && n_past > 0) {
-        std::map<int, int> mult;                          // once per occurrence (:1736-1742)
-        for (int i = 0; i < n_past; ++i) ++mult[past[i]];
-        std::vector<int> toks, cnts;
-        for (auto& kv : mult) { toks.push_back(kv.first); cnts.push_back(kv.second); }
-        const size_t n = toks.size();
-        if (n > sample_past_cap) {
-            if (d_sample_past) cudaFree(d_sample_past);
-            sample_past_cap = n * 2;
-            TZ_CUDA(cudaMalloc((void**)&d_sample_past, sample_past_cap * 2 * sizeof(int)));
-        }
-        TZ_CUDA(cudaMemcpyAsync(d_sample_past, toks.data(), n * 4, cudaMemcpyHostToDevice, stream));
-        TZ_CUDA(cudaMemcpyAsync(d_sample_past + sample_past_cap, cnts.data(), n * 4, cudaMemcpyHostToDevice, stream));
-        TZ_CUDA(launch_penalty(b_logits, V, d_sample_past, d_sample_past + sample_past_cap, (int)n, p.repetition_penalty, stream));
-        launches += 1;
-    }
-    const int k = p.temperature <= 0.0f ? 1 : (p.top_k < 1 ? 1 : (p.top_k > 64 ? 64 : p.top_k));
-    if (!d_cand) {
-        TZ_CUDA(cudaMalloc((void**)&d_cand, 16 + (size_t)kMaxCandidates * 8));
-        owned.push_back(d_cand);
-        TZ_CUDA(cudaMallocHost((void**)&h_cand, 16 + (size_t)kMaxCandidates * 8));
-    }
-    int* d_count = reinterpret_cast<int*>(d_cand);
-    float* d_val = reinterpret_cast<float*>(static_cast<unsigned char*>(d_cand) + 16);
-    int* d_idx = reinterpret_cast<int*>(d_val + kMaxCandidates);
-    TZ_CUDA(launch_select_candidates(b_logits, V, k, d_count, d_val, d_idx, stream));
-    launches += 1;
-    TZ_CUDA(cudaMemcpyAsync(h_cand, d_cand, 16 + (size_t)kMaxCandidates * 8, cudaMemcpyDeviceToHost, stream));
-    TZ_CUDA(cudaStreamSynchronize(stream));
-    const int count = *reinterpret_cast<const int*>(h_cand);
-    const float* hv = reinterpret_cast<const float*>(static_cast<unsigned char*>(h_cand) + 16);
-    const int* hi = reinterpret_cast<const int*>(hv + kMaxCandidates);
-    if (count > kMaxCandidates) {                         // a huge tie at the threshold: take the whole vector
-        std::vector<float> lg((size_t)V);
-        TZ_CUDA(cudaMemcpy(lg.data(), b_logits, lg.size() * 4, cudaMemcpyDeviceToHost));
-        return sample_pairs(lg.data(), nullptr, V, p, -1.0f);
-    }
-    return sample_pairs(hv, hi, count, p, -1.0f);
 }
 
 }  // namespace tz

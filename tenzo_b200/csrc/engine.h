@@ -1,4 +1,4 @@
-// Engine state shared between engine.cu (behaviour) and capi.cu (the extern "C" boundary).
+// The BitNet engine: state shared between engine.cu (behaviour) and capi_bitnet.cu (its part of the extern "C" boundary).
 #pragma once
 #include <cuda_runtime.h>
 #include <stdint.h>
@@ -10,24 +10,11 @@
 #include "../../include/tenzo.h"
 #include "../../include/tenzo_ext.h"
 #include "decode_persistent.h"
+#include "engine_core.h"
 
 namespace tz {
 
 void rope_tables_host(int max_seq, int head_dim, float theta, float* cs, float* sn);
-
-
-extern thread_local std::string g_last_error;
-void set_error(const std::string& m);
-
-struct CudaError : std::runtime_error {
-    cudaError_t code;
-    CudaError(cudaError_t c, const char* what) : std::runtime_error(std::string(what) + ": " + cudaGetErrorString(c)), code(c) {}
-};
-#define TZ_CUDA(expr)                                            \
-    do {                                                         \
-        cudaError_t _e = (expr);                                 \
-        if (_e != cudaSuccess) throw tz::CudaError(_e, #expr);   \
-    } while (0)
 
 
 struct LayerDev {
@@ -40,68 +27,43 @@ struct LayerDev {
     bool has_mlp = false, set = false;
 };
 
-class Engine {
+class Engine final : public EngineCore {
 public:
     Engine(const tenzo_config_t& cfg, const tenzo_ext_options_t& opt);
-    ~Engine();
+    ~Engine() override;
     void init(const tenzo_config_t& cfg, const tenzo_ext_options_t& opt);
-    Engine(const Engine&) = delete;
-    Engine& operator=(const Engine&) = delete;
 
     void set_layer(int l, const tenzo_layer_weights_t& w);
     void set_final_norm(const float* w);
     void set_lm_head(const int8_t* w, const float* scales);
 
-    void prefill(const int* tokens);                       // one token per sequence, no logits
-    void prefill_chunk(const int* tokens, int n);          // n consecutive tokens of the one sequence, together
-    void generate(const int* cur, int* out);               // device argmax
-    void decode_greedy(const int* first, int n_steps, int* out);
-    int sample(const tenzo_sampling_params_t& p, const int* past, int n_past);   // on the logits of the last step
+    void enqueue_step(bool with_logits, bool feed_back, int max_len) override;
+    void enqueue_layer(int l, int max_len) override;
+    void chunk_rows(int seq, const int* tokens, int n) override;
+    void rows_logits(const int* want, int n_want, float* host) override;
+    const float* buffer(int which, int seq, size_t* count) override;
+    void check_device_status(bool force) override;
+    bool direct_step(bool with_logits, bool feed_back, int max_len, int longest) override;
+    void after_sync() override { pc_check(); }
+    void invalidate_graphs() override;
+    void kv_fill(int len, unsigned long long seed) override;
+    void generate(const int* cur, int* out) override;      // device argmax
 
-    void push_state(const int* tokens);
-    void run_step(bool with_logits, bool feed_back);
-    void enqueue_step(bool with_logits, bool feed_back, int max_len);
-    void enqueue_layer(int l, int max_len, bool gemv_only = false);
+    void enqueue_layer(int l, int max_len, bool gemv_only);
     float bench_gemv_stack(int iters, unsigned long long* n_launches);
-    void invalidate_graphs();
     void free_prefill_rows();
     void release_all();
-    void* upload(const void* host, size_t bytes);
-    float last_ms();
-    void check_device_status(bool force);
     unsigned status_poll = 0;
-    void kv_fill(int len, unsigned long long seed);
-
-    // kv_mode "paged_int8" (PagedKVCache + PagedBlockManager of the reference, TenzoEngine.h:117-193): the caches are pools
-    // of 16-token blocks [block][layer][kv_head][16][128]; every sequence has a row of the block table. Blocks are taken
-    // from the free list on the host before the step that first writes into them (the reference does it inside layer 0,
-    // TenzoEngine.cpp:294-300) and the table row is copied to the device ahead of the launch.
-    static constexpr int kBlock = 16;
-    bool paged = false;
-    int total_blocks = 0, table_stride = 0;
-    int *d_table = nullptr, *h_table = nullptr;          // [batch][table_stride]; h_table is the pinned master copy
-    std::vector<int> free_blocks, n_blocks;              // free list (taken from the back: 0, 1, 2, ... as the reference's)
-    bool table_dirty = false;
-    void reserve_blocks(int seq, int len);               // the table of `seq` covers tokens [0, len)
-    void release_blocks(int seq, int len);               // blocks past token len go back to the free list
-    void prepare_kv(int extra);                          // before a step that appends `extra` tokens to every sequence
-    void reset_kv();
     size_t kv_row(int seq, int layer, int kvh, int t) const;   // row of a cached token in cache_k/v (x128) and scale_k/v
 
-    tenzo_config_t cfg;
-    int batch = 1, device = 0, use_graph = 1, use_pdl = 1;
     float rope_theta = 10000.0f;
-    int h = 0, qd = 0, kvd = 0, ffn = 0, L = 0, V = 0;
-    cudaStream_t stream = nullptr;
-    cudaEvent_t ev0 = nullptr, ev1 = nullptr;
+    int qd = 0, kvd = 0, ffn = 0;
     std::vector<LayerDev> layers;
     float* final_norm = nullptr;
     int8_t* lm_w = nullptr;
     float* lm_scales = nullptr;
 
-    int *d_tokens = nullptr, *d_pos = nullptr, *d_next = nullptr, *d_history = nullptr;
-    size_t history_cap = 0;
-    float *b_x = nullptr, *b_qkv = nullptr, *b_attn = nullptr, *b_h1 = nullptr, *b_act = nullptr, *b_logits = nullptr;
+    float *b_qkv = nullptr, *b_attn = nullptr, *b_h1 = nullptr, *b_act = nullptr;
     int8_t *cache_k = nullptr, *cache_v = nullptr;
     float *scale_k = nullptr, *scale_v = nullptr;
     size_t kv_rows_per_seq = 0;
@@ -113,15 +75,6 @@ public:
     float *pf_x = nullptr, *pf_qkv = nullptr, *pf_attn = nullptr, *pf_h1 = nullptr, *pf_act = nullptr;   // chunked prefill rows
     int *pf_tokens = nullptr, *pf_pos = nullptr, pf_cap = 0;
     void* pf_ws = nullptr;
-    void *d_cand = nullptr, *h_cand = nullptr;           // sampler: candidate count + (value, index) pairs
-    int* d_sample_past = nullptr;
-    size_t sample_past_cap = 0;
-    int *h_pin = nullptr, *h_tokens = nullptr, *h_pos = nullptr, *h_next = nullptr;
-    std::vector<int> seq_len;
-    std::vector<void*> owned;
-    std::map<int, cudaGraphExec_t> graphs;
-    std::map<int, unsigned long long> graph_kernels;
-    unsigned long long launches = 0;
 
     // Single-sequence engines: the whole token as one persistent cooperative kernel (decode_persistent.cu) instead of the
     // kernel chain, whenever the shapes fit it (pc_usable). Its scratch is owned here: zeroed accumulators, the barrier
@@ -147,7 +100,3 @@ public:
 };
 
 }  // namespace tz
-
-struct tenzo_engine_opaque {
-    tz::Engine* impl;
-};
