@@ -35,6 +35,25 @@ TENZO_API tenzo_ext_options_t tenzo_ext_default_options(void);
 TENZO_API tenzo_engine_t tenzo_ext_create_engine(const tenzo_config_t* config, const tenzo_ext_options_t* opt);
 TENZO_API int tenzo_ext_batch(tenzo_engine_t engine);
 
+/* Models by folder: config.json names the architecture, the rest of the folder is what that family loads - "Sozopel"
+ * (hybrid decoder): model.safetensors; "BitNet": weights.bin + model.mlir, with the fields of tenzo_config_t in
+ * config.json. `compute` is the arithmetic of activations and matrix products: TENZO_COMPUTE_BF16 (bf16 operands, 32-bit
+ * accumulation) or TENZO_COMPUTE_F32 (32-bit throughout); BitNet has its own integer arithmetic and takes only the
+ * default. opt->batch, use_graph and use_pdl apply to every family. NULL on failure, see tenzo_ext_last_error(). */
+enum { TENZO_COMPUTE_BF16 = 0, TENZO_COMPUTE_F32 = 1 };
+TENZO_API tenzo_engine_t tenzo_ext_open_model(const char* model_dir, const tenzo_ext_options_t* opt, int compute);
+/* Architectures this library was built with: name `index`, NULL past the last one. */
+TENZO_API const char* tenzo_ext_architecture(int index);
+/* Sizes of an engine (fields that a family has no single value for are 0). */
+TENZO_API tenzo_status_t tenzo_ext_get_config(tenzo_engine_t engine, tenzo_config_t* out);
+/* The next n tokens of sequence `seq`, from the state that earlier calls left; logits[n_want][vocab] (host) receives the
+ * logits at the places want[] (ascending, 0..n-1) among them. One token of a single-sequence engine takes the decode
+ * step of tenzo_generate_step, several go through the layers together as in tenzo_ext_prefill_chunk. */
+TENZO_API tenzo_status_t tenzo_ext_forward(tenzo_engine_t engine, int seq, const int* tokens, int n, const int* want, int n_want,
+                                           float* logits);
+/* The slot of one sequence is given back: its next token is at position 0. */
+TENZO_API tenzo_status_t tenzo_ext_reset_seq(tenzo_engine_t engine, int seq);
+
 /* One token per sequence through all layers, no logits (batched tenzo_prefill_token). */
 TENZO_API tenzo_status_t tenzo_ext_prefill_tokens(tenzo_engine_t engine, const int* tokens);
 /* One decode step per sequence; greedy only (temperature <= 0, repetition_penalty == 1) when

@@ -8,23 +8,27 @@ no CPU path — loading fails loudly if the library was not built.
 from __future__ import annotations
 
 import ctypes as C
+import json
 import os
 from pathlib import Path
 
 from . import abi
 
-__all__ = ["load_library", "library_path", "abi"]
+__all__ = ["load_library", "load_library_for", "library_path", "abi"]
 
 _PKG = Path(__file__).resolve().parent
 _lib = None
 
 
-def library_path() -> Path:
-    return _PKG / "lib" / "libtenzo_runtime.so"
+def library_path(family: str | None = None) -> Path:
+    return _PKG / "lib" / (f"libtenzo_{family}.so" if family else "libtenzo_runtime.so")
 
 
-def load_library(build_if_missing: bool = True):
-    """dlopen libtenzo_runtime.so and declare every prototype. Raises if it cannot be loaded."""
+def load_library(build_if_missing: bool = True, family: str | None = None):
+    """dlopen libtenzo_runtime.so and declare every prototype. Raises if it cannot be loaded.
+
+    `family`: when the library with every model family is not there yet, a library with this one alone will do (built
+    if missing); whichever was loaded first stays."""
     global _lib
     if _lib is not None:
         return _lib
@@ -32,11 +36,18 @@ def load_library(build_if_missing: bool = True):
     if not path.exists():
         if not build_if_missing:
             raise RuntimeError(f"{path} is missing: run `python -m tenzo_b200.build` (there is no CPU fallback)")
-        from .build import build
-        build()
+        from .build import build, build_family
+        path = build_family(family) if family else build()
     L = C.CDLL(str(path), mode=os.RTLD_GLOBAL)
-    abi.declare_tenzo_abi(L)
-    abi.declare_ext_abi(L)
-    abi.declare_kernel_abi(L)
+    abi.declare_tenzo_abi(abi.present(L))
+    abi.declare_ext_abi(abi.present(L))
+    abi.declare_kernel_abi(abi.present(L))
     _lib = L
     return L
+
+
+def load_library_for(model_dir):
+    """The library that serves the model in a folder (its config.json names the architecture)."""
+    from .build import ARCHITECTURES
+    arch = json.loads((Path(model_dir) / "config.json").read_text()).get("architecture")
+    return load_library(family=ARCHITECTURES.get(arch))

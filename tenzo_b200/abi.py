@@ -6,6 +6,7 @@ used to drive this repository's library and, in tests, the compiled reference.
 from __future__ import annotations
 
 import ctypes as C
+from types import SimpleNamespace
 
 c_f32p = C.POINTER(C.c_float)
 c_i8p = C.POINTER(C.c_int8)
@@ -80,8 +81,10 @@ EXT_SYMBOLS = [
     "tenzo_ext_kv_fill_random", "tenzo_ext_set_seq_len", "tenzo_ext_get_seq_len", "tenzo_ext_read_buffer",
     "tenzo_ext_write_x", "tenzo_ext_run_layer", "tenzo_ext_synchronize", "tenzo_ext_last_device_ms",
     "tenzo_ext_kernel_launches", "tenzo_ext_last_error", "tenzo_ext_bench_gemv_stack", "tenzo_ext_rope_tables", "tenzo_ext_parse_manifest", "tenzo_ext_sample_pairs", "tenzo_ext_prefill_chunk",
-    "tenzo_ext_persistent_phase_ns",
+    "tenzo_ext_persistent_phase_ns", "tenzo_ext_open_model", "tenzo_ext_architecture", "tenzo_ext_get_config", "tenzo_ext_forward",
+    "tenzo_ext_reset_seq",
 ]
+COMPUTE = {"bfloat16": 0, "float32": 1}
 KERNEL_SYMBOLS = [
     "tenzo_cuda_tl1_gemv", "tenzo_cuda_tl1_gemv_ksplit", "tenzo_cuda_tl1_gemm_ksplit", "tenzo_cuda_tl1_gemm_layout", "tenzo_cuda_tl1_gemv_workspace_bytes", "tenzo_cuda_tl1_gemv_take_timeouts", "tenzo_cuda_selftest_wait_expiry", "tenzo_cuda_rmsnorm_quant", "tenzo_cuda_attention_int8",
     "tenzo_cuda_attention_heads_per_cta", "tenzo_cuda_attention_take_timeouts", "tenzo_cuda_attention_workspace_bytes", "tenzo_cuda_lm_head_i8", "tenzo_cuda_lm_head_scratch_bytes",
@@ -90,6 +93,19 @@ KERNEL_SYMBOLS = [
     "tenzo_cuda_topk_candidates", "tenzo_cuda_topk_max_candidates",
 ]
 HAL_SYMBOLS = ["tenzo_hal_initialize", "tenzo_hal_bitlinear_tl1_host", "tenzo_hal_rmsnorm_host", "tenzo_hal_gemm_f32_host", "tenzo_hal_call_count"]
+
+
+class present:
+    """A library seen through the prototypes below: entry points it was not built with are skipped."""
+
+    def __init__(self, lib):
+        object.__setattr__(self, "_lib", lib)
+
+    def __getattr__(self, name):
+        try:
+            return getattr(self._lib, name)
+        except AttributeError:
+            return SimpleNamespace()
 
 
 def declare_tenzo_abi(L):
@@ -143,6 +159,11 @@ def declare_ext_abi(L):
     L.tenzo_ext_rope_tables.restype, L.tenzo_ext_rope_tables.argtypes = i32, [i32, i32, f32, c_f32p, c_f32p]
     L.tenzo_ext_sample_pairs.restype, L.tenzo_ext_sample_pairs.argtypes = i32, [c_f32p, c_i32p, i32, C.POINTER(TenzoSampling), f32]
     L.tenzo_ext_prefill_chunk.restype, L.tenzo_ext_prefill_chunk.argtypes = i32, [vp, c_i32p, i32]
+    L.tenzo_ext_open_model.restype, L.tenzo_ext_open_model.argtypes = vp, [C.c_char_p, C.POINTER(TenzoExtOptions), i32]
+    L.tenzo_ext_architecture.restype, L.tenzo_ext_architecture.argtypes = C.c_char_p, [i32]
+    L.tenzo_ext_get_config.restype, L.tenzo_ext_get_config.argtypes = i32, [vp, C.POINTER(TenzoConfig)]
+    L.tenzo_ext_forward.restype, L.tenzo_ext_forward.argtypes = i32, [vp, i32, c_i32p, i32, c_i32p, i32, c_f32p]
+    L.tenzo_ext_reset_seq.restype, L.tenzo_ext_reset_seq.argtypes = i32, [vp, i32]
     L.tenzo_ext_parse_manifest.restype = i32
     L.tenzo_ext_parse_manifest.argtypes = [C.c_char_p, C.POINTER(C.c_ulonglong), i32, C.POINTER(i32), c_f32p, i32, C.POINTER(i32)]
     return L

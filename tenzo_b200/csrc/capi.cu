@@ -12,6 +12,7 @@
 #include "../../include/tenzo_ext.h"
 #include "../../include/tenzo_kernels.h"
 #include "capi_common.h"
+#include "model_registry.h"
 #include "sampler.h"
 
 using tz::guarded;
@@ -101,6 +102,50 @@ int tenzo_generate_step(tenzo_engine_t engine, int cur_token, const tenzo_sampli
 // ---------------------------------------------------------------------------------------------
 // extension
 // ---------------------------------------------------------------------------------------------
+
+tenzo_engine_t tenzo_ext_open_model(const char* model_dir, const tenzo_ext_options_t* opt, int compute) {
+    tenzo_engine_t handle = nullptr;
+    guarded([&]() -> tenzo_status_t {
+        if (!model_dir || (compute != TENZO_COMPUTE_BF16 && compute != TENZO_COMPUTE_F32)) throw std::invalid_argument("bad model folder or compute type");
+        int n_dev = 0;
+        if (cudaGetDeviceCount(&n_dev) != cudaSuccess || n_dev == 0)
+            throw std::runtime_error("no CUDA device is visible; this library has no CPU path");
+        tz::OpenOptions o;
+        o.dir = model_dir;
+        o.opt = opt ? *opt : tenzo_ext_default_options();
+        o.compute = compute;
+        handle = new tenzo_engine_opaque{tz::open_model(o)};
+        return TENZO_SUCCESS;
+    });
+    return handle;
+}
+
+const char* tenzo_ext_architecture(int index) {
+    const auto& f = tz::model_families();
+    return index >= 0 && index < (int)f.size() ? f[index].architecture : nullptr;
+}
+
+tenzo_status_t tenzo_ext_get_config(tenzo_engine_t engine, tenzo_config_t* out) {
+    if (!live(engine) || !out) return TENZO_ERROR_INVALID_ARGUMENT;
+    *out = engine->impl->cfg;
+    return TENZO_SUCCESS;
+}
+
+tenzo_status_t tenzo_ext_forward(tenzo_engine_t engine, int seq, const int* tokens, int n, const int* want, int n_want, float* logits) {
+    if (!live(engine) || !tokens || n_want < 0 || (n_want > 0 && (!want || !logits))) return TENZO_ERROR_INVALID_ARGUMENT;
+    return guarded([&]() -> tenzo_status_t {
+        engine->impl->forward(seq, tokens, n, want, n_want, logits);
+        return TENZO_SUCCESS;
+    });
+}
+
+tenzo_status_t tenzo_ext_reset_seq(tenzo_engine_t engine, int seq) {
+    if (!live(engine) || seq < 0 || seq >= engine->impl->batch) return TENZO_ERROR_INVALID_ARGUMENT;
+    return guarded([&]() -> tenzo_status_t {
+        engine->impl->reset_seq(seq);
+        return TENZO_SUCCESS;
+    });
+}
 
 int tenzo_ext_batch(tenzo_engine_t engine) { return live(engine) ? engine->impl->batch : 0; }
 

@@ -6,6 +6,7 @@
 #include <string>
 
 #include "engine_core.h"
+#include "model_registry.h"
 
 namespace tz {
 
@@ -23,6 +24,12 @@ inline tenzo_status_t guarded(F&& f) {
     } catch (const std::out_of_range& e) {
         tz::set_error(e.what());
         return TENZO_ERROR_INVALID_ARGUMENT;
+    } catch (const IoError& e) {
+        set_error(e.what());
+        return TENZO_ERROR_IO;
+    } catch (const ParseError& e) {
+        set_error(e.what());
+        return TENZO_ERROR_MODEL_PARSE;
     } catch (const std::exception& e) {
         tz::set_error(e.what());
         const std::string m = e.what();

@@ -1,0 +1,199 @@
+// Matrix products with bf16 weights for the hybrid decoders: few rows (decode) as a weight-streaming GEMV, many fp32 rows
+// as a tiled FMA product; many bf16 rows go to the tensor cores (gemm_umma.cu). Also the greedy argmax over fp32 logits.
+#include "hybrid_common.cuh"
+#include "lm_head.cuh"
+
+namespace tz {
+
+constexpr int kGemvThreads = 256, kGemvWarps = kGemvThreads / 32, kGemvMaxRows = 8;
+
+template <typename T>
+__device__ __forceinline__ void gemm_store(const GemmArgs& a, int m, int n, float v) {
+    if (a.epilogue == GEMM_XIELU) reinterpret_cast<T*>(a.c)[(size_t)m * a.ld_c + n] = from_f<T>(xielu_f(v, a.act_pos, a.act_neg));
+    else reinterpret_cast<float*>(a.c)[(size_t)m * a.ld_c + n] = v;
+}
+
+__device__ __forceinline__ int gemm_segment(const GemmArgs& a, int n) {
+    int s = 0;
+    while (s + 1 < a.n_seg && n >= a.seg_end[s]) ++s;
+    return s;
+}
+
+// One warp per output column n (= weight row), all MR activation rows at once. The first 2048 weights of the row are in
+// registers before the kernel waits for its producer: weights do not depend on it.
+template <typename T, int MR>
+__global__ void __launch_bounds__(kGemvThreads) gemv_kernel(const GemmArgs a) {
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int n = blockIdx.x * kGemvWarps + warp;
+    const bool live = n < a.N;
+    const bf16* wrow = a.w + (size_t)(live ? n : 0) * a.ld_k;
+    const int chunks = a.ld_k / 8;
+    constexpr int kPre = 8;
+    uint4 pre[kPre];
+#pragma unroll
+    for (int i = 0; i < kPre; ++i)
+        if (live && i * 32 + lane < chunks) pre[i] = ld_stream_u4(wrow + (size_t)(i * 32 + lane) * 8);
+    pdl_wait();
+    pdl_launch_dependents();
+    if (!live) return;
+    const T* x = reinterpret_cast<const T*>(a.a) + (size_t)gemm_segment(a, n) * a.a_seg_stride;
+    float acc[MR];
+#pragma unroll
+    for (int m = 0; m < MR; ++m) acc[m] = 0.0f;
+    auto step = [&](const uint4& wv, int ch) {
+        float w[8];
+        unpack8(wv, w);
+#pragma unroll
+        for (int m = 0; m < MR; ++m) {
+            if (m < a.M) {
+                float xv[8];
+                load8(x + (size_t)m * a.ld_k + (size_t)ch * 8, xv);
+#pragma unroll
+                for (int j = 0; j < 8; ++j) acc[m] = fmaf(w[j], xv[j], acc[m]);
+            }
+        }
+    };
+#pragma unroll
+    for (int i = 0; i < kPre; ++i)
+        if (i * 32 + lane < chunks) step(pre[i], i * 32 + lane);
+    for (int ch = kPre * 32 + lane; ch < chunks; ch += 4 * 32) {
+        uint4 w[4];
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+            if (ch + u * 32 < chunks) w[u] = ld_stream_u4(wrow + (size_t)(ch + u * 32) * 8);
+#pragma unroll
+        for (int u = 0; u < 4; ++u)
+            if (ch + u * 32 < chunks) step(w[u], ch + u * 32);
+    }
+#pragma unroll
+    for (int m = 0; m < MR; ++m) acc[m] = warp_sum(acc[m]);
+    if (lane == 0) {
+#pragma unroll
+        for (int m = 0; m < MR; ++m)
+            if (m < a.M) gemm_store<T>(a, m, n, acc[m]);
+    }
+}
+
+// 64 x 64 output tile, 16-wide K steps, 4 x 4 outputs per thread.
+template <typename T>
+__global__ void __launch_bounds__(256) gemm_fma_kernel(const GemmArgs a) {
+    __shared__ float s_a[16][68], s_w[16][68];
+    const int n0 = blockIdx.x * 64, m0 = blockIdx.y * 64, tid = threadIdx.x, tx = tid & 15, ty = tid >> 4;
+    pdl_wait();
+    pdl_launch_dependents();
+    // a segment border inside the tile: columns of both segments are computed from their own A, tile by tile of 64 columns
+    const int s_first = gemm_segment(a, n0), s_last = gemm_segment(a, min(n0 + 63, a.N - 1));
+    for (int seg = s_first; seg <= s_last; ++seg) {
+        const T* x = reinterpret_cast<const T*>(a.a) + (size_t)seg * a.a_seg_stride;
+        float acc[4][4] = {};
+        for (int k0 = 0; k0 < a.ld_k; k0 += 16) {
+            {
+                const int r = tid >> 2, kk = (tid & 3) * 4;
+                const int m = m0 + r, n = n0 + r;
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    s_a[kk + j][r] = m < a.M ? to_f(x[(size_t)m * a.ld_k + k0 + kk + j]) : 0.0f;
+                    s_w[kk + j][r] = n < a.N ? to_f(a.w[(size_t)n * a.ld_k + k0 + kk + j]) : 0.0f;
+                }
+            }
+            __syncthreads();
+#pragma unroll
+            for (int k = 0; k < 16; ++k) {
+                const float4 av = *reinterpret_cast<const float4*>(&s_a[k][ty * 4]), wv = *reinterpret_cast<const float4*>(&s_w[k][tx * 4]);
+                const float af[4] = {av.x, av.y, av.z, av.w}, wf[4] = {wv.x, wv.y, wv.z, wv.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(af[i], wf[j], acc[i][j]);
+            }
+            __syncthreads();
+        }
+#pragma unroll
+        for (int i = 0; i < 4; ++i)
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                const int m = m0 + ty * 4 + i, n = n0 + tx * 4 + j;
+                if (m < a.M && n < a.N && gemm_segment(a, n) == seg) gemm_store<T>(a, m, n, acc[i][j]);
+            }
+    }
+}
+
+template <typename T>
+static int launch_gemv(const GemmArgs& a, cudaStream_t st) {
+    const dim3 grid((a.N + kGemvWarps - 1) / kGemvWarps), block(kGemvThreads);
+    auto go = [&](auto kernel) { return launch_kernel(kernel, grid, block, 0, st, a.use_pdl, 1, a); };
+    if (a.M == 1) return go(gemv_kernel<T, 1>);
+    if (a.M == 2) return go(gemv_kernel<T, 2>);
+    if (a.M <= 4) return go(gemv_kernel<T, 4>);
+    return go(gemv_kernel<T, 8>);
+}
+
+int launch_gemm(const GemmArgs& a, cudaStream_t st) {
+    if (a.M <= 0 || a.N <= 0) return 0;
+    if (a.ld_k % 64 || a.n_seg < 1 || a.n_seg > 8) return -1;
+    if (!a.f32 && gemm_umma_applicable(a)) return launch_gemm_umma(a, st);
+    if (a.f32 && a.M > kGemvMaxRows) {
+        gemm_fma_kernel<float><<<dim3((a.N + 63) / 64, (a.M + 63) / 64), 256, 0, st>>>(a);
+        return (int)cudaGetLastError();
+    }
+    // groups of up to eight rows; the weights of the second group come from L2
+    for (int m0 = 0; m0 < a.M; m0 += kGemvMaxRows) {
+        GemmArgs p = a;
+        p.M = a.M - m0 < kGemvMaxRows ? a.M - m0 : kGemvMaxRows;
+        const size_t es = a.f32 ? 4 : 2, cs = a.epilogue == GEMM_STORE ? 4 : es;
+        p.a = static_cast<const char*>(a.a) + (size_t)m0 * a.ld_k * es;
+        p.c = static_cast<char*>(a.c) + (size_t)m0 * a.ld_c * cs;
+        if (int rc = a.f32 ? launch_gemv<float>(p, st) : launch_gemv<bf16>(p, st)) return rc;
+    }
+    return 0;
+}
+
+// ---- greedy argmax ------------------------------------------------------------------------------------------------------
+constexpr int kArgmaxSplits = 64;
+
+__device__ __forceinline__ LmBest block_best(LmBest b) {
+    __shared__ LmBest s[8];
+#pragma unroll
+    for (int m = 16; m > 0; m >>= 1) {
+        const float v = __shfl_xor_sync(0xffffffffu, b.val, m);
+        const int i = __shfl_xor_sync(0xffffffffu, b.idx, m);
+        if (better(v, i, b.val, b.idx)) { b.val = v; b.idx = i; }
+    }
+    if ((threadIdx.x & 31) == 0) s[threadIdx.x >> 5] = b;
+    __syncthreads();
+    if (threadIdx.x == 0)
+        for (int w = 1; w < (int)(blockDim.x >> 5); ++w)
+            if (better(s[w].val, s[w].idx, b.val, b.idx)) b = s[w];
+    return b;
+}
+
+__global__ void __launch_bounds__(256) argmax_part_kernel(const float* __restrict__ logits, int vocab, LmBest* part) {
+    const float* row = logits + (size_t)blockIdx.y * vocab;
+    LmBest b = {-INFINITY, 0x7fffffff};
+    for (int i = blockIdx.x * 256 + threadIdx.x; i < vocab; i += gridDim.x * 256)
+        if (better(row[i], i, b.val, b.idx)) { b.val = row[i]; b.idx = i; }
+    b = block_best(b);
+    if (threadIdx.x == 0) part[(size_t)blockIdx.y * gridDim.x + blockIdx.x] = b;
+}
+
+__global__ void __launch_bounds__(64) argmax_finish_rows_kernel(const LmBest* part, int n, int* out) {
+    LmBest b = {-INFINITY, 0x7fffffff};
+    for (int i = threadIdx.x; i < n; i += 64) {
+        const LmBest p = part[(size_t)blockIdx.x * n + i];
+        if (better(p.val, p.idx, b.val, b.idx)) b = p;
+    }
+    b = block_best(b);
+    if (threadIdx.x == 0) out[blockIdx.x] = b.idx == 0x7fffffff ? 0 : b.idx;
+}
+
+size_t argmax_scratch_bytes(int rows) { return (size_t)rows * kArgmaxSplits * sizeof(LmBest); }
+
+int launch_argmax(const float* logits, int vocab, int rows, int* out, void* scratch, cudaStream_t st) {
+    int splits = (vocab + 1023) / 1024;
+    if (splits > kArgmaxSplits) splits = kArgmaxSplits;
+    argmax_part_kernel<<<dim3(splits, rows), 256, 0, st>>>(logits, vocab, static_cast<LmBest*>(scratch));
+    argmax_finish_rows_kernel<<<rows, 64, 0, st>>>(static_cast<const LmBest*>(scratch), splits, out);
+    return (int)cudaGetLastError();
+}
+
+}  // namespace tz

@@ -31,6 +31,7 @@
 #include "../../include/tenzo_kernels.h"
 #include "common.cuh"
 #include "engine.h"
+#include "model_registry.h"
 
 namespace tz {
 
@@ -281,6 +282,30 @@ tenzo_status_t load_model_files(Engine& e, const char* weights_path, const char*
     e.invalidate_graphs();
     return TENZO_SUCCESS;
 }
+
+// A BitNet folder: config.json with the fields of tenzo_config_t, weights.bin and model.mlir beside it.
+static EngineCore* open_bitnet(const Json& c, const OpenOptions& o) {
+    if (o.compute != TENZO_COMPUTE_BF16) throw std::invalid_argument("BitNet models compute in their own integer arithmetic only");
+    tenzo_config_t cfg = {};
+    cfg.hidden_size = c.at("hidden_size").integer();
+    cfg.num_q_heads = c.at("num_q_heads").integer();
+    cfg.num_kv_heads = c.at("num_kv_heads").integer();
+    cfg.head_dim = c.at("head_dim").integer();
+    cfg.num_layers = c.at("num_layers").integer();
+    cfg.ffn_dim = c.at("ffn_dim").integer();
+    cfg.vocab_size = c.at("vocab_size").integer();
+    cfg.max_seq_len = c.at("max_seq_len").integer();
+    cfg.kv_mode = c.has("kv_mode") && c.at("kv_mode").string() == "paged_int8" ? "paged_int8" : "int8_fused";
+    Engine* e = new Engine(cfg, o.opt);
+    try {
+        if (load_model_files(*e, (o.dir + "/weights.bin").c_str(), (o.dir + "/model.mlir").c_str()) != TENZO_SUCCESS) throw IoError(g_last_error);
+    } catch (...) {
+        delete e;
+        throw;
+    }
+    return e;
+}
+static const ModelRegistration registration({"BitNet", open_bitnet});
 
 }  // namespace tz
 

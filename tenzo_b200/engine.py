@@ -11,7 +11,7 @@ from typing import Sequence
 
 import numpy as np
 
-from . import abi, load_library
+from . import abi, load_library, load_library_for
 
 
 def _p(a: np.ndarray | None, ty):
@@ -35,6 +35,21 @@ class Engine:
         if not self._h:
             raise RuntimeError("Failed to initialize Tenzo execution engine: " + self.last_error())
         self.batch = batch
+
+    @classmethod
+    def open(cls, model_dir, *, compute: str = "bfloat16", batch: int = 1, use_graph: int = -1, use_pdl: int = -1) -> "Engine":
+        """The model in a folder; its config.json names the architecture. compute: "bfloat16" or "float32"."""
+        self = cls.__new__(cls)
+        self._h = None
+        self.lib = load_library_for(model_dir)
+        opt = abi.TenzoExtOptions(batch, 0.0, use_graph, use_pdl, -1, -1)
+        self._h = self.lib.tenzo_ext_open_model(str(model_dir).encode(), C.byref(opt), abi.COMPUTE[compute])
+        if not self._h:
+            raise RuntimeError(f"Failed to open the model in {model_dir}: " + self.last_error())
+        self.config = abi.TenzoConfig()
+        self.lib.tenzo_ext_get_config(self._h, C.byref(self.config))
+        self.batch = batch
+        return self
 
     # -- lifetime ---------------------------------------------------------------------------
     def close(self):
@@ -116,6 +131,32 @@ class Engine:
         """All of `tokens` (consecutive tokens of the one sequence) through the layers together."""
         t = np.ascontiguousarray(tokens, dtype=np.int32)
         self._check(self.lib.tenzo_ext_prefill_chunk(self._h, _p(t, abi.c_i32p), int(t.size)), "tenzo_ext_prefill_chunk")
+
+    def forward(self, tokens: Sequence[int], want: Sequence[int] = (), seq: int = 0) -> np.ndarray:
+        """The next tokens of a sequence; returns the logits at the places `want` (ascending) among them."""
+        t = np.ascontiguousarray(tokens, dtype=np.int32)
+        w = np.ascontiguousarray(want, dtype=np.int32)
+        out = np.zeros((w.size, self.config.vocab_size), np.float32)
+        self._check(self.lib.tenzo_ext_forward(self._h, seq, _p(t, abi.c_i32p), int(t.size), _p(w, abi.c_i32p) if w.size else None,
+                                               int(w.size), _p(out, abi.c_f32p) if w.size else None), "tenzo_ext_forward")
+        return out
+
+    def reset_seq(self, seq: int = 0):
+        self._check(self.lib.tenzo_ext_reset_seq(self._h, seq), "tenzo_ext_reset_seq")
+
+    def generate(self, prompt: Sequence[int], n: int, params: abi.TenzoSampling | None = None) -> list[int]:
+        """n tokens after a prompt: all of it but its last token as one chunk, then one decode step per token. Greedy unless
+        sampling parameters are given."""
+        prompt = [int(t) for t in prompt]
+        greedy = abi.TenzoSampling(0.0, 0.9, 40, 1.0)
+        if len(prompt) > 1:
+            self.prefill_chunk(prompt[:-1])
+        cur, seen, out = prompt[-1], list(prompt), []
+        for _ in range(n):
+            cur = self.generate_step(cur, params or greedy, seen)
+            seen.append(cur)
+            out.append(cur)
+        return out
 
     def generate_steps(self, cur_tokens: Sequence[int]) -> np.ndarray:
         t = np.ascontiguousarray(cur_tokens, dtype=np.int32)
