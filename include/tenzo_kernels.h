@@ -227,6 +227,120 @@ TENZO_API int tenzo_cuda_embedding_i8(const int8_t* w, const float* row_scales, 
  * the [N/64][K/2][32] layout above. */
 TENZO_API int tenzo_cuda_tl1_pack_rows2bit(const uint8_t* raw, int N, int K, uint8_t* packed, void* stream);
 
+/* ---- Pieces of the hybrid decoders ---------------------------------------------------------------------------------------
+ * (No counterpart in the reference.) Two storage types: what enters a matrix product and cached keys / values are bf16
+ * (f32 = 0) or fp32 (f32 = 1), "storage type" below; weights of matrix products are bf16 in both cases. Residual, norms,
+ * scores, softmax, decays and recurrent states are fp32 always, and the fp32 path is plain FMA arithmetic.
+ *
+ * decode = 1: one row per sequence, row b uses the carried state of sequence b (at b * its stride), in place. decode = 0: M
+ * consecutive rows of one sequence; carried convolution inputs are read from *_in and their successors written to *_out,
+ * a different buffer, because rows of the same launch still need the old ones. */
+
+/* Row kernel: x = source; x_out = x; u = x / sqrt(mean(x^2) + eps) * gain; y = u + conv(u); out = y, or with mu the mixes
+ * out_s = y + (y of the row before - y) * mu_s. */
+typedef struct {
+    const int *tokens, *pos;          /* not NULL: x = embed[token] + pos_table[pos] */
+    const void *embed, *pos_table;    /* bf16 [vocab][width], [n_pos][width] */
+    int vocab, n_pos;
+    const float *x_in;                /* otherwise x = x_in (+ y0) (+ 0.5 (y0 / rms(y0) * w0 + y1 / rms(y1) * w1) when y1) */
+    const float *y0, *y1, *w0, *w1;
+    int ld_y;
+    float* x_out;                     /* [M][width], not x_in */
+    int width, M;
+    float eps, gain;
+    const float* conv_w;              /* [taps][width]; NULL: no convolution */
+    int taps;                         /* 1..16 */
+    const float* tail_in;             /* [taps-1][width] per sequence: u of the tokens before, oldest first */
+    float* tail_out;
+    const float* mu;                  /* [n_mix][width] or NULL */
+    int n_mix;
+    const float* prev_in;             /* [width] per sequence: y of the token before */
+    float* prev_out;
+    size_t seq_stride;                /* floats between the carried states of two sequences */
+    int decode;
+    void* out;                        /* storage type [max(n_mix,1)][M][ld_out] */
+    int ld_out;
+    int f32, use_pdl;
+} tenzo_rows_args;
+TENZO_API int tenzo_cuda_rows(const tenzo_rows_args* args, void* stream);
+
+/* c[m][n] = sum_k a[m][k] w[n][k]: a GEMV up to 8 rows, tcgen05 from 16 (bf16), tiled FMA for fp32. Rows of w in segment s
+ * (n < seg_end[s]) multiply the matrix at a + s * a_seg_stride; on tcgen05 segments end at multiples of 128. */
+enum { TENZO_GEMM_STORE = 0, TENZO_GEMM_XIELU = 1 };
+typedef struct {
+    const void* a;                    /* storage type, rows of ld_k elements, padding finite */
+    const void* w;                    /* bf16 [N][ld_k], padding zero; ld_k a multiple of 64 */
+    int M, N, ld_k;
+    int n_seg, seg_end[8];
+    size_t a_seg_stride;              /* elements, a multiple of ld_k */
+    int epilogue;                     /* XIELU: z > 0: act_pos z^2 + z/2, else act_neg (exp(z) - 1 - z) + z/2 */
+    float act_pos, act_neg;
+    void* c;                          /* STORE: float [M][ld_c]; XIELU: storage type */
+    int ld_c;
+    int f32, use_pdl;
+    void* workspace;                  /* tenzo_cuda_gemm_workspace_bytes(), zeroed once; NULL keeps off the tensor cores */
+    size_t workspace_bytes;
+} tenzo_gemm_args;
+TENZO_API int tenzo_cuda_gemm(const tenzo_gemm_args* args, void* stream);
+TENZO_API size_t tenzo_cuda_gemm_workspace_bytes(void);
+TENZO_API int tenzo_cuda_gemm_take_timeouts(void);
+
+/* Causal sliding-window attention over grouped heads: a convolution of `taps` on every q, k, v channel, score
+ * scale * q.k - slope_h * distance with slope_h = 2^(-slope_base (h+1) / heads) (slope_base 0: no bias), keys up to
+ * window - 1 back, softmax denominator sum exp(score) + sink. */
+typedef struct {
+    const float *q, *k, *v;           /* projections, row stride ld */
+    int ld;
+    const float *conv_q, *conv_k, *conv_v;   /* [taps][channels] */
+    int taps;
+    const float* tail_in;             /* [taps-1][q|k|v channels] per sequence, oldest first */
+    float* tail_out;
+    size_t tail_seq_stride;
+    int heads, kv_heads, dim, vdim;   /* head sizes up to 256 */
+    float scale, slope_base, sink;
+    int window, ring;                 /* ring >= min(window, longest sequence): slot = position % ring */
+    void *ring_k, *ring_v;            /* storage type [kv_heads][ring][head size rounded up to 8] per sequence, padding zero */
+    size_t ring_k_stride, ring_v_stride;     /* elements between two sequences */
+    const int* pos;                   /* decode: position of every row (device) */
+    int pos0;                         /* chunk: position of the first row */
+    int M, decode;
+    void* out;                        /* storage type [M][ld_out], head after head */
+    int ld_out;
+    void *lin_q, *lin_k, *lin_v;      /* chunk scratch, storage type: [M][heads][dim8], [kv_heads][ring + M][dim8], [..][vdim8] */
+    int f32, use_pdl;
+} tenzo_window_attention_args;
+TENZO_API int tenzo_cuda_window_attention(const tenzo_window_attention_args* args, void* stream);
+
+/* S_t = diag(w_t) S_(t-1) + k_t v_t^T; o_t = S_t^T q_t, or with a bonus u o_t = (S_(t-1) + diag(u) k_t v_t^T)^T q_t; then
+ * out = o / sqrt(mean over the head(o^2) + eps) * norm * silu(g). */
+enum { TENZO_DECAY_CONST = 0, TENZO_DECAY_SIGMOID_ROOT = 1, TENZO_DECAY_EXP_EXP = 2 };
+typedef struct {
+    const float *q, *k, *v, *g;       /* row stride ld */
+    int ld;
+    float q_scale, k_scale;
+    int heads, dim, vdim;             /* up to 256 */
+    int decay_kind;
+    const float* decay;               /* CONST: w = decay[head] */
+    const float* low;                 /* others: z = up f(low) + bias over `rank` values per row (row stride ld); */
+    const void* up;                   /* bf16 [heads*dim][rank] */
+    const float* bias;                /* SIGMOID_ROOT: f(x) = x, w = sigmoid(z)^(1/tau); EXP_EXP: f = tanh, w = exp(-exp(z)) */
+    int rank;
+    float tau;
+    const float* bonus;               /* [heads*dim] or NULL */
+    const float* norm;                /* [vdim], or [heads*vdim] with norm_per_head, or NULL */
+    int norm_per_head;
+    float eps;
+    float* state;                     /* [heads][dim][vdim rounded up to 4] per sequence */
+    size_t state_seq_stride;          /* a multiple of 4 */
+    int M, decode;
+    void* out;                        /* storage type [M][ld_out] */
+    int ld_out;
+    float *w_rows, *o_rows, *part;    /* chunk scratch: [M][heads*dim], [M][heads*vdim], tenzo_cuda_linear_scan_part_floats() */
+    int f32, use_pdl;
+} tenzo_scan_args;
+TENZO_API int tenzo_cuda_linear_scan(const tenzo_scan_args* args, void* stream);
+TENZO_API size_t tenzo_cuda_linear_scan_part_floats(int M, int heads, int dim, int vdim);
+
 #ifdef __cplusplus
 }
 #endif

@@ -49,5 +49,8 @@ def load_library(build_if_missing: bool = True, family: str | None = None):
 def load_library_for(model_dir):
     """The library that serves the model in a folder (its config.json names the architecture)."""
     from .build import ARCHITECTURES
-    arch = json.loads((Path(model_dir) / "config.json").read_text()).get("architecture")
+    try:
+        arch = json.loads((Path(model_dir) / "config.json").read_text()).get("architecture")
+    except (OSError, ValueError, AttributeError):
+        arch = None                                        # opening the folder reports what is wrong with it
     return load_library(family=ARCHITECTURES.get(arch))

@@ -70,6 +70,34 @@ class AttentionArgs(C.Structure):
     ]
 
 
+def _fields(spec: str):
+    """'name:type ...' -> ctypes fields; p pointer, i int, f float, z size_t."""
+    kinds = {"p": C.c_void_p, "i": C.c_int, "f": C.c_float, "z": C.c_size_t, "i8": C.c_int * 8}
+    return [(n, kinds[k]) for n, k in (e.split(":") for e in spec.split())]
+
+
+class RowsArgs(C.Structure):
+    _fields_ = _fields("tokens:p pos:p embed:p pos_table:p vocab:i n_pos:i x_in:p y0:p y1:p w0:p w1:p ld_y:i x_out:p width:i M:i eps:f gain:f "
+                       "conv_w:p taps:i tail_in:p tail_out:p mu:p n_mix:i prev_in:p prev_out:p seq_stride:z decode:i out:p ld_out:i f32:i use_pdl:i")
+
+
+class GemmArgs(C.Structure):
+    _fields_ = _fields("a:p w:p M:i N:i ld_k:i n_seg:i seg_end:i8 a_seg_stride:z epilogue:i act_pos:f act_neg:f c:p ld_c:i f32:i use_pdl:i "
+                       "workspace:p workspace_bytes:z")
+
+
+class WindowAttentionArgs(C.Structure):
+    _fields_ = _fields("q:p k:p v:p ld:i conv_q:p conv_k:p conv_v:p taps:i tail_in:p tail_out:p tail_seq_stride:z heads:i kv_heads:i dim:i "
+                       "vdim:i scale:f slope_base:f sink:f window:i ring:i ring_k:p ring_v:p ring_k_stride:z ring_v_stride:z pos:p pos0:i M:i "
+                       "decode:i out:p ld_out:i lin_q:p lin_k:p lin_v:p f32:i use_pdl:i")
+
+
+class ScanArgs(C.Structure):
+    _fields_ = _fields("q:p k:p v:p g:p ld:i q_scale:f k_scale:f heads:i dim:i vdim:i decay_kind:i decay:p low:p up:p bias:p rank:i tau:f "
+                       "bonus:p norm:p norm_per_head:i eps:f state:p state_seq_stride:z M:i decode:i out:p ld_out:i w_rows:p o_rows:p part:p "
+                       "f32:i use_pdl:i")
+
+
 ENGINE_SYMBOLS = [
     "tenzo_get_version", "tenzo_default_config", "tenzo_default_sampling_params", "tenzo_create_engine",
     "tenzo_destroy_engine", "tenzo_reset", "tenzo_get_seq_len", "tenzo_set_layer_weights", "tenzo_set_final_norm",
@@ -90,7 +118,8 @@ KERNEL_SYMBOLS = [
     "tenzo_cuda_attention_heads_per_cta", "tenzo_cuda_attention_take_timeouts", "tenzo_cuda_attention_workspace_bytes", "tenzo_cuda_lm_head_i8", "tenzo_cuda_lm_head_scratch_bytes",
     "tenzo_cuda_embedding_i8", "tenzo_cuda_tl1_pack_rows2bit", "tenzo_cuda_lm_head_i8_static",
     "tenzo_cuda_lm_head_static_max_batch", "tenzo_cuda_lm_head_take_timeouts", "tenzo_cuda_repetition_penalty",
-    "tenzo_cuda_topk_candidates", "tenzo_cuda_topk_max_candidates",
+    "tenzo_cuda_topk_candidates", "tenzo_cuda_topk_max_candidates", "tenzo_cuda_rows", "tenzo_cuda_gemm", "tenzo_cuda_gemm_workspace_bytes",
+    "tenzo_cuda_gemm_take_timeouts", "tenzo_cuda_window_attention", "tenzo_cuda_linear_scan", "tenzo_cuda_linear_scan_part_floats",
 ]
 HAL_SYMBOLS = ["tenzo_hal_initialize", "tenzo_hal_bitlinear_tl1_host", "tenzo_hal_rmsnorm_host", "tenzo_hal_gemm_f32_host", "tenzo_hal_call_count"]
 
@@ -195,6 +224,12 @@ def declare_kernel_abi(L):
     L.tenzo_cuda_lm_head_scratch_bytes.restype, L.tenzo_cuda_lm_head_scratch_bytes.argtypes = sz, [i32]
     L.tenzo_cuda_embedding_i8.restype, L.tenzo_cuda_embedding_i8.argtypes = i32, [vp, vp, i32, vp, i32, vp, i32, i32, vp]
     L.tenzo_cuda_tl1_pack_rows2bit.restype, L.tenzo_cuda_tl1_pack_rows2bit.argtypes = i32, [vp, i32, i32, vp, vp]
+    for name, args in (("rows", RowsArgs), ("gemm", GemmArgs), ("window_attention", WindowAttentionArgs), ("linear_scan", ScanArgs)):
+        fn = getattr(L, "tenzo_cuda_" + name)
+        fn.restype, fn.argtypes = i32, [C.POINTER(args), vp]
+    L.tenzo_cuda_gemm_workspace_bytes.restype, L.tenzo_cuda_gemm_workspace_bytes.argtypes = sz, []
+    L.tenzo_cuda_gemm_take_timeouts.restype, L.tenzo_cuda_gemm_take_timeouts.argtypes = i32, []
+    L.tenzo_cuda_linear_scan_part_floats.restype, L.tenzo_cuda_linear_scan_part_floats.argtypes = sz, [i32, i32, i32, i32]
     L.tenzo_hal_initialize.restype, L.tenzo_hal_initialize.argtypes = i32, []
     L.tenzo_hal_bitlinear_tl1_host.restype = i32
     L.tenzo_hal_bitlinear_tl1_host.argtypes = [c_f32p, c_u8p, c_f32p, sz, sz, sz, f32]

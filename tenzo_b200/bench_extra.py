@@ -12,6 +12,9 @@
   decode_tp     greedy decode of the synthetic 8B shape (32 layers, 4096/14336, 32q/8kv, vocab 128256), batch 32,
                 context 2048, tensor-parallel over the launched ranks (row splits + NCCL all-gathers; tenzo_b200/tp.py).
 
+  sozopel       the Sozopel hybrid decoder beside BitNet at equal size: prompt and decode throughput at three widths, and
+                every kernel alone against its roofline (tenzo_b200/bench_hybrid.py).
+
 Each prints one JSON line in the same format as the default workload.
 """
 from __future__ import annotations
@@ -479,8 +482,14 @@ def run_decode_tp(args):
         dist.destroy_process_group()
 
 
+def run_sozopel(args):
+    from . import bench_hybrid
+    return bench_hybrid.run(args)
+
+
 def run(args):
-    fn = {"gemv": run_gemv, "lm_head": run_lm_head, "gemm": run_gemm, "attn": run_attn, "decode_batch": run_decode_batch, "decode_tp": run_decode_tp}.get(args.workload)
+    fn = {"gemv": run_gemv, "lm_head": run_lm_head, "gemm": run_gemm, "attn": run_attn, "decode_batch": run_decode_batch, "decode_tp": run_decode_tp,
+          "sozopel": run_sozopel}.get(args.workload)
     if fn is None:
         raise SystemExit(f"unknown workload {args.workload!r}")
     return fn(args)

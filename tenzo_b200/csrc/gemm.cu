@@ -9,7 +9,7 @@ constexpr int kGemvThreads = 256, kGemvWarps = kGemvThreads / 32, kGemvMaxRows =
 
 template <typename T>
 __device__ __forceinline__ void gemm_store(const GemmArgs& a, int m, int n, float v) {
-    if (a.epilogue == GEMM_XIELU) reinterpret_cast<T*>(a.c)[(size_t)m * a.ld_c + n] = from_f<T>(xielu_f(v, a.act_pos, a.act_neg));
+    if (a.epilogue == TENZO_GEMM_XIELU) reinterpret_cast<T*>(a.c)[(size_t)m * a.ld_c + n] = from_f<T>(xielu_f(v, a.act_pos, a.act_neg));
     else reinterpret_cast<float*>(a.c)[(size_t)m * a.ld_c + n] = v;
 }
 
@@ -26,7 +26,7 @@ __global__ void __launch_bounds__(kGemvThreads) gemv_kernel(const GemmArgs a) {
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int n = blockIdx.x * kGemvWarps + warp;
     const bool live = n < a.N;
-    const bf16* wrow = a.w + (size_t)(live ? n : 0) * a.ld_k;
+    const bf16* wrow = static_cast<const bf16*>(a.w) + (size_t)(live ? n : 0) * a.ld_k;
     const int chunks = a.ld_k / 8;
     constexpr int kPre = 8;
     uint4 pre[kPre];
@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(256) gemm_fma_kernel(const GemmArgs a) {
 #pragma unroll
                 for (int j = 0; j < 4; ++j) {
                     s_a[kk + j][r] = m < a.M ? to_f(x[(size_t)m * a.ld_k + k0 + kk + j]) : 0.0f;
-                    s_w[kk + j][r] = n < a.N ? to_f(a.w[(size_t)n * a.ld_k + k0 + kk + j]) : 0.0f;
+                    s_w[kk + j][r] = n < a.N ? to_f(static_cast<const bf16*>(a.w)[(size_t)n * a.ld_k + k0 + kk + j]) : 0.0f;
                 }
             }
             __syncthreads();
@@ -140,7 +140,7 @@ int launch_gemm(const GemmArgs& a, cudaStream_t st) {
     for (int m0 = 0; m0 < a.M; m0 += kGemvMaxRows) {
         GemmArgs p = a;
         p.M = a.M - m0 < kGemvMaxRows ? a.M - m0 : kGemvMaxRows;
-        const size_t es = a.f32 ? 4 : 2, cs = a.epilogue == GEMM_STORE ? 4 : es;
+        const size_t es = a.f32 ? 4 : 2, cs = a.epilogue == TENZO_GEMM_STORE ? 4 : es;
         p.a = static_cast<const char*>(a.a) + (size_t)m0 * a.ld_k * es;
         p.c = static_cast<char*>(a.c) + (size_t)m0 * a.ld_c * cs;
         if (int rc = a.f32 ? launch_gemv<float>(p, st) : launch_gemv<bf16>(p, st)) return rc;
@@ -197,3 +197,10 @@ int launch_argmax(const float* logits, int vocab, int rows, int* out, void* scra
 }
 
 }  // namespace tz
+
+extern "C" int tenzo_cuda_gemm(const tenzo_gemm_args* args, void* stream) {
+    if (!args) return TENZO_ERROR_INVALID_ARGUMENT;
+    tz::GemmArgs a;
+    static_cast<tenzo_gemm_args&>(a) = *args;
+    return tz::launch_gemm(a, static_cast<cudaStream_t>(stream));
+}

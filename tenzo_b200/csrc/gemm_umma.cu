@@ -41,7 +41,7 @@ __device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t da, uint64_t
 
 __device__ __forceinline__ void gu_store16(const GemmArgs& a, int n, int m0, const float (&v)[16]) {
     if (n >= a.N) return;
-    if (a.epilogue == GEMM_XIELU) {
+    if (a.epilogue == TENZO_GEMM_XIELU) {
         bf16* c = reinterpret_cast<bf16*>(a.c) + n;
 #pragma unroll
         for (int i = 0; i < 16; ++i)
@@ -199,7 +199,7 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
 }
 
 constexpr size_t kGuCounterBytes = 4096;
-size_t gemm_workspace_bytes() { return kGuCounterBytes + (size_t)kGuSplitTiles * kGuMaxN * kGuRows * 4; }
+constexpr size_t kGuWorkspaceBytes = kGuCounterBytes + (size_t)kGuSplitTiles * kGuMaxN * kGuRows * 4;
 
 bool gemm_umma_applicable(const GemmArgs& a) {
     if (a.f32 || a.M < kGemmUmmaMinRows || a.ld_k % kGuKc || !a.workspace) return false;
@@ -249,11 +249,13 @@ int launch_gemm_umma(const GemmArgs& a, cudaStream_t st) {
     return (int)cudaLaunchKernelEx(&cfg, gemm_umma_kernel, L, wmap, amap);
 }
 
-int gemm_umma_take_timeouts() {
+}  // namespace tz
+
+extern "C" size_t tenzo_cuda_gemm_workspace_bytes(void) { return tz::kGuWorkspaceBytes; }
+
+extern "C" int tenzo_cuda_gemm_take_timeouts(void) {
     int v = 0, zero = 0;
-    if (cudaMemcpyFromSymbol(&v, g_gu_timeouts, sizeof v) != cudaSuccess) return -1;
-    if (v) cudaMemcpyToSymbol(g_gu_timeouts, &zero, sizeof zero);
+    if (cudaMemcpyFromSymbol(&v, tz::g_gu_timeouts, sizeof v) != cudaSuccess) return -1;
+    if (v) cudaMemcpyToSymbol(tz::g_gu_timeouts, &zero, sizeof zero);
     return v;
 }
-
-}  // namespace tz

@@ -1,5 +1,6 @@
 // Device helpers of the hybrid-decoder kernels.
 #pragma once
+#include "../../include/tenzo.h"
 #include "common.cuh"
 #include "hybrid_ops.h"
 

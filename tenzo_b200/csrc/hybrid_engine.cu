@@ -68,7 +68,7 @@ void HybridEngine::init(const Json& c, const OpenOptions& o) {
         m.ring_k = dalloc(B * m.ring_k_stride * es);
         m.ring_v = dalloc(B * m.ring_v_stride * es);
     }
-    gemm_ws = dalloc(gemm_workspace_bytes());
+    gemm_ws = dalloc(tenzo_cuda_gemm_workspace_bytes());
     argmax_ws = dalloc(argmax_scratch_bytes(batch));
     alloc_rows(dec, batch);
     b_x = dec.x[0];
@@ -173,7 +173,7 @@ void HybridEngine::load(const Json& c, const std::string& dir) {
             ScanMixer& s = y.scan;
             read_scan(s, mix, false);
             s.k_scale = (float)std::pow((double)s.dim, -0.5);
-            s.decay_kind = DECAY_CONST;
+            s.decay_kind = TENZO_DECAY_CONST;
             std::vector<float> d;
             for (const Json& v : mix.at("decay").array()) d.push_back((float)v.number());
             if ((int)d.size() != s.heads) throw std::invalid_argument("'decay' needs one entry per head");
@@ -184,7 +184,7 @@ void HybridEngine::load(const Json& c, const std::string& dir) {
         } else if (type == "wkv") {
             ScanMixer& s = y.scan;
             read_scan(s, mix, true);
-            s.decay_kind = DECAY_EXP_EXP;
+            s.decay_kind = TENZO_DECAY_EXP_EXP;
             low_rank(mp + "w1", mp + "w2", mp + "w0");
             s.bonus = upload_floats(st.floats(mp + "u", {s.heads, s.dim}));
             s.norm = upload_floats(st.floats(mp + "norm", {s.heads * s.vdim}));
@@ -215,7 +215,7 @@ void HybridEngine::load(const Json& c, const std::string& dir) {
             ScanMixer& s = y.scan;
             read_scan(s, mix.at("right"), false);
             s.q_scale = (float)std::pow((double)s.dim, -0.5);
-            s.decay_kind = DECAY_SIGMOID_ROOT;
+            s.decay_kind = TENZO_DECAY_SIGMOID_ROOT;
             s.tau = (float)mix.at("right").at("tau").number();
             low_rank(rp + "a1", rp + "a2", rp + "a2.b");
             s.norm = upload_floats(st.floats(rp + "norm", {s.vdim}));
@@ -355,10 +355,10 @@ void HybridEngine::run_gemm(Pass& p, const void* a, const DenseWeight& w, void* 
         g.a_seg_stride = (size_t)p.M * w.ld_k;
     }
     g.epilogue = epilogue;
-    if (epilogue == GEMM_XIELU) { g.act_pos = y->act_pos; g.act_neg = y->act_neg; }
+    if (epilogue == TENZO_GEMM_XIELU) { g.act_pos = y->act_pos; g.act_neg = y->act_neg; }
     g.c = c; g.ld_c = ld_c;
     g.f32 = f32; g.use_pdl = p.decode && use_pdl;
-    g.workspace = gemm_ws; g.workspace_bytes = gemm_workspace_bytes();
+    g.workspace = gemm_ws; g.workspace_bytes = tenzo_cuda_gemm_workspace_bytes();
     TZ_KERNEL(launch_gemm(g, stream));
     launches += p.M > 8 && p.M < kGemmUmmaMinRows && !f32 ? 2 : 1;
 }
@@ -374,7 +374,7 @@ void HybridEngine::run_layer(Pass& p, int l) {
         ra.prev_out = p.decode ? carried : tail_stage + y.prev;
     }
     run_rows(p, ra);
-    run_gemm(p, r.in, y.in, r.proj, max_proj, GEMM_STORE, y.n_mix ? &y : nullptr);
+    run_gemm(p, r.in, y.in, r.proj, max_proj, TENZO_GEMM_STORE, y.n_mix ? &y : nullptr);
 
     if (y.has_window) {
         const WindowMixer& m = y.win;
@@ -416,18 +416,18 @@ void HybridEngine::run_layer(Pass& p, int l) {
         TZ_KERNEL(launch_scan(a, stream, &launches));
     }
     if (y.has_window && y.has_scan) {
-        run_gemm(p, r.mix_a, y.win.o, r.ya, h, GEMM_STORE, nullptr);
-        run_gemm(p, r.mix_b, y.scan.o, r.yb, h, GEMM_STORE, nullptr);
+        run_gemm(p, r.mix_a, y.win.o, r.ya, h, TENZO_GEMM_STORE, nullptr);
+        run_gemm(p, r.mix_b, y.scan.o, r.yb, h, TENZO_GEMM_STORE, nullptr);
         p.add.y0 = r.ya; p.add.y1 = r.yb; p.add.w0 = y.left_out; p.add.w1 = y.right_out;
     } else {
-        run_gemm(p, r.mix_a, y.has_window ? y.win.o : y.scan.o, r.ya, h, GEMM_STORE, nullptr);
+        run_gemm(p, r.mix_a, y.has_window ? y.win.o : y.scan.o, r.ya, h, TENZO_GEMM_STORE, nullptr);
         p.add.y0 = r.ya;
     }
     if (y.has_mlp) {
         RowsArgs rb = row_args(p, y.norm2, y.canon2, y.tail2);
         run_rows(p, rb);
-        run_gemm(p, r.in, y.up, r.act, y.down.ld_k, GEMM_XIELU, &y);
-        run_gemm(p, r.act, y.down, r.ya, h, GEMM_STORE, nullptr);
+        run_gemm(p, r.in, y.up, r.act, y.down.ld_k, TENZO_GEMM_XIELU, &y);
+        run_gemm(p, r.act, y.down, r.ya, h, TENZO_GEMM_STORE, nullptr);
         p.add.y0 = r.ya;
     }
 }
@@ -446,7 +446,7 @@ void HybridEngine::enqueue_step(bool with_logits, bool feed_back, int) {
     RowsArgs ra = row_args(p, final_gain, nullptr, 0);
     run_rows(p, ra);
     if (with_logits) {
-        run_gemm(p, dec.in, head, b_logits, V, GEMM_STORE, nullptr);
+        run_gemm(p, dec.in, head, b_logits, V, TENZO_GEMM_STORE, nullptr);
         TZ_KERNEL(launch_argmax(b_logits, V, batch, d_next, argmax_ws, stream));
         launches += 2;
     }
@@ -484,9 +484,9 @@ void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
             }
             if (y.has_scan) {
                 const ScanMixer& s = y.scan;
-                if (s.decay_kind != DECAY_CONST) w = std::max(w, m * s.heads * s.dim);
+                if (s.decay_kind != TENZO_DECAY_CONST) w = std::max(w, m * s.heads * s.dim);
                 o = std::max(o, m * s.heads * s.vdim);
-                part = std::max(part, scan_part_floats(cap, s.heads, s.dim, s.vdim));
+                part = std::max(part, tenzo_cuda_linear_scan_part_floats(cap, s.heads, s.dim, s.vdim));
             }
         }
         chunk_tokens = (int*)get(m * 4);
@@ -511,7 +511,7 @@ void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
     TZ_CUDA(cudaMemcpyAsync(tails + (size_t)seq * tail_floats, tail_stage, tail_floats * 4, cudaMemcpyDeviceToDevice, stream));
     TZ_CUDA(cudaMemcpyAsync(dec.x[0] + (size_t)seq * h, chunk.x[0] + (size_t)(M - 1) * h, (size_t)h * 4, cudaMemcpyDeviceToDevice, stream));
     TZ_CUDA(cudaStreamSynchronize(stream));
-    if (gemm_umma_take_timeouts() > 0) throw std::runtime_error("a matrix product gave up waiting for a tile copy; results are invalid");
+    if (tenzo_cuda_gemm_take_timeouts() > 0) throw std::runtime_error("a matrix product gave up waiting for a tile copy; results are invalid");
     seq_len[seq] += M;
 }
 
@@ -532,7 +532,7 @@ void HybridEngine::rows_logits(const int* want, int n_want, float* host) {
             i = j;
         }
         Pass p = {&chunk, n, 0, 0, 0, nullptr, nullptr};
-        run_gemm(p, logit_in, head, want_logits, V, GEMM_STORE, nullptr);
+        run_gemm(p, logit_in, head, want_logits, V, TENZO_GEMM_STORE, nullptr);
         TZ_CUDA(cudaMemcpyAsync(host + (size_t)a * V, want_logits, (size_t)n * V * 4, cudaMemcpyDeviceToHost, stream));
     }
     TZ_CUDA(cudaStreamSynchronize(stream));
@@ -549,7 +549,7 @@ const float* HybridEngine::buffer(int which, int seq, size_t* n) {
 void HybridEngine::check_device_status(bool force) {
     // only launches of 16 and more rows have bounded waits; single-sequence decode is polled now and then
     if (!force && batch == 1 && (++status_poll & 31) != 0) return;
-    if (gemm_umma_take_timeouts() > 0) throw std::runtime_error("a matrix product gave up waiting for a tile copy; results are invalid");
+    if (tenzo_cuda_gemm_take_timeouts() > 0) throw std::runtime_error("a matrix product gave up waiting for a tile copy; results are invalid");
 }
 
 static EngineCore* open_sozopel(const Json& config, const OpenOptions& o) { return new HybridEngine(config, o); }

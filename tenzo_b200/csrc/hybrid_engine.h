@@ -33,7 +33,7 @@ struct WindowMixer {
 };
 
 struct ScanMixer {
-    int heads = 0, dim = 0, vdim = 0, decay_kind = DECAY_CONST, rank = 0, norm_per_head = 0;
+    int heads = 0, dim = 0, vdim = 0, decay_kind = TENZO_DECAY_CONST, rank = 0, norm_per_head = 0;
     float q_scale = 1, k_scale = 1, tau = 1;
     int off_q = 0, off_k = 0, off_v = 0, off_g = 0, off_low = 0;
     float *decay = nullptr, *bias = nullptr, *bonus = nullptr, *norm = nullptr;

@@ -15,11 +15,11 @@ constexpr int kScanThreads = 256, kScanBlock = 64;
 
 // decay of channel ch (head * dim + d) for one row of low-rank values (fp32 in `low`, already through tanh if asked for)
 __device__ __forceinline__ float scan_decay(const ScanArgs& a, int ch, const float* low) {
-    if (a.decay_kind == DECAY_CONST) return a.decay[ch / a.dim];
+    if (a.decay_kind == TENZO_DECAY_CONST) return a.decay[ch / a.dim];
     float z = a.bias[ch];
-    const bf16* u = a.up + (size_t)ch * a.rank;
+    const bf16* u = static_cast<const bf16*>(a.up) + (size_t)ch * a.rank;
     for (int r = 0; r < a.rank; ++r) z = fmaf(to_f(u[r]), low[r], z);
-    return a.decay_kind == DECAY_SIGMOID_ROOT ? expf(-softplus_neg(z) / a.tau) : expf(-expf(z));
+    return a.decay_kind == TENZO_DECAY_SIGMOID_ROOT ? expf(-softplus_neg(z) / a.tau) : expf(-expf(z));
 }
 
 // ---- decode --------------------------------------------------------------------------------------------------------------
@@ -54,7 +54,7 @@ __global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(const ScanArg
     const size_t row = (size_t)seq * a.ld;
     for (int i = tid; i < a.rank; i += kScanThreads) {
         const float l = a.low[row + i];
-        s_low[i] = a.decay_kind == DECAY_EXP_EXP ? tanhf(l) : l;
+        s_low[i] = a.decay_kind == TENZO_DECAY_EXP_EXP ? tanhf(l) : l;
     }
     for (int i = tid; i < a.dim; i += kScanThreads) {
         s_q[i] = a.q[row + head * a.dim + i] * a.q_scale;
@@ -112,7 +112,7 @@ __global__ void __launch_bounds__(256) scan_decay_rows_kernel(const ScanArgs a) 
     const size_t t = blockIdx.x;
     for (int i = threadIdx.x; i < a.rank; i += 256) {
         const float l = a.low[t * a.ld + i];
-        s_low[i] = a.decay_kind == DECAY_EXP_EXP ? tanhf(l) : l;
+        s_low[i] = a.decay_kind == TENZO_DECAY_EXP_EXP ? tanhf(l) : l;
     }
     __syncthreads();
     const int n = a.heads * a.dim;
@@ -144,7 +144,7 @@ __global__ void __launch_bounds__(64) scan_block_kernel(const ScanArgs a, int n_
         if (!OUT) P[OUT ? 0 : j] = 1.0f;
         if (OUT) U[OUT ? j : 0] = a.bonus && d < a.dim ? a.bonus[head * a.dim + d] : 0.0f;
     }
-    const float w_const = a.decay_kind == DECAY_CONST ? a.decay[head] : 0.0f;
+    const float w_const = a.decay_kind == TENZO_DECAY_CONST ? a.decay[head] : 0.0f;
     for (int tb = t_begin; tb < t_end; tb += kScanTile) {
         const int nt = min(kScanTile, t_end - tb);
         __syncthreads();
@@ -154,7 +154,7 @@ __global__ void __launch_bounds__(64) scan_block_kernel(const ScanArgs a, int n_
             const bool in = d < a.dim;
             s_k[r][d] = in ? a.k[row] * a.k_scale : 0.0f;
             if (OUT) s_q[OUT ? r : 0][d] = in ? a.q[row] * a.q_scale : 0.0f;
-            s_w[r][d] = in ? (a.decay_kind == DECAY_CONST ? w_const : a.w_rows[(size_t)(tb + r) * a.heads * a.dim + head * a.dim + d]) : 0.0f;
+            s_w[r][d] = in ? (a.decay_kind == TENZO_DECAY_CONST ? w_const : a.w_rows[(size_t)(tb + r) * a.heads * a.dim + head * a.dim + d]) : 0.0f;
         }
         for (int i = tid; i < nt * kScanCols; i += 64) {
             const int r = i / kScanCols, c = i - r * kScanCols, vc = blockIdx.x * kScanCols + c;
@@ -256,15 +256,10 @@ __global__ void __launch_bounds__(256) scan_gate_kernel(const ScanArgs a) {
     }
 }
 
-size_t scan_part_floats(int M, int heads, int dim, int vdim) {
-    const size_t blocks = (M + kScanBlock - 1) / kScanBlock;
-    return blocks * heads * dim * (size_t)(round_up(vdim, 4) + 1);
-}
-
 int launch_scan(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
     if (a.M <= 0) return 0;
     if (a.dim < 1 || a.dim > kMaxHeadDim || a.vdim < 1 || a.vdim > kMaxHeadDim || a.heads < 1) return -1;
-    const int rank = a.decay_kind == DECAY_CONST ? 0 : a.rank;
+    const int rank = a.decay_kind == TENZO_DECAY_CONST ? 0 : a.rank;
     ScanArgs p = a;
     p.rank = rank;
     const int ldv = round_up(a.vdim, 4);
@@ -305,3 +300,16 @@ int launch_scan(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernel
 }
 
 }  // namespace tz
+
+extern "C" int tenzo_cuda_linear_scan(const tenzo_scan_args* args, void* stream) {
+    if (!args) return TENZO_ERROR_INVALID_ARGUMENT;
+    tz::ScanArgs a;
+    static_cast<tenzo_scan_args&>(a) = *args;
+    unsigned long long n = 0;
+    return tz::launch_scan(a, static_cast<cudaStream_t>(stream), &n);
+}
+
+extern "C" size_t tenzo_cuda_linear_scan_part_floats(int M, int heads, int dim, int vdim) {
+    const size_t blocks = (M + tz::kScanBlock - 1) / tz::kScanBlock;
+    return blocks * heads * dim * (size_t)(tz::round_up(vdim, 4) + 1);
+}

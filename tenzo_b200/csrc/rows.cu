@@ -17,7 +17,7 @@ struct RowsLaunch {
 };
 
 __device__ __forceinline__ float rows_source(const RowsArgs& a, int t, int c, float inv0, float inv1, int tok, int p) {
-    if (a.tokens) return to_f(a.embed[(size_t)tok * a.width + c]) + to_f(a.pos_table[(size_t)p * a.width + c]);
+    if (a.tokens) return to_f(static_cast<const bf16*>(a.embed)[(size_t)tok * a.width + c]) + to_f(static_cast<const bf16*>(a.pos_table)[(size_t)p * a.width + c]);
     float x = a.x_in[(size_t)t * a.width + c];
     if (a.y1) {
         const float l = a.y0[(size_t)t * a.ld_y + c] * inv0 * a.w0[c], r = a.y1[(size_t)t * a.ld_y + c] * inv1 * a.w1[c];
@@ -34,7 +34,8 @@ __device__ __forceinline__ float group_sum(float v, float* scratch) {
     return DECODE ? block_sum(v, scratch) : warp_sum(v);
 }
 
-template <typename T, bool DECODE>
+// NT: taps rounded up to 4 or 16.
+template <typename T, bool DECODE, int NT>
 __global__ void __launch_bounds__(kRowThreads) rows_kernel(const RowsLaunch L) {
     extern __shared__ float s_h[];                      // [halo + TR][width]
     __shared__ float s_red[kRowThreads / 32];
@@ -101,30 +102,38 @@ __global__ void __launch_bounds__(kRowThreads) rows_kernel(const RowsLaunch L) {
     // convolution, mixes
     T* out = reinterpret_cast<T*>(a.out);
     const size_t mix_stride = (size_t)a.M * a.ld_out;
+    const bool lead = a.mu && !DECODE && t0 > 0;                 // the shift starts from the row before, recomputed
     for (int c = threadIdx.x; c < width; c += kRowThreads) {
-        float w[kMaxTaps];
+        // w[NT-1] belongs to the current row; u holds the last NT inputs, those before the convolution's reach as zero
+        float w[NT], u[NT];
+        const int start = lead ? -1 : 0;
 #pragma unroll
-        for (int j = 0; j < kMaxTaps; ++j) w[j] = j < nt + 1 && a.conv_w ? a.conv_w[(size_t)j * width + c] : 0.0f;
-        auto conv_at = [&](int r) {                              // row r of the shared tile
-            const float h = s_h[(size_t)r * width + c];
-            if (!a.conv_w) return h;
-            float y = 0.0f;
+        for (int j = 0; j < NT; ++j) {
+            const bool in = j >= NT - taps;
+            w[j] = in && a.conv_w ? a.conv_w[(size_t)(j - NT + taps) * width + c] : 0.0f;
+            u[j] = j > NT - taps && a.conv_w ? s_h[(size_t)max(0, halo + start - NT + j) * width + c] : 0.0f;
+        }
+        float prev = a.mu && !lead ? prev_in[c] : 0.0f;
+        for (int i = start; i < n_rows; ++i) {
 #pragma unroll
-            for (int j = 0; j < kMaxTaps; ++j)
-                if (j < taps) y = fmaf(w[j], s_h[(size_t)(r - nt + j) * width + c], y);
-            return h + y;
-        };
-        float prev = 0.0f;
-        if (a.mu) prev = DECODE || t0 == 0 ? prev_in[c] : conv_at(halo - 1);
-        for (int i = 0; i < n_rows; ++i) {
-            const float y = conv_at(halo + i);
-            const size_t row = (size_t)(t0 + i) * a.ld_out + c;
-            if (a.mu) {
-                for (int s = 0; s < a.n_mix; ++s) out[s * mix_stride + row] = from_f<T>(fmaf(prev - y, a.mu[(size_t)s * width + c], y));
-                prev = y;
-            } else {
-                out[row] = from_f<T>(y);
+            for (int j = 0; j + 1 < NT; ++j) u[j] = u[j + 1];
+            u[NT - 1] = s_h[(size_t)(halo + i) * width + c];
+            float y = u[NT - 1];
+            if (a.conv_w) {
+                float z = 0.0f;
+#pragma unroll
+                for (int j = 0; j < NT; ++j) z = fmaf(w[j], u[j], z);
+                y += z;
             }
+            if (i >= 0) {
+                const size_t row = (size_t)(t0 + i) * a.ld_out + c;
+                if (a.mu) {
+                    for (int s = 0; s < a.n_mix; ++s) out[s * mix_stride + row] = from_f<T>(fmaf(prev - y, a.mu[(size_t)s * width + c], y));
+                } else {
+                    out[row] = from_f<T>(y);
+                }
+            }
+            prev = y;
         }
         if (t0 + n_rows == a.M || DECODE) {                      // the state after the last row
             if (a.mu) prev_out[c] = prev;
@@ -152,8 +161,19 @@ int launch_rows(const RowsArgs& a, cudaStream_t st) {
         if (int rc = allow_smem(kernel, smem)) return rc;
         return launch_kernel(kernel, grid, dim3(kRowThreads), smem, st, a.use_pdl, 1, L);
     };
-    if (a.f32) return a.decode ? go(rows_kernel<float, true>) : go(rows_kernel<float, false>);
-    return a.decode ? go(rows_kernel<bf16, true>) : go(rows_kernel<bf16, false>);
+    if (a.taps <= 4) {
+        if (a.f32) return a.decode ? go(rows_kernel<float, true, 4>) : go(rows_kernel<float, false, 4>);
+        return a.decode ? go(rows_kernel<bf16, true, 4>) : go(rows_kernel<bf16, false, 4>);
+    }
+    if (a.f32) return a.decode ? go(rows_kernel<float, true, kMaxTaps>) : go(rows_kernel<float, false, kMaxTaps>);
+    return a.decode ? go(rows_kernel<bf16, true, kMaxTaps>) : go(rows_kernel<bf16, false, kMaxTaps>);
 }
 
 }  // namespace tz
+
+extern "C" int tenzo_cuda_rows(const tenzo_rows_args* args, void* stream) {
+    if (!args) return TENZO_ERROR_INVALID_ARGUMENT;
+    tz::RowsArgs a;
+    static_cast<tenzo_rows_args&>(a) = *args;
+    return tz::launch_rows(a, static_cast<cudaStream_t>(stream));
+}

@@ -195,7 +195,7 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
             for (int i = tid; i < GQ * ldv; i += kWaThreads) {
                 const int g = i / ldv, d = i - g * ldv;
                 if (q0 + g >= group || d >= a.vdim) continue;
-                float mx = 0.0f;                              // the sink's score
+                float mx = a.sink > 0.0f ? 0.0f : -1e30f;     // the sink is a score of 0
                 for (int r = 0; r < n_rank; ++r) mx = fmaxf(mx, cluster.map_shared_rank(s_ml, r)[g]);
                 float den = a.sink * expf(-mx), num = 0.0f;
                 for (int r = 0; r < n_rank; ++r) {
@@ -319,7 +319,7 @@ __global__ void __launch_bounds__(kWaThreads) window_chunk_kernel(const WaChunkL
     for (int d = lane; d < ldd; d += 32)
         s_q[warp * ldd + d] = live ? to_f(reinterpret_cast<const T*>(a.lin_q)[((size_t)t * a.heads + h) * ldd + d]) * a.scale : 0.0f;
     const float slope = head_slope(a, h);
-    float m = 0.0f, l = a.sink, acc[kWaMaxCols];             // the maximum starts at the sink's
+    float m = a.sink > 0.0f ? 0.0f : -1e30f, l = a.sink, acc[kWaMaxCols];   // the sink is a score of 0
 #pragma unroll
     for (int c = 0; c < kWaMaxCols; ++c) acc[c] = 0.0f;
     const int i_last = L.hist + min(a.M, (int)(blockIdx.x + 1) * kWaQ) - 1;
@@ -403,3 +403,11 @@ int launch_window_attention(const WindowAttnArgs& a, cudaStream_t st, unsigned l
 }
 
 }  // namespace tz
+
+extern "C" int tenzo_cuda_window_attention(const tenzo_window_attention_args* args, void* stream) {
+    if (!args) return TENZO_ERROR_INVALID_ARGUMENT;
+    tz::WindowAttnArgs a;
+    static_cast<tenzo_window_attention_args&>(a) = *args;
+    unsigned long long n = 0;
+    return tz::launch_window_attention(a, static_cast<cudaStream_t>(stream), &n);
+}

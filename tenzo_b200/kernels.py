@@ -164,3 +164,36 @@ def tl1_pack_rows2bit(raw, N, K):
     packed = torch.empty(N * K // 4, dtype=torch.uint8, device=raw.device)
     _ok(lib.tenzo_cuda_tl1_pack_rows2bit(_ptr(raw), N, K, _ptr(packed), _stream()), "tenzo_cuda_tl1_pack_rows2bit")
     return packed
+
+
+# ---- pieces of the hybrid decoders ------------------------------------------------------------------------------------
+def _struct_call(name: str, struct, defaults: dict, fields: dict):
+    """One flat kernel call: keyword arguments are the struct's fields, tensors are passed by address."""
+    args = struct()
+    for k, v in {**defaults, **fields}.items():
+        setattr(args, k, v.data_ptr() if isinstance(v, torch.Tensor) else (C.c_int * 8)(*v) if isinstance(v, (list, tuple)) else v)
+    _ok(getattr(load_library(), "tenzo_cuda_" + name)(C.byref(args), _stream()), "tenzo_cuda_" + name)
+
+
+def rows(**fields):
+    _struct_call("rows", abi.RowsArgs, {"gain": 1.0, "taps": 1}, fields)
+
+
+def gemm(**fields):
+    _struct_call("gemm", abi.GemmArgs, {"n_seg": 1}, fields)
+
+
+def window_attention(**fields):
+    _struct_call("window_attention", abi.WindowAttentionArgs, {"taps": 1, "scale": 1.0, "slope_base": 8.0, "sink": 1.0}, fields)
+
+
+def linear_scan(**fields):
+    _struct_call("linear_scan", abi.ScanArgs, {"q_scale": 1.0, "k_scale": 1.0, "tau": 1.0}, fields)
+
+
+def gemm_workspace() -> torch.Tensor:
+    return torch.zeros(load_library().tenzo_cuda_gemm_workspace_bytes(), dtype=torch.uint8, device="cuda")
+
+
+def linear_scan_part(M: int, heads: int, dim: int, vdim: int) -> torch.Tensor:
+    return torch.empty(load_library().tenzo_cuda_linear_scan_part_floats(M, heads, dim, vdim), dtype=torch.float32, device="cuda")

@@ -126,3 +126,125 @@ class SyntheticModel:
 
 def prompt_tokens(seed: int, n: int, vocab: int) -> np.ndarray:
     return np.random.default_rng([seed, 99]).integers(0, vocab, n, dtype=np.int32)
+
+
+# ---- Sozopel folders ----------------------------------------------------------------------------------------------------
+def bf16_bits(x: np.ndarray) -> np.ndarray:
+    """fp32 -> bf16 bit patterns, round to nearest even."""
+    b = np.ascontiguousarray(x, np.float32).view(np.uint32)
+    return ((b + 0x7FFF + ((b >> 16) & 1)) >> 16).astype(np.uint16)
+
+
+def write_safetensors(path, tensors: dict):
+    """name -> fp32 array, stored as bf16."""
+    import json
+    import struct
+    head, off = {}, 0
+    for name, a in tensors.items():
+        head[name] = {"dtype": "BF16", "shape": list(a.shape), "data_offsets": [off, off + 2 * a.size]}
+        off += 2 * a.size
+    text = json.dumps(head).encode()
+    text += b" " * (-len(text) % 8)
+    with open(path, "wb") as f:
+        f.write(struct.pack("<Q", len(text)) + text)
+        for a in tensors.values():
+            f.write(bf16_bits(a).tobytes())
+
+
+def sozopel_tensors(cfg: dict, rank: int) -> dict:
+    """name -> (shape, spread, centre) of every tensor of a Sozopel configuration; `rank` is the size of the low-rank gates."""
+    W, V = cfg["width"], cfg["vocab"]
+    t = {"embed": ((V, W), 1.0, 0.0), "pos": ((cfg["max_positions"], W), 0.3, 0.0), "final.norm": ((), 0.05, 1.0), "head": ((V, W), W ** -0.5, 0.0)}
+
+    def lin(name, rows, cols, gain=1.0):
+        t[name] = ((rows, cols), gain * cols ** -0.5, 0.0)
+
+    for i, layer in enumerate(cfg["layers"]):
+        p, mix = f"l{i}.", layer["mixer"]
+        m = p + "mix."
+        t[p + "norm1"] = ((), 0.05, 1.0)
+        t[p + "canon1"] = ((W, cfg["canon"]["taps"]), 0.3, 0.0)
+        if layer["type"] == "parallel":
+            lf, rt = mix["left"], mix["right"]
+            for s, n in (("q", lf["heads"] * lf["dim"]), ("k", lf["kv_heads"] * lf["dim"]), ("v", lf["kv_heads"] * lf["vdim"])):
+                lin(m + "left." + s, n, W)
+                t[m + f"left.{s}.conv"] = ((n, lf["conv"]), 0.7, 0.2)
+            lin(m + "left.o", W, lf["heads"] * lf["vdim"])
+            n, nv = rt["heads"] * rt["dim"], rt["heads"] * rt["vdim"]
+            for s, r in (("q", n), ("k", n), ("v", nv), ("g", nv)):
+                lin(m + "right." + s, r, W)
+            lin(m + "right.o", W, nv)
+            t[m + "right.norm"] = ((rt["vdim"],), 0.2, 1.0)
+            lin(m + "right.a1", rank, W)
+            lin(m + "right.a2", n, rank)
+            t[m + "right.a2.b"] = ((n,), 1.0, 0.0)
+            t[m + "left.out"] = ((W,), 0.2, 1.0)
+            t[m + "right.out"] = ((W,), 0.2, 1.0)
+        elif layer["type"] == "retention":
+            n, nv = mix["heads"] * mix["dim"], mix["heads"] * mix["vdim"]
+            for s, r in (("q", n), ("k", n), ("v", nv), ("g", nv)):
+                lin(m + s, r, W)
+            lin(m + "o", W, nv)
+        elif layer["type"] == "wkv":
+            n = mix["heads"] * mix["dim"]
+            for s in "rkvgw":
+                t[m + "mu." + s] = ((W,), 0.3, 0.5)
+            for s in "rkvg":
+                lin(m + s, n, W)
+            lin(m + "w1", rank, W)
+            lin(m + "w2", n, rank)
+            t[m + "w0"] = ((n,), 1.0, -2.5)
+            t[m + "u"] = ((mix["heads"], mix["dim"]), 0.5, 0.5)
+            t[m + "norm"] = ((n,), 0.2, 1.0)
+            lin(m + "o", W, n)
+        if layer["mlp"] is not None:
+            t[p + "norm2"] = ((), 0.05, 1.0)
+            t[p + "canon2"] = ((W, cfg["canon"]["taps"]), 0.3, 0.0)
+            lin(p + "mlp.up", layer["mlp"]["ff"], W)
+            lin(p + "mlp.down", W, layer["mlp"]["ff"])
+            t[p + "mlp.act"] = ((2,), 0.5, 0.3)
+    return t
+
+
+def write_sozopel(folder, cfg: dict, *, rank: int = 8, seed: int = 0, change=None) -> dict:
+    """A Sozopel model folder with random weights; `change(tensors)` may edit them first. Returns the fp32 tensors, already
+    rounded to what the file holds."""
+    import json
+    from pathlib import Path
+    rng = np.random.default_rng(seed)
+    out = {name: (centre + spread * rng.standard_normal(shape)).astype(np.float32) for name, (shape, spread, centre) in sozopel_tensors(cfg, rank).items()}
+    if change is not None:
+        change(out)
+    folder = Path(folder)
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(dict(cfg, architecture="Sozopel")))
+    write_safetensors(folder / "model.safetensors", {n: np.asarray(a) for n, a in out.items()})
+    return {n: (bf16_bits(a).astype(np.uint32) << 16).view(np.float32).reshape(np.shape(a)) for n, a in out.items()}
+
+
+def write_sozopel_pooled(folder, cfg: dict, *, rank: int, seed: int = 0):
+    """write_sozopel for large models: values come from one pool of random numbers, tensors go to the file one by one."""
+    import json
+    import struct
+    from pathlib import Path
+    rng = np.random.default_rng(seed)
+    pool = rng.standard_normal(1 << 22, dtype=np.float32)
+    spec = sozopel_tensors(cfg, rank)
+    head, off = {}, 0
+    for name, (shape, _, _) in spec.items():
+        n = int(np.prod(shape))
+        head[name] = {"dtype": "BF16", "shape": list(shape), "data_offsets": [off, off + 2 * n]}
+        off += 2 * n
+    text = json.dumps(head).encode()
+    text += b" " * (-len(text) % 8)
+    folder = Path(folder)
+    (folder / "config.json").write_text(json.dumps(dict(cfg, architecture="Sozopel")))
+    with open(folder / "model.safetensors", "wb") as f:
+        f.write(struct.pack("<Q", len(text)) + text)
+        for shape, spread, centre in spec.values():
+            bits, n = bf16_bits(centre + spread * pool), int(np.prod(shape))
+            while n > 0:
+                a = int(rng.integers(0, pool.size - 1))
+                part = bits[a:a + n]
+                f.write(part.tobytes())
+                n -= part.size
