@@ -245,7 +245,7 @@ typedef struct {
     const float *x_in;                /* otherwise x = x_in (+ y0) (+ 0.5 (y0 / rms(y0) * w0 + y1 / rms(y1) * w1) when y1) */
     const float *y0, *y1, *w0, *w1;
     int ld_y;
-    float* x_out;                     /* [M][width], not x_in */
+    float* x_out;                     /* [M][width] */
     int width, M;
     float eps, gain;
     const float* conv_w;              /* [taps][width]; NULL: no convolution */
@@ -260,6 +260,7 @@ typedef struct {
     int decode;
     void* out;                        /* storage type [max(n_mix,1)][M][ld_out] */
     int ld_out;
+    float* row_inv;                   /* [M] scratch; decode needs it for width > 4096 or taps > 4 only */
     int f32, use_pdl;
 } tenzo_rows_args;
 TENZO_API int tenzo_cuda_rows(const tenzo_rows_args* args, void* stream);
@@ -322,7 +323,7 @@ typedef struct {
     int decay_kind;
     const float* decay;               /* CONST: w = decay[head] */
     const float* low;                 /* others: z = up f(low) + bias over `rank` values per row (row stride ld); */
-    const void* up;                   /* bf16 [heads*dim][rank] */
+    const void* up;                   /* bf16 [heads*dim][rank rounded up to 8], padding zero */
     const float* bias;                /* SIGMOID_ROOT: f(x) = x, w = sigmoid(z)^(1/tau); EXP_EXP: f = tanh, w = exp(-exp(z)) */
     int rank;
     float tau;

@@ -78,7 +78,7 @@ def _fields(spec: str):
 
 class RowsArgs(C.Structure):
     _fields_ = _fields("tokens:p pos:p embed:p pos_table:p vocab:i n_pos:i x_in:p y0:p y1:p w0:p w1:p ld_y:i x_out:p width:i M:i eps:f gain:f "
-                       "conv_w:p taps:i tail_in:p tail_out:p mu:p n_mix:i prev_in:p prev_out:p seq_stride:z decode:i out:p ld_out:i f32:i use_pdl:i")
+                       "conv_w:p taps:i tail_in:p tail_out:p mu:p n_mix:i prev_in:p prev_out:p seq_stride:z decode:i out:p ld_out:i row_inv:p f32:i use_pdl:i")
 
 
 class GemmArgs(C.Structure):

@@ -234,9 +234,10 @@ def _kernels(width, ff, only=None):
             n_rot = 8 if M == CHUNK else 1
             xs = [rnd(M, width) for _ in range(n_rot)]
             y, xo, out = rnd(M, width), torch.empty(M, width, device="cuda"), torch.empty(M, width, dtype=bf, device="cuda")
+            inv = torch.empty(M, device="cuda")
             cw, tail = rnd(4, width), torch.zeros(M if dec else 2, 3 * width, device="cuda")
             us = _time([lambda x=x_: K.rows(x_in=x, y0=y, ld_y=width, x_out=xo, width=width, M=M, eps=1e-5, conv_w=cw, taps=4, tail_in=tail, tail_out=tail if dec else tail[1],
-                        seq_stride=3 * width, decode=dec, out=out, ld_out=width, use_pdl=dec) for x_ in xs])
+                        seq_stride=3 * width, decode=dec, row_inv=inv, out=out, ld_out=width, use_pdl=dec) for x_ in xs])
             add(f"rows (residual, norm, convolution), {M} rows", us, M * width * 14)
             us = _time([lambda x=x_: K.rmsnorm_quant(x, want_y=False) for x_ in xs])
             add(f"BitNet norm + quantiser, {M} rows", us, M * width * 5, like=f"rows (residual, norm, convolution), {M} rows")

@@ -7,7 +7,7 @@
 //   scan     decays, recurrence, per-head norm, gate                  }
 //   gemm     output projection(s)
 //   rows, gemm (+ activation), gemm    the feed-forward, when the layer has one
-// Residual sums happen at the start of the next row kernel, two residual buffers taking turns.
+// Residual sums happen at the start of the next row kernel.
 #include "hybrid_engine.h"
 
 #include <algorithm>
@@ -71,7 +71,7 @@ void HybridEngine::init(const Json& c, const OpenOptions& o) {
     gemm_ws = dalloc(tenzo_cuda_gemm_workspace_bytes());
     argmax_ws = dalloc(argmax_scratch_bytes(batch));
     alloc_rows(dec, batch);
-    b_x = dec.x[0];
+    b_x = dec.x;
     TZ_CUDA(cudaStreamSynchronize(stream));
 }
 
@@ -166,7 +166,10 @@ void HybridEngine::load(const Json& c, const std::string& dir) {
             ScanMixer& s = y.scan;
             s.rank = (int)st.bf16(down, {-1, W}).shape[0];
             const int n = s.heads * s.dim;
-            s.up = (bf16*)upload(st.bf16(up_name, {n, s.rank}).data, (size_t)n * s.rank * 2);
+            s.up = (bf16*)dalloc((size_t)n * round_up(s.rank, 8) * 2);
+            TZ_CUDA(cudaMemcpy2DAsync(s.up, (size_t)round_up(s.rank, 8) * 2, st.bf16(up_name, {n, s.rank}).data, (size_t)s.rank * 2, (size_t)s.rank * 2,
+                                      (size_t)n, cudaMemcpyHostToDevice, stream));
+            TZ_CUDA(cudaStreamSynchronize(stream));
             s.bias = upload_floats(st.floats(bias, {n}));
         };
         if (type == "retention") {
@@ -282,8 +285,8 @@ void HybridEngine::alloc_rows(Rows& r, int cap) {
         TZ_CUDA(cudaMemsetAsync(p, 0, bytes ? bytes : 16, stream));      // padding columns stay finite
         return p;
     };
-    r.x[0] = (float*)get(m * h * 4);
-    r.x[1] = (float*)get(m * h * 4);
+    r.row_inv = (float*)get(m * 4);
+    r.x = (float*)get(m * h * 4);
     r.in = get(m * max_in * max_seg * es);
     r.proj = (float*)get(m * max_proj * 4);
     r.mix_a = get(m * max_mix * es);
@@ -334,15 +337,14 @@ void HybridEngine::run_rows(Pass& p, RowsArgs& a) {
         a.vocab = V; a.n_pos = n_pos;
         p.embed = false;
     } else {
-        a.x_in = p.rows->x[p.cur];
+        a.x_in = p.rows->x;
         a.y0 = p.add.y0; a.y1 = p.add.y1; a.w0 = p.add.w0; a.w1 = p.add.w1;
         a.ld_y = h;
     }
     p.add = Pending();
-    p.cur ^= 1;
-    a.x_out = p.rows->x[p.cur];
-    TZ_KERNEL(launch_rows(a, stream));
-    launches += 1;
+    a.x_out = p.rows->x;
+    a.row_inv = p.rows->row_inv;
+    TZ_KERNEL(launch_rows(a, stream, &launches));
 }
 
 void HybridEngine::run_gemm(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c, int epilogue, const HybridLayer* y) {
@@ -432,16 +434,8 @@ void HybridEngine::run_layer(Pass& p, int l) {
     }
 }
 
-// Row kernels of a whole pass; the first one must leave the last one's residual in buffer 0.
-static int first_buffer(const std::vector<HybridLayer>& layers) {
-    int n = 1;
-    for (const HybridLayer& y : layers) n += 1 + (y.has_mlp ? 1 : 0);
-    return n & 1;
-}
-
 void HybridEngine::enqueue_step(bool with_logits, bool feed_back, int) {
     Pass p = {&dec, batch, 1, 0, 0, d_tokens, d_pos};
-    p.cur = first_buffer(layers);
     for (int l = 0; l < L; ++l) run_layer(p, l);
     RowsArgs ra = row_args(p, final_gain, nullptr, 0);
     run_rows(p, ra);
@@ -459,7 +453,6 @@ void HybridEngine::enqueue_layer(int l, int) {
     run_layer(p, l);
     RowsArgs ra = row_args(p, 1.0f, nullptr, 0);
     run_rows(p, ra);
-    if (p.cur != 0) TZ_CUDA(cudaMemcpyAsync(dec.x[0], dec.x[1], (size_t)batch * h * 4, cudaMemcpyDeviceToDevice, stream));
 }
 
 void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
@@ -467,6 +460,7 @@ void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
         int cap = 64;
         while (cap < M) cap *= 2;
         alloc_rows(chunk, cap);
+        chunk.cap = 0;                                 // until every buffer below exists too
         const size_t m = cap, es = f32 ? 4 : 2;
         auto get = [&](size_t bytes) -> void* {
             void* p = nullptr;
@@ -497,6 +491,7 @@ void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
         w_rows = (float*)get(w * 4);
         o_rows = (float*)get(o * 4);
         scan_part = (float*)get(part * 4);
+        chunk.cap = cap;
     }
     const int pos0 = seq_len[seq];
     std::vector<int> hp(M);
@@ -504,12 +499,11 @@ void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
     TZ_CUDA(cudaMemcpyAsync(chunk_tokens, tokens, (size_t)M * 4, cudaMemcpyHostToDevice, stream));
     TZ_CUDA(cudaMemcpyAsync(chunk_pos, hp.data(), (size_t)M * 4, cudaMemcpyHostToDevice, stream));
     Pass p = {&chunk, M, 0, seq, pos0, chunk_tokens, chunk_pos};
-    p.cur = first_buffer(layers);
     for (int l = 0; l < L; ++l) run_layer(p, l);
     RowsArgs ra = row_args(p, final_gain, nullptr, 0);
     run_rows(p, ra);                                   // leaves the normalised rows for rows_logits in chunk.in
     TZ_CUDA(cudaMemcpyAsync(tails + (size_t)seq * tail_floats, tail_stage, tail_floats * 4, cudaMemcpyDeviceToDevice, stream));
-    TZ_CUDA(cudaMemcpyAsync(dec.x[0] + (size_t)seq * h, chunk.x[0] + (size_t)(M - 1) * h, (size_t)h * 4, cudaMemcpyDeviceToDevice, stream));
+    TZ_CUDA(cudaMemcpyAsync(dec.x + (size_t)seq * h, chunk.x + (size_t)(M - 1) * h, (size_t)h * 4, cudaMemcpyDeviceToDevice, stream));
     TZ_CUDA(cudaStreamSynchronize(stream));
     if (tenzo_cuda_gemm_take_timeouts() > 0) throw std::runtime_error("a matrix product gave up waiting for a tile copy; results are invalid");
     seq_len[seq] += M;
@@ -540,7 +534,7 @@ void HybridEngine::rows_logits(const int* want, int n_want, float* host) {
 
 const float* HybridEngine::buffer(int which, int seq, size_t* n) {
     switch (which) {
-        case TENZO_BUF_X: *n = h; return dec.x[0] + (size_t)seq * h;
+        case TENZO_BUF_X: *n = h; return dec.x + (size_t)seq * h;
         case TENZO_BUF_LOGITS: *n = V; return b_logits + (size_t)seq * V;
         default: throw std::invalid_argument("this model keeps no such buffer");
     }

@@ -78,9 +78,9 @@ public:
 private:
     struct Rows {                            // activations of M rows; decode and chunk each have their own set
         int cap = 0;
-        float *x[2] = {nullptr, nullptr};
+        float* x = nullptr;                  // residual
         void *in = nullptr, *mix_a = nullptr, *mix_b = nullptr, *act = nullptr;
-        float *proj = nullptr, *ya = nullptr, *yb = nullptr;
+        float *row_inv = nullptr, *proj = nullptr, *ya = nullptr, *yb = nullptr;
         std::vector<void*> owned;
     };
     struct Pending {                         // what the next row kernel adds to the residual
@@ -90,7 +90,6 @@ private:
         Rows* rows;
         int M, decode, seq, pos0;
         const int *tokens, *pos;
-        int cur = 0;                         // residual buffer in use
         bool embed = true;
         Pending add;
     };

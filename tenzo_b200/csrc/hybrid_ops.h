@@ -31,7 +31,7 @@ struct ScanArgs : tenzo_scan_args {
     ScanArgs() : tenzo_scan_args{} { q_scale = k_scale = tau = 1; }
 };
 
-int launch_rows(const RowsArgs& a, cudaStream_t st);                                                      // rows.cu
+int launch_rows(const RowsArgs& a, cudaStream_t st, unsigned long long* n_kernels);                       // rows.cu
 int launch_gemm(const GemmArgs& a, cudaStream_t st);                                                      // gemm.cu
 int launch_gemm_umma(const GemmArgs& a, cudaStream_t st);                                                 // gemm_umma.cu
 bool gemm_umma_applicable(const GemmArgs& a);

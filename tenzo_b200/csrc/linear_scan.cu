@@ -7,19 +7,17 @@
 // Chunk: rows are cut into blocks of kScanBlock. The blocks' own states from zero and their decay products are formed in
 // parallel, a short pass carries the state across blocks, and every block is then walked from its true starting
 // state. Products of decays only ever multiply states, so small decays underflow harmlessly.
+#include <type_traits>
+
 #include "hybrid_common.cuh"
 
 namespace tz {
 
 constexpr int kScanThreads = 256, kScanBlock = 64;
 
-// decay of channel ch (head * dim + d) for one row of low-rank values (fp32 in `low`, already through tanh if asked for)
-__device__ __forceinline__ float scan_decay(const ScanArgs& a, int ch, const float* low) {
-    if (a.decay_kind == TENZO_DECAY_CONST) return a.decay[ch / a.dim];
-    float z = a.bias[ch];
-    const bf16* u = static_cast<const bf16*>(a.up) + (size_t)ch * a.rank;
-    for (int r = 0; r < a.rank; ++r) z = fmaf(to_f(u[r]), low[r], z);
-    return a.decay_kind == TENZO_DECAY_SIGMOID_ROOT ? expf(-softplus_neg(z) / a.tau) : expf(-expf(z));
+// decay from the gate's value
+__device__ __forceinline__ float gate_decay(int kind, float z, float tau) {
+    return kind == TENZO_DECAY_SIGMOID_ROOT ? expf(-softplus_neg(z) / tau) : expf(-expf(z));
 }
 
 // ---- decode --------------------------------------------------------------------------------------------------------------
@@ -45,15 +43,23 @@ __global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(const ScanArg
     float* s_k = s_q + a.dim;
     float* s_w = s_k + a.dim;
     float* s_u = s_w + a.dim;                            // bonus
-    float* s_low = s_u + a.dim;                          // [rank]
-    float* s_v = s_low + a.rank;                         // [ldv]
-    float* s_o = sm + ((4 * a.dim + a.rank + ldv + 3) & ~3);    // [n_rg][ldv]
+    float* s_low = s_u + a.dim;                          // [rank, padded to 8]
+    float* s_v = s_low + ((a.rank + 7) & ~7);            // [ldv]
+    float* s_o = sm + ((4 * a.dim + ((a.rank + 7) & ~7) + ldv + 3) & ~3);   // [n_rg][ldv]
     float* s_red = s_o + n_rg * ldv;                     // [8]
+    // low-rank gate: four lanes per channel, 16-byte pieces of its row; the first two are fetched ahead as well
+    const bool gated = a.decay_kind != TENZO_DECAY_CONST;
+    const int rank8 = (a.rank + 7) & ~7, sub = tid & 3;
+    const bf16* up = static_cast<const bf16*>(a.up) + (size_t)head * a.dim * rank8;
+    uint4 gate[2] = {};
+#pragma unroll
+    for (int i = 0; i < 2; ++i)
+        if (gated && tid / 4 < a.dim && (sub + 4 * i) * 8 < rank8) gate[i] = *reinterpret_cast<const uint4*>(up + (size_t)(tid / 4) * rank8 + (sub + 4 * i) * 8);
     pdl_wait();
     pdl_launch_dependents();
     const size_t row = (size_t)seq * a.ld;
-    for (int i = tid; i < a.rank; i += kScanThreads) {
-        const float l = a.low[row + i];
+    for (int i = tid; i < rank8; i += kScanThreads) {
+        const float l = i < a.rank ? a.low[row + i] : 0.0f;
         s_low[i] = a.decay_kind == TENZO_DECAY_EXP_EXP ? tanhf(l) : l;
     }
     for (int i = tid; i < a.dim; i += kScanThreads) {
@@ -63,7 +69,25 @@ __global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(const ScanArg
     }
     for (int i = tid; i < ldv; i += kScanThreads) s_v[i] = i < a.vdim ? a.v[row + head * a.vdim + i] : 0.0f;
     __syncthreads();
-    for (int i = tid; i < a.dim; i += kScanThreads) s_w[i] = scan_decay(a, head * a.dim + i, s_low);
+    if (gated) {
+        for (int d0 = 0; d0 < a.dim; d0 += kScanThreads / 4) {          // uniform trips: the exchanges are warp-wide
+            const int d = d0 + tid / 4;
+            float z = 0.0f;
+            if (d < a.dim)
+                for (int i = 0; (sub + 4 * i) * 8 < rank8; ++i) {
+                    const int c = (sub + 4 * i) * 8;
+                    float u[8];
+                    if (d0 == 0 && i < 2) unpack8(i ? gate[1] : gate[0], u); else load8(up + (size_t)d * rank8 + c, u);
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) z = fmaf(u[j], s_low[c + j], z);
+                }
+            z += __shfl_xor_sync(0xffffffffu, z, 1);
+            z += __shfl_xor_sync(0xffffffffu, z, 2);
+            if (sub == 0 && d < a.dim) s_w[d] = gate_decay(a.decay_kind, z + a.bias[head * a.dim + d], a.tau);
+        }
+    } else {
+        for (int i = tid; i < a.dim; i += kScanThreads) s_w[i] = a.decay[head];
+    }
     __syncthreads();
     float o[4] = {0.0f, 0.0f, 0.0f, 0.0f};
     if (live) {
@@ -106,111 +130,163 @@ __global__ void __launch_bounds__(kScanThreads) scan_decode_kernel(const ScanArg
 }
 
 // ---- chunk ---------------------------------------------------------------------------------------------------------------
-// Decays of all rows and channels. One CTA per row.
+// Decays of all rows and channels: 64 channels x 32 rows per CTA, 32 of the rank at a time in shared memory.
 __global__ void __launch_bounds__(256) scan_decay_rows_kernel(const ScanArgs a) {
-    extern __shared__ float s_low[];
-    const size_t t = blockIdx.x;
-    for (int i = threadIdx.x; i < a.rank; i += 256) {
-        const float l = a.low[t * a.ld + i];
-        s_low[i] = a.decay_kind == TENZO_DECAY_EXP_EXP ? tanhf(l) : l;
+    __shared__ float s_up[32][65], s_low[32][33];
+    const int n = a.heads * a.dim, rank8 = (a.rank + 7) & ~7, tid = threadIdx.x;
+    const int c = tid & 63, r0 = (tid >> 6) * 8, ch0 = blockIdx.x * 64, t0 = blockIdx.y * 32;
+    float z[8] = {};
+    for (int k0 = 0; k0 < a.rank; k0 += 32) {
+        for (int i = tid; i < 64 * 32; i += 256) {
+            const int k = i & 31, cc = i >> 5;
+            s_up[k][cc] = ch0 + cc < n && k0 + k < a.rank ? to_f(static_cast<const bf16*>(a.up)[(size_t)(ch0 + cc) * rank8 + k0 + k]) : 0.0f;
+        }
+        for (int i = tid; i < 32 * 32; i += 256) {
+            const int k = i & 31, r = i >> 5;
+            const float l = t0 + r < a.M && k0 + k < a.rank ? a.low[(size_t)(t0 + r) * a.ld + k0 + k] : 0.0f;
+            s_low[r][k] = a.decay_kind == TENZO_DECAY_EXP_EXP ? tanhf(l) : l;
+        }
+        __syncthreads();
+#pragma unroll 8
+        for (int k = 0; k < 32; ++k)
+#pragma unroll
+            for (int r = 0; r < 8; ++r) z[r] = fmaf(s_up[k][c], s_low[r0 + r][k], z[r]);
+        __syncthreads();
     }
-    __syncthreads();
-    const int n = a.heads * a.dim;
-    for (int ch = threadIdx.x; ch < n; ch += 256) a.w_rows[t * n + ch] = scan_decay(a, ch, s_low);
+    if (ch0 + c >= n) return;
+#pragma unroll
+    for (int r = 0; r < 8; ++r)
+        if (t0 + r0 + r < a.M) a.w_rows[(size_t)(t0 + r0 + r) * n + ch0 + c] = gate_decay(a.decay_kind, z[r] + a.bias[ch0 + c], a.tau);
 }
 
-// A block of rows for 16 value columns of one head, 32 threads: lane = 4 * column pair + key slice; a key slice owns the
-// rows 4 * (slice + 4 j) .. + 3 of the state, so that the four slices read adjacent 16-byte pieces of k, q and w.
+// A block of rows for 32 value columns of one head, 64 threads: lane = 4 * column pair + key slice; a key slice owns the
+// rows 4 * (slice + 4 j) .. + 3 of the state, so that the four slices read adjacent 16-byte pieces of k, q and w. Rows are
+// staged by asynchronous copies, one tile ahead.
 // Pass 1 (OUT = 0) starts from zero and leaves the block's own state and decay products, pass 2 (OUT = 1) starts
-// from the state before the block and writes the outputs.
-constexpr int kScanCols = 32;                            // columns per CTA (two warps of 16)
+// from the state before the block and writes the outputs. WC: the decay is one constant per head.
+constexpr int kScanCols = 32;
 
-template <int KJ, bool OUT>
-__global__ void __launch_bounds__(64) scan_block_kernel(const ScanArgs a, int n_blocks, float* own, float* prod, const float* start) {
-    constexpr int KD = KJ * 16, kScanTile = KJ > 8 ? 8 : 16;   // padded key dimension, rows staged at a time
-    __shared__ __align__(16) float s_k[kScanTile][KD], s_q[OUT ? kScanTile : 1][KD], s_w[kScanTile][KD];
-    __shared__ __align__(16) float s_v[kScanTile][kScanCols];
+struct ScanBlockLaunch {
+    ScanArgs a;
+    float *own, *prod;
+    const float* start;
+    int vec_k, vec_v;            // key / value rows can be copied 16 bytes at a time
+};
+
+template <int KJ, bool OUT, bool WC>
+struct ScanBlockShape {
+    static constexpr int KD = KJ * 16, TILE = KJ > 8 ? 8 : 16;            // padded key size, rows per tile
+    static constexpr int K = 0, Q = TILE * KD, W = Q + (OUT ? TILE * KD : 0), V = W + (WC ? 0 : TILE * KD), FLOATS = V + TILE * kScanCols;
+};
+
+__device__ __forceinline__ void async_copy(float* dst, const float* src, int vec) {
+    if (vec) asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
+    else asm volatile("cp.async.ca.shared.global [%0], [%1], 4;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
+}
+// `rows` x `cols` floats, destination rows of ld_dst
+__device__ __forceinline__ void async_tile(float* dst, int ld_dst, const float* src, size_t ld_src, int rows, int cols, int vec) {
+    const int step = vec ? 4 : 1, per = cols / step;
+    for (int i = threadIdx.x; i < rows * per; i += 64) {
+        const int r = i / per, c = (i - r * per) * step;
+        async_copy(dst + r * ld_dst + c, src + (size_t)r * ld_src + c, vec);
+    }
+}
+
+template <int KJ, bool OUT, bool WC>
+__global__ void __launch_bounds__(64) scan_block_kernel(const ScanBlockLaunch L) {
+    using S = ScanBlockShape<KJ, OUT, WC>;
+    constexpr int KD = S::KD, TILE = S::TILE;
+    extern __shared__ __align__(16) float smem[];
+    const ScanArgs& a = L.a;
     const int head = blockIdx.y, b = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int slice = lane & 3, c0 = blockIdx.x * kScanCols + warp * 16 + (lane >> 2) * 2;
-    const int ldv = (a.vdim + 3) & ~3;
+    const int slice = lane & 3, cl = warp * 16 + (lane >> 2) * 2, c0 = blockIdx.x * kScanCols + cl;
+    const int ldv = (a.vdim + 3) & ~3, n = a.heads * a.dim;
     const int t_begin = b * kScanBlock, t_end = min(a.M, t_begin + kScanBlock);
-    float S[2][KJ * 4], P[OUT ? 1 : KJ * 4], U[OUT ? KJ * 4 : 1];
+    const int v_cols = min(kScanCols, a.vdim - (int)blockIdx.x * kScanCols);
+    for (int i = tid; i < 2 * S::FLOATS / 4; i += 64) reinterpret_cast<float4*>(smem)[i] = make_float4(0, 0, 0, 0);     // padding
+    float st[2][KJ * 4], P[OUT ? 1 : KJ * 4], U[OUT ? KJ * 4 : 1];
 #pragma unroll
     for (int j = 0; j < KJ * 4; ++j) {
         const int d = 4 * (slice + 4 * (j >> 2)) + (j & 3);
 #pragma unroll
         for (int c = 0; c < 2; ++c)
-            S[c][j] = OUT && d < a.dim && c0 + c < a.vdim ? start[((size_t)b * a.heads + head) * a.dim * ldv + (size_t)d * ldv + c0 + c] : 0.0f;
+            st[c][j] = OUT && d < a.dim && c0 + c < a.vdim ? L.start[((size_t)b * a.heads + head) * a.dim * ldv + (size_t)d * ldv + c0 + c] : 0.0f;
         if (!OUT) P[OUT ? 0 : j] = 1.0f;
         if (OUT) U[OUT ? j : 0] = a.bonus && d < a.dim ? a.bonus[head * a.dim + d] : 0.0f;
     }
-    const float w_const = a.decay_kind == TENZO_DECAY_CONST ? a.decay[head] : 0.0f;
-    for (int tb = t_begin; tb < t_end; tb += kScanTile) {
-        const int nt = min(kScanTile, t_end - tb);
-        __syncthreads();
-        for (int i = tid; i < nt * KD; i += 64) {
-            const int r = i / KD, d = i - r * KD;
-            const size_t row = (size_t)(tb + r) * a.ld + head * a.dim + d;
-            const bool in = d < a.dim;
-            s_k[r][d] = in ? a.k[row] * a.k_scale : 0.0f;
-            if (OUT) s_q[OUT ? r : 0][d] = in ? a.q[row] * a.q_scale : 0.0f;
-            s_w[r][d] = in ? (a.decay_kind == TENZO_DECAY_CONST ? w_const : a.w_rows[(size_t)(tb + r) * a.heads * a.dim + head * a.dim + d]) : 0.0f;
+    const float w_const = WC ? a.decay[head] : 0.0f;
+    auto stage = [&](int tb, float* buf) {
+        const int nt = min(TILE, t_end - tb);
+        async_tile(buf + S::K, KD, a.k + (size_t)tb * a.ld + head * a.dim, a.ld, nt, a.dim, L.vec_k);
+        if (OUT) async_tile(buf + S::Q, KD, a.q + (size_t)tb * a.ld + head * a.dim, a.ld, nt, a.dim, L.vec_k);
+        if (!WC) async_tile(buf + S::W, KD, a.w_rows + (size_t)tb * n + head * a.dim, n, nt, a.dim, L.vec_k);
+        async_tile(buf + S::V, kScanCols, a.v + (size_t)tb * a.ld + head * a.vdim + blockIdx.x * kScanCols, a.ld, nt, v_cols, L.vec_v);
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    __syncthreads();
+    stage(t_begin, smem);
+    int flip = 0;
+    for (int tb = t_begin; tb < t_end; tb += TILE, flip ^= 1) {
+        const int nt = min(TILE, t_end - tb);
+        if (tb + TILE < t_end) {
+            stage(tb + TILE, smem + (flip ^ 1) * S::FLOATS);
+            asm volatile("cp.async.wait_group 1;" ::: "memory");
+        } else {
+            asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
-        for (int i = tid; i < nt * kScanCols; i += 64) {
-            const int r = i / kScanCols, c = i - r * kScanCols, vc = blockIdx.x * kScanCols + c;
-            s_v[r][c] = vc < a.vdim ? a.v[(size_t)(tb + r) * a.ld + head * a.vdim + vc] : 0.0f;
-        }
         __syncthreads();
+        const float* buf = smem + flip * S::FLOATS;
         for (int r = 0; r < nt; ++r) {
-            const float2 v = *reinterpret_cast<const float2*>(&s_v[r][warp * 16 + (lane >> 2) * 2]);
-            float o0 = 0.0f, o1 = 0.0f;
+            float2 v = *reinterpret_cast<const float2*>(buf + S::V + r * kScanCols + cl);
+            v.x *= a.k_scale;
+            v.y *= a.k_scale;
+            float o0[2] = {}, o1[2] = {};
 #pragma unroll
             for (int jj = 0; jj < KJ; ++jj) {
-                const int d = 4 * (slice + 4 * jj);
-                const float4 k4 = *reinterpret_cast<const float4*>(&s_k[r][d]), w4 = *reinterpret_cast<const float4*>(&s_w[r][d]);
-                const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, ww[4] = {w4.x, w4.y, w4.z, w4.w};
-                float qq[4] = {};
-                if (OUT) {
-                    const float4 q4 = *reinterpret_cast<const float4*>(&s_q[OUT ? r : 0][d]);
-                    qq[0] = q4.x; qq[1] = q4.y; qq[2] = q4.z; qq[3] = q4.w;
-                }
+                const int d = r * KD + 4 * (slice + 4 * jj);
+                const float4 k4 = *reinterpret_cast<const float4*>(buf + S::K + d);
+                const float4 w4 = WC ? make_float4(w_const, w_const, w_const, w_const) : *reinterpret_cast<const float4*>(buf + S::W + d);
+                const float4 q4 = OUT ? *reinterpret_cast<const float4*>(buf + S::Q + d) : make_float4(0, 0, 0, 0);
+                const float kk[4] = {k4.x, k4.y, k4.z, k4.w}, ww[4] = {w4.x, w4.y, w4.z, w4.w}, qq[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
                     const int j = jj * 4 + i;
                     const float kv0 = kk[i] * v.x, kv1 = kk[i] * v.y;
                     if (OUT && a.bonus) {
-                        o0 = fmaf(qq[i], fmaf(U[OUT ? j : 0], kv0, S[0][j]), o0);
-                        o1 = fmaf(qq[i], fmaf(U[OUT ? j : 0], kv1, S[1][j]), o1);
+                        o0[i & 1] = fmaf(qq[i], fmaf(U[OUT ? j : 0], kv0, st[0][j]), o0[i & 1]);
+                        o1[i & 1] = fmaf(qq[i], fmaf(U[OUT ? j : 0], kv1, st[1][j]), o1[i & 1]);
                     }
-                    S[0][j] = fmaf(ww[i], S[0][j], kv0);
-                    S[1][j] = fmaf(ww[i], S[1][j], kv1);
+                    st[0][j] = fmaf(ww[i], st[0][j], kv0);
+                    st[1][j] = fmaf(ww[i], st[1][j], kv1);
                     if (OUT && !a.bonus) {
-                        o0 = fmaf(qq[i], S[0][j], o0);
-                        o1 = fmaf(qq[i], S[1][j], o1);
+                        o0[i & 1] = fmaf(qq[i], st[0][j], o0[i & 1]);
+                        o1[i & 1] = fmaf(qq[i], st[1][j], o1[i & 1]);
                     }
                     if (!OUT) P[OUT ? 0 : j] *= ww[i];
                 }
             }
             if (OUT) {
-                o0 += __shfl_xor_sync(0xffffffffu, o0, 1);
-                o1 += __shfl_xor_sync(0xffffffffu, o1, 1);
-                o0 += __shfl_xor_sync(0xffffffffu, o0, 2);
-                o1 += __shfl_xor_sync(0xffffffffu, o1, 2);
+                float s0 = o0[0] + o0[1], s1 = o1[0] + o1[1];
+                s0 += __shfl_xor_sync(0xffffffffu, s0, 1);
+                s1 += __shfl_xor_sync(0xffffffffu, s1, 1);
+                s0 += __shfl_xor_sync(0xffffffffu, s0, 2);
+                s1 += __shfl_xor_sync(0xffffffffu, s1, 2);
                 float* o = a.o_rows + (size_t)(tb + r) * a.heads * a.vdim + head * a.vdim + c0;
-                if (slice == 0 && c0 < a.vdim) o[0] = o0;
-                if (slice == 1 && c0 + 1 < a.vdim) o[1] = o1;
+                if (slice == 0 && c0 < a.vdim) o[0] = s0 * a.q_scale;
+                if (slice == 1 && c0 + 1 < a.vdim) o[1] = s1 * a.q_scale;
             }
         }
+        __syncthreads();                                     // the tile is free for the copies after next
     }
     if (!OUT) {
 #pragma unroll
         for (int j = 0; j < KJ * 4; ++j) {
             const int d = 4 * (slice + 4 * (j >> 2)) + (j & 3);
             if (d >= a.dim) continue;
-            float* dst = own + ((size_t)b * a.heads + head) * a.dim * ldv + (size_t)d * ldv + c0;
-            if (c0 < a.vdim) dst[0] = S[0][j];
-            if (c0 + 1 < a.vdim) dst[1] = S[1][j];
-            if (blockIdx.x == 0 && tid < 4) prod[((size_t)b * a.heads + head) * a.dim + d] = P[OUT ? 0 : j];
+            float* dst = L.own + ((size_t)b * a.heads + head) * a.dim * ldv + (size_t)d * ldv + c0;
+            if (c0 < a.vdim) dst[0] = st[0][j];
+            if (c0 + 1 < a.vdim) dst[1] = st[1][j];
+            if (blockIdx.x == 0 && tid < 4) L.prod[((size_t)b * a.heads + head) * a.dim + d] = P[OUT ? 0 : j];
         }
     }
 }
@@ -222,10 +298,19 @@ __global__ void __launch_bounds__(256) scan_carry_kernel(const ScanArgs a, int n
     if (i >= n || (int)(i % ldv) >= a.vdim) return;
     const size_t row = i / ldv;
     float s = a.state[i];
-    for (int b = 0; b < n_blocks; ++b) {
-        const float mine = own[(size_t)b * n + i];
-        own[(size_t)b * n + i] = s;
-        s = fmaf(prod[(size_t)b * a.heads * a.dim + row], s, mine);
+    for (int b0 = 0; b0 < n_blocks; b0 += 8) {                // eight blocks' values in flight
+        float mine[8], p[8];
+#pragma unroll
+        for (int u = 0; u < 8; ++u) {
+            mine[u] = b0 + u < n_blocks ? own[(size_t)(b0 + u) * n + i] : 0.0f;
+            p[u] = b0 + u < n_blocks ? prod[(size_t)(b0 + u) * a.heads * a.dim + row] : 0.0f;
+        }
+#pragma unroll
+        for (int u = 0; u < 8; ++u)
+            if (b0 + u < n_blocks) {
+                own[(size_t)(b0 + u) * n + i] = s;
+                s = fmaf(p[u], s, mine[u]);
+            }
     }
     a.state[i] = s;
 }
@@ -266,7 +351,7 @@ int launch_scan(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernel
     if (a.decode) {
         int nc2 = 1;
         while (nc2 < ldv / 4) nc2 *= 2;
-        const size_t smem = 4 * (size_t)(((4 * a.dim + rank + ldv + 3) & ~3) + kScanThreads / nc2 * ldv + 8);
+        const size_t smem = 4 * (size_t)(((4 * a.dim + round_up(rank, 8) + ldv + 3) & ~3) + kScanThreads / nc2 * ldv + 8);
         const dim3 grid(a.heads, a.M);
         *n_kernels += 1;
         auto go = [&](auto kernel) {
@@ -279,19 +364,29 @@ int launch_scan(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernel
     float* own = a.part;
     float* prod = own + (size_t)n_blocks * a.heads * a.dim * ldv;
     if (rank) {
-        scan_decay_rows_kernel<<<a.M, 256, rank * 4, st>>>(p);
+        scan_decay_rows_kernel<<<dim3((a.heads * a.dim + 63) / 64, (a.M + 31) / 32), 256, 0, st>>>(p);
         *n_kernels += 1;
     }
+    auto aligned = [](const void* q) { return (reinterpret_cast<uintptr_t>(q) & 15) == 0; };
+    ScanBlockLaunch L = {p, own, prod, own, 0, 0};
+    L.vec_k = a.dim % 4 == 0 && a.ld % 4 == 0 && aligned(a.q) && aligned(a.k) && aligned(a.w_rows);
+    L.vec_v = a.vdim % 4 == 0 && a.ld % 4 == 0 && aligned(a.v);
     const dim3 grid((a.vdim + kScanCols - 1) / kScanCols, a.heads, n_blocks);
-    auto blocks = [&](auto k1, auto k2) {
-        k1<<<grid, 64, 0, st>>>(p, n_blocks, own, prod, nullptr);
+    auto blocks = [&](auto kj, auto wc) {
+        constexpr int KJ = decltype(kj)::value;
+        constexpr bool WC = decltype(wc)::value;
+        const size_t s1 = 8 * ScanBlockShape<KJ, false, WC>::FLOATS, s2 = 8 * ScanBlockShape<KJ, true, WC>::FLOATS;
+        if (int rc = allow_smem(scan_block_kernel<KJ, false, WC>, s1)) return rc;
+        if (int rc = allow_smem(scan_block_kernel<KJ, true, WC>, s2)) return rc;
+        scan_block_kernel<KJ, false, WC><<<grid, 64, s1, st>>>(L);
         scan_carry_kernel<<<(unsigned)(((size_t)a.heads * a.dim * ldv + 255) / 256), 256, 0, st>>>(p, n_blocks, own, prod);
-        k2<<<grid, 64, 0, st>>>(p, n_blocks, nullptr, nullptr, own);
+        scan_block_kernel<KJ, true, WC><<<grid, 64, s2, st>>>(L);
+        return (int)cudaGetLastError();
     };
-    if (a.dim <= 32) blocks(scan_block_kernel<2, false>, scan_block_kernel<2, true>);
-    else if (a.dim <= 64) blocks(scan_block_kernel<4, false>, scan_block_kernel<4, true>);
-    else if (a.dim <= 128) blocks(scan_block_kernel<8, false>, scan_block_kernel<8, true>);
-    else blocks(scan_block_kernel<16, false>, scan_block_kernel<16, true>);
+    auto sized = [&](auto kj) { return rank ? blocks(kj, std::false_type()) : blocks(kj, std::true_type()); };
+    const int rc = a.dim <= 32 ? sized(std::integral_constant<int, 2>()) : a.dim <= 64 ? sized(std::integral_constant<int, 4>())
+                 : a.dim <= 128 ? sized(std::integral_constant<int, 8>()) : sized(std::integral_constant<int, 16>());
+    if (rc) return rc;
     const unsigned gate_ctas = (unsigned)(((size_t)a.M * a.heads + 7) / 8);
     if (a.f32) scan_gate_kernel<float><<<gate_ctas, 256, 0, st>>>(p);
     else scan_gate_kernel<bf16><<<gate_ctas, 256, 0, st>>>(p);

@@ -1,172 +1,246 @@
 // Row kernels of the hybrid decoders: residual update, RMS norm with one gain, causal convolution over time on every
-// channel, and the token-shift mixes of a time-mixing layer, in one pass over the residual.
+// channel, and the token-shift mixes of a time-mixing layer (tenzo_rows_args).
 //
-// A CTA owns TR consecutive rows (one row in decode) and keeps their normalised inputs in shared memory, plus the rows
-// before them that the convolution and the shift reach back to. Those halo rows are recomputed from the residual
-// source instead of being exchanged between CTAs, which is why the updated residual goes to a second buffer; before the
-// first row of the launch they come from the sequence's carried state.
+// Decode: one CTA per sequence does all of it; a thread keeps its columns in registers, with the convolution's weights and
+// the carried inputs fetched before the kernel waits for its producer (the launch that wrote them lies a whole step back).
+// Chunk (and decode of rows wider than that): one kernel updates the residual and leaves each row's inverse RMS, a second
+// one walks tiles of rows per channel with the convolution's inputs in registers.
 #include "hybrid_common.cuh"
 
 namespace tz {
 
-constexpr int kRowThreads = 512;
+constexpr int kStepThreads = 1024, kStepTaps = 4, kStepMaxCols = 4;
+constexpr int kNormThreads = 256, kConvThreads = 128, kConvRows = 16;
 
-struct RowsLaunch {
-    RowsArgs a;
-    int TR, halo;
+// Sums of two values over the block, the same bits in every thread. scratch: 2 * 32 floats, not reused by the next call.
+__device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
+    const int lane = threadIdx.x & 31, nw = blockDim.x >> 5;
+    v.x = warp_sum(v.x);
+    v.y = warp_sum(v.y);
+    if (lane == 0) scratch[threadIdx.x >> 5] = v;
+    __syncthreads();
+    const float2 p = lane < nw ? scratch[lane] : make_float2(0.0f, 0.0f);
+    return make_float2(warp_sum(p.x), warp_sum(p.y));
+}
+
+struct RowSource {                              // where a row's residual comes from
+    const RowsArgs& a;
+    const bf16 *e = nullptr, *p = nullptr;
+    const float *x = nullptr, *y0 = nullptr, *y1 = nullptr;
+    __device__ __forceinline__ RowSource(const RowsArgs& args, int t) : a(args) {
+        if (a.tokens) {
+            const int tok = min(max(a.tokens[t], 0), a.vocab - 1), pos = min(max(a.pos[t], 0), a.n_pos - 1);
+            e = static_cast<const bf16*>(a.embed) + (size_t)tok * a.width;
+            p = static_cast<const bf16*>(a.pos_table) + (size_t)pos * a.width;
+        } else {
+            x = a.x_in + (size_t)t * a.width;
+            y0 = a.y0 ? a.y0 + (size_t)t * a.ld_y : nullptr;
+            y1 = a.y1 ? a.y1 + (size_t)t * a.ld_y : nullptr;
+        }
+    }
+    // without the two normed addends
+    __device__ __forceinline__ float plain(int c) const {
+        if (e) return to_f(e[c]) + to_f(p[c]);
+        return y0 && !y1 ? x[c] + y0[c] : x[c];
+    }
 };
 
-__device__ __forceinline__ float rows_source(const RowsArgs& a, int t, int c, float inv0, float inv1, int tok, int p) {
-    if (a.tokens) return to_f(static_cast<const bf16*>(a.embed)[(size_t)tok * a.width + c]) + to_f(static_cast<const bf16*>(a.pos_table)[(size_t)p * a.width + c]);
-    float x = a.x_in[(size_t)t * a.width + c];
-    if (a.y1) {
-        const float l = a.y0[(size_t)t * a.ld_y + c] * inv0 * a.w0[c], r = a.y1[(size_t)t * a.ld_y + c] * inv1 * a.w1[c];
-        x += 0.5f * (l + r);
-    } else if (a.y0) {
-        x += a.y0[(size_t)t * a.ld_y + c];
+// CPT columns per thread: c = threadIdx.x + i * kStepThreads.
+template <typename T, int CPT>
+__global__ void __launch_bounds__(kStepThreads) rows_step_kernel(const RowsArgs a) {
+    __shared__ float2 s_red[2][32];
+    const int row = blockIdx.x, width = a.width, taps = a.conv_w ? a.taps : 1, nt = taps - 1;
+    const size_t off = (size_t)row * a.seq_stride;
+    // w[3] belongs to the current input, u[0..2] are the three before it; both are zero beyond the convolution's reach
+    float w[CPT][kStepTaps], u[CPT][kStepTaps - 1], prev[CPT];
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+        const int c = threadIdx.x + i * kStepThreads;
+        const bool in = c < width;
+#pragma unroll
+        for (int j = 0; j < kStepTaps; ++j) w[i][j] = in && a.conv_w && j >= kStepTaps - taps ? a.conv_w[(size_t)(j - kStepTaps + taps) * width + c] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < kStepTaps - 1; ++j)
+            u[i][j] = in && j >= kStepTaps - 1 - nt ? a.tail_in[off + (size_t)(j - (kStepTaps - 1 - nt)) * width + c] : 0.0f;
+        prev[i] = in && a.mu ? a.prev_in[off + c] : 0.0f;
     }
-    return x;
-}
-
-// Sum over the group's threads: a warp (chunk launches: one warp per row) or the whole block (decode).
-template <bool DECODE>
-__device__ __forceinline__ float group_sum(float v, float* scratch) {
-    return DECODE ? block_sum(v, scratch) : warp_sum(v);
-}
-
-// NT: taps rounded up to 4 or 16.
-template <typename T, bool DECODE, int NT>
-__global__ void __launch_bounds__(kRowThreads) rows_kernel(const RowsLaunch L) {
-    extern __shared__ float s_h[];                      // [halo + TR][width]
-    __shared__ float s_red[kRowThreads / 32];
-    const RowsArgs& a = L.a;
-    const int width = a.width, halo = L.halo;
-    const int t0 = blockIdx.x * L.TR, n_rows = min(L.TR, a.M - t0);
     pdl_wait();
     pdl_launch_dependents();
-    const float* tail_in = a.tail_in;
-    const float* prev_in = a.prev_in;
-    float *tail_out = a.tail_out, *prev_out = a.prev_out;
-    if (DECODE) {
-        const size_t off = (size_t)blockIdx.x * a.seq_stride;
-        tail_in += off; tail_out += off;
-        if (prev_in) { prev_in += off; prev_out += off; }
-    }
-    const int lane_g = DECODE ? threadIdx.x : (threadIdx.x & 31), size_g = DECODE ? kRowThreads : 32;
-    const int groups = DECODE ? 1 : kRowThreads / 32, group = DECODE ? 0 : threadIdx.x >> 5;
-    const float inv_w = 1.0f / (float)width;
-    // rows of this launch: residual, norm
-    for (int r = group; r < halo + n_rows; r += groups) {
-        const int t = t0 - halo + r;
-        if (DECODE ? r < halo : t < 0) continue;
-        int tok = 0, p = 0;
-        if (a.tokens) {
-            tok = min(max(a.tokens[t], 0), a.vocab - 1);
-            p = min(max(a.pos[t], 0), a.n_pos - 1);
+    const RowSource src(a, row);
+    float x[CPT], l[CPT], r[CPT];
+    float2 q = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+        const int c = threadIdx.x + i * kStepThreads;
+        x[i] = l[i] = r[i] = 0.0f;
+        if (c >= width) continue;
+        x[i] = src.plain(c);
+        if (src.y1) {
+            l[i] = src.y0[c];
+            r[i] = src.y1[c];
+            q.x = fmaf(l[i], l[i], q.x);
+            q.y = fmaf(r[i], r[i], q.y);
         }
-        float inv0 = 0.0f, inv1 = 0.0f;
-        if (a.y1) {
-            float q0 = 0.0f, q1 = 0.0f;
-            for (int c = lane_g; c < width; c += size_g) {
-                const float u = a.y0[(size_t)t * a.ld_y + c], v = a.y1[(size_t)t * a.ld_y + c];
-                q0 = fmaf(u, u, q0);
-                q1 = fmaf(v, v, q1);
-            }
-            q0 = group_sum<DECODE>(q0, s_red);
-            q1 = group_sum<DECODE>(q1, s_red);
-            inv0 = 1.0f / sqrtf(q0 * inv_w + a.eps);
-            inv1 = 1.0f / sqrtf(q1 * inv_w + a.eps);
-        }
-        float* hrow = s_h + (size_t)r * width;
-        float q = 0.0f;
-#pragma unroll 4
-        for (int c = lane_g; c < width; c += size_g) {
-            const float x = rows_source(a, t, c, inv0, inv1, tok, p);
-            q = fmaf(x, x, q);
-            hrow[c] = x;
-            if (r >= halo) a.x_out[(size_t)t * width + c] = x;
-        }
-        q = group_sum<DECODE>(q, s_red);
-        const float inv = 1.0f / sqrtf(q * inv_w + a.eps);
-        for (int c = lane_g; c < width; c += size_g) hrow[c] = hrow[c] * inv * a.gain;   // a thread rescales what it stored
     }
-    // rows before the launch, from the carried state
-    const int taps = a.conv_w ? a.taps : 1, nt = taps - 1;
-    for (int r = 0; r < halo; ++r) {
-        const int t = DECODE ? r - halo : t0 - halo + r;        // relative to the launch's first row
-        if (t >= 0) break;
-        if (t < -nt) continue;                                   // only the shift's own state reaches there
-        for (int c = threadIdx.x; c < width; c += kRowThreads) s_h[(size_t)r * width + c] = tail_in[(size_t)(nt + t) * width + c];
+    if (src.y1) {
+        q = block_sum2(q, s_red[0]);
+        const float i0 = 1.0f / sqrtf(q.x / (float)width + a.eps), i1 = 1.0f / sqrtf(q.y / (float)width + a.eps);
+#pragma unroll
+        for (int i = 0; i < CPT; ++i) {
+            const int c = threadIdx.x + i * kStepThreads;
+            if (c < width) x[i] += 0.5f * (l[i] * i0 * a.w0[c] + r[i] * i1 * a.w1[c]);
+        }
     }
-    __syncthreads();
-    // convolution, mixes
-    T* out = reinterpret_cast<T*>(a.out);
+    q = make_float2(0.0f, 0.0f);
+#pragma unroll
+    for (int i = 0; i < CPT; ++i) {
+        const int c = threadIdx.x + i * kStepThreads;
+        if (c < width) a.x_out[(size_t)row * width + c] = x[i];
+        q.x = fmaf(x[i], x[i], q.x);
+    }
+    q = block_sum2(q, s_red[1]);
+    const float inv = 1.0f / sqrtf(q.x / (float)width + a.eps);
+    T* out = reinterpret_cast<T*>(a.out) + (size_t)row * a.ld_out;
     const size_t mix_stride = (size_t)a.M * a.ld_out;
-    const bool lead = a.mu && !DECODE && t0 > 0;                 // the shift starts from the row before, recomputed
-    for (int c = threadIdx.x; c < width; c += kRowThreads) {
-        // w[NT-1] belongs to the current row; u holds the last NT inputs, those before the convolution's reach as zero
-        float w[NT], u[NT];
-        const int start = lead ? -1 : 0;
 #pragma unroll
-        for (int j = 0; j < NT; ++j) {
-            const bool in = j >= NT - taps;
-            w[j] = in && a.conv_w ? a.conv_w[(size_t)(j - NT + taps) * width + c] : 0.0f;
-            u[j] = j > NT - taps && a.conv_w ? s_h[(size_t)max(0, halo + start - NT + j) * width + c] : 0.0f;
+    for (int i = 0; i < CPT; ++i) {
+        const int c = threadIdx.x + i * kStepThreads;
+        if (c >= width) continue;
+        const float h = x[i] * inv * a.gain;
+        float z = 0.0f;
+#pragma unroll
+        for (int j = 0; j < kStepTaps - 1; ++j) z = fmaf(w[i][j], u[i][j], z);
+        const float y = h + fmaf(w[i][kStepTaps - 1], h, z);
+        if (a.mu) {
+            for (int s = 0; s < a.n_mix; ++s) out[s * mix_stride + c] = from_f<T>(fmaf(prev[i] - y, a.mu[(size_t)s * width + c], y));
+            a.prev_out[off + c] = y;
+        } else {
+            out[c] = from_f<T>(y);
         }
-        float prev = a.mu && !lead ? prev_in[c] : 0.0f;
-        for (int i = start; i < n_rows; ++i) {
 #pragma unroll
-            for (int j = 0; j + 1 < NT; ++j) u[j] = u[j + 1];
-            u[NT - 1] = s_h[(size_t)(halo + i) * width + c];
-            float y = u[NT - 1];
-            if (a.conv_w) {
-                float z = 0.0f;
-#pragma unroll
-                for (int j = 0; j < NT; ++j) z = fmaf(w[j], u[j], z);
-                y += z;
-            }
-            if (i >= 0) {
-                const size_t row = (size_t)(t0 + i) * a.ld_out + c;
-                if (a.mu) {
-                    for (int s = 0; s < a.n_mix; ++s) out[s * mix_stride + row] = from_f<T>(fmaf(prev - y, a.mu[(size_t)s * width + c], y));
-                } else {
-                    out[row] = from_f<T>(y);
-                }
-            }
-            prev = y;
-        }
-        if (t0 + n_rows == a.M || DECODE) {                      // the state after the last row
-            if (a.mu) prev_out[c] = prev;
-            for (int i = 0; i < nt; ++i)                         // rows n_rows - nt .. n_rows - 1 relative to the tile
-                tail_out[(size_t)i * width + c] = s_h[(size_t)(halo + n_rows - nt + i) * width + c];
+        for (int j = 0; j < kStepTaps - 1; ++j) {                // the tail moves up by one
+            const int k = j - (kStepTaps - 1 - nt);
+            if (k >= 0) a.tail_out[off + (size_t)k * width + c] = j + 1 < kStepTaps - 1 ? u[i][j + 1] : h;
         }
     }
 }
 
-int launch_rows(const RowsArgs& a, cudaStream_t st) {
+// Residual and inverse RMS of a row.
+__global__ void __launch_bounds__(kNormThreads) rows_norm_kernel(const RowsArgs a) {
+    __shared__ float2 s_red[2][32];
+    const int t = blockIdx.x, width = a.width;
+    pdl_wait();
+    pdl_launch_dependents();
+    const RowSource src(a, t);
+    float i0 = 0.0f, i1 = 0.0f;
+    float2 q = make_float2(0.0f, 0.0f);
+    if (src.y1) {
+#pragma unroll 4
+        for (int c = threadIdx.x; c < width; c += kNormThreads) {
+            const float u = src.y0[c], v = src.y1[c];
+            q.x = fmaf(u, u, q.x);
+            q.y = fmaf(v, v, q.y);
+        }
+        q = block_sum2(q, s_red[0]);
+        i0 = 1.0f / sqrtf(q.x / (float)width + a.eps);
+        i1 = 1.0f / sqrtf(q.y / (float)width + a.eps);
+    }
+    q = make_float2(0.0f, 0.0f);
+    float* xo = a.x_out + (size_t)t * width;
+#pragma unroll 4
+    for (int c = threadIdx.x; c < width; c += kNormThreads) {
+        float x = src.plain(c);
+        if (src.y1) x += 0.5f * (src.y0[c] * i0 * a.w0[c] + src.y1[c] * i1 * a.w1[c]);
+        xo[c] = x;
+        q.x = fmaf(x, x, q.x);
+    }
+    q = block_sum2(q, s_red[1]);
+    if (threadIdx.x == 0) a.row_inv[t] = 1.0f / sqrtf(q.x / (float)width + a.eps);
+}
+
+// Convolution and mixes over kConvRows rows of one channel per thread; decode: one row, with its own carried state.
+// NT: taps rounded up to 4 or 16.
+template <typename T, bool DECODE, int NT>
+__global__ void __launch_bounds__(kConvThreads) rows_conv_kernel(const RowsArgs a) {
+    const int c = blockIdx.x * kConvThreads + threadIdx.x, width = a.width, taps = a.conv_w ? a.taps : 1, nt = taps - 1;
+    pdl_wait();
+    pdl_launch_dependents();
+    if (c >= width) return;
+    const int t0 = blockIdx.y * (DECODE ? 1 : kConvRows), n_rows = DECODE ? 1 : min(kConvRows, a.M - t0);
+    const size_t off = DECODE ? (size_t)t0 * a.seq_stride : 0;
+    const float* tail_in = a.tail_in + off;
+    // input of the convolution at row t: from the launch, or from the carried rows before it
+    auto input = [&](int t) {
+        const int rel = DECODE ? t - t0 : t;
+        if (rel < 0) return rel >= -nt ? tail_in[(size_t)(nt + rel) * width + c] : 0.0f;
+        return a.x_out[(size_t)t * width + c] * a.row_inv[t] * a.gain;
+    };
+    const bool lead = a.mu && !DECODE && t0 > 0;                 // the shift starts from the row before, recomputed
+    const int start = lead ? -1 : 0;
+    float w[NT], u[NT];                                          // w[NT-1] belongs to the current row
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+        w[j] = a.conv_w && j >= NT - taps ? a.conv_w[(size_t)(j - NT + taps) * width + c] : 0.0f;
+        u[j] = a.conv_w && j > NT - taps ? input(t0 + start - NT + j) : 0.0f;
+    }
+    float prev = a.mu && !lead ? a.prev_in[off + c] : 0.0f, in[kConvRows + 1];
+#pragma unroll
+    for (int i = 0; i <= (DECODE ? 0 : kConvRows); ++i) in[i] = start + i < n_rows ? input(t0 + start + i) : 0.0f;
+    T* out = reinterpret_cast<T*>(a.out);
+    const size_t mix_stride = (size_t)a.M * a.ld_out;
+#pragma unroll
+    for (int k = 0; k <= (DECODE ? 0 : kConvRows); ++k) {
+        const int i = start + k;
+        if (i >= n_rows) break;
+#pragma unroll
+        for (int j = 0; j + 1 < NT; ++j) u[j] = u[j + 1];
+        u[NT - 1] = in[k];
+        float z = 0.0f;
+#pragma unroll
+        for (int j = 0; j < NT; ++j) z = fmaf(w[j], u[j], z);
+        const float y = in[k] + z;
+        if (i >= 0) {
+            const size_t row = (size_t)(t0 + i) * a.ld_out + c;
+            if (a.mu) {
+                for (int s = 0; s < a.n_mix; ++s) out[s * mix_stride + row] = from_f<T>(fmaf(prev - y, a.mu[(size_t)s * width + c], y));
+            } else {
+                out[row] = from_f<T>(y);
+            }
+        }
+        prev = y;
+    }
+    if (DECODE || t0 + n_rows == a.M) {                          // the state after the last row
+        if (a.mu) a.prev_out[off + c] = prev;
+        float last[NT];
+#pragma unroll
+        for (int j = 0; j < NT; ++j) last[j] = j < nt ? input(t0 + n_rows - nt + j) : 0.0f;
+#pragma unroll
+        for (int j = 0; j < NT; ++j)
+            if (j < nt) a.tail_out[off + (size_t)j * width + c] = last[j];
+    }
+}
+
+int launch_rows(const RowsArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
     if (a.M <= 0) return 0;
     if (a.taps < 1 || a.taps > kMaxTaps || a.width <= 0 || a.n_mix > 8) return -1;
-    RowsLaunch L;
-    L.a = a;
-    const int nt = a.conv_w ? a.taps - 1 : 0;
-    L.halo = a.decode ? nt : nt + (a.mu ? 1 : 0);
-    const size_t row_bytes = (size_t)a.width * 4;
-    L.TR = 1;
-    if (!a.decode)
-        while (L.TR < 8 && (L.halo + 2 * L.TR) * row_bytes <= 108 * 1024) L.TR *= 2;
-    const size_t smem = (L.halo + L.TR) * row_bytes;
-    if (smem > 220 * 1024) return -1;
-    const dim3 grid((a.M + L.TR - 1) / L.TR);
-    auto go = [&](auto kernel) {
-        if (int rc = allow_smem(kernel, smem)) return rc;
-        return launch_kernel(kernel, grid, dim3(kRowThreads), smem, st, a.use_pdl, 1, L);
-    };
-    if (a.taps <= 4) {
-        if (a.f32) return a.decode ? go(rows_kernel<float, true, 4>) : go(rows_kernel<float, false, 4>);
-        return a.decode ? go(rows_kernel<bf16, true, 4>) : go(rows_kernel<bf16, false, 4>);
+    if (a.decode && a.width <= kStepThreads * kStepMaxCols && a.taps <= kStepTaps) {
+        auto go = [&](auto kernel) { return launch_kernel(kernel, dim3(a.M), dim3(kStepThreads), 0, st, a.use_pdl, 1, a); };
+        *n_kernels += 1;
+        const int cols = (a.width + kStepThreads - 1) / kStepThreads;
+        if (a.f32) return cols == 1 ? go(rows_step_kernel<float, 1>) : cols == 2 ? go(rows_step_kernel<float, 2>) : go(rows_step_kernel<float, 4>);
+        return cols == 1 ? go(rows_step_kernel<bf16, 1>) : cols == 2 ? go(rows_step_kernel<bf16, 2>) : go(rows_step_kernel<bf16, 4>);
     }
-    if (a.f32) return a.decode ? go(rows_kernel<float, true, kMaxTaps>) : go(rows_kernel<float, false, kMaxTaps>);
-    return a.decode ? go(rows_kernel<bf16, true, kMaxTaps>) : go(rows_kernel<bf16, false, kMaxTaps>);
+    if (!a.row_inv) return -1;
+    *n_kernels += 2;
+    if (int rc = launch_kernel(rows_norm_kernel, dim3(a.M), dim3(kNormThreads), 0, st, a.use_pdl, 1, a)) return rc;
+    const dim3 grid((a.width + kConvThreads - 1) / kConvThreads, a.decode ? a.M : (a.M + kConvRows - 1) / kConvRows);
+    auto go = [&](auto kernel) { return launch_kernel(kernel, grid, dim3(kConvThreads), 0, st, a.use_pdl, 1, a); };
+    if (a.taps <= 4) {
+        if (a.f32) return a.decode ? go(rows_conv_kernel<float, true, 4>) : go(rows_conv_kernel<float, false, 4>);
+        return a.decode ? go(rows_conv_kernel<bf16, true, 4>) : go(rows_conv_kernel<bf16, false, 4>);
+    }
+    if (a.f32) return a.decode ? go(rows_conv_kernel<float, true, kMaxTaps>) : go(rows_conv_kernel<float, false, kMaxTaps>);
+    return a.decode ? go(rows_conv_kernel<bf16, true, kMaxTaps>) : go(rows_conv_kernel<bf16, false, kMaxTaps>);
 }
 
 }  // namespace tz
@@ -175,5 +249,6 @@ extern "C" int tenzo_cuda_rows(const tenzo_rows_args* args, void* stream) {
     if (!args) return TENZO_ERROR_INVALID_ARGUMENT;
     tz::RowsArgs a;
     static_cast<tenzo_rows_args&>(a) = *args;
-    return tz::launch_rows(a, static_cast<cudaStream_t>(stream));
+    unsigned long long n = 0;
+    return tz::launch_rows(a, static_cast<cudaStream_t>(stream), &n);
 }

@@ -34,13 +34,49 @@ __device__ __forceinline__ float conv_step(const float* w, int ch, int n_ch, int
 struct WaDecodeLaunch {
     WindowAttnArgs a;
     int ldd, ldv, group;         // padded row lengths, query heads per kv head
-    int nvc;                     // value chunks of 8 per lane group, rounded up to a power of two
+    int nvc;                     // value chunks of 8 per key, rounded up to a power of two
 };
 
-// GQ query heads at a time.
-template <typename T, int GQ>
-__global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecodeLaunch L) {
+__device__ __forceinline__ void load_raw(const bf16* p, uint4 (&r)[1]) { r[0] = *reinterpret_cast<const uint4*>(p); }
+__device__ __forceinline__ void load_raw(const float* p, uint4 (&r)[2]) {
+    r[0] = reinterpret_cast<const uint4*>(p)[0];
+    r[1] = reinterpret_cast<const uint4*>(p)[1];
+}
+__device__ __forceinline__ void raw_floats(const uint4 (&r)[1], float (&f)[8]) { unpack8(r[0], f); }
+__device__ __forceinline__ void raw_floats(const uint4 (&r)[2], float (&f)[8]) {
+    const uint32_t b[8] = {r[0].x, r[0].y, r[0].z, r[0].w, r[1].x, r[1].y, r[1].z, r[1].w};
+#pragma unroll
+    for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(b[i]);
+}
+
+// Sums of GQ values over groups of LK lanes: halves of the values travel while there are several, so that the total is
+// GQ - 1 + log2(LK / GQ) exchanges. The lane is left with the sum of value `which`.
+template <int GQ, int LK>
+__device__ __forceinline__ float group_sums(float (&s)[GQ], int lane, int& which) {
+    which = 0;
+    int m = LK / 2;
+#pragma unroll
+    for (int n = GQ; n > 1; n >>= 1, m >>= 1) {
+        const bool up = lane & m;
+#pragma unroll
+        for (int i = 0; i < n / 2; ++i) {
+            const float send = up ? s[i] : s[i + n / 2], keep = up ? s[i + n / 2] : s[i];
+            s[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+        }
+        if (up) which += n / 2;
+    }
+#pragma unroll
+    for (; m > 0; m >>= 1) s[0] += __shfl_xor_sync(0xffffffffu, s[0], m);
+    return s[0];
+}
+
+// GQ query heads at a time (1, 2 or 4); LK lanes share a key, eight elements each. A lane's piece of the queries is in
+// registers, and the rows of several keys are requested before the first is used.
+template <typename T, int GQ, int LK>
+__global__ void __launch_bounds__(kWaThreads, 2) window_decode_kernel(const WaDecodeLaunch L) {
     extern __shared__ float sm[];
+    constexpr int RAW = sizeof(T) / 2;                   // 16-byte words of eight elements
+    constexpr int KU = (GQ == 4 ? 4 : 8) / RAW, VU = KU, KW = 32 / LK;   // rows in flight per lane, keys per warp and trip
     const WindowAttnArgs& a = L.a;
     cg::cluster_group cluster = cg::this_cluster();
     const int rank = (int)cluster.block_rank(), n_rank = (int)cluster.num_blocks();
@@ -52,7 +88,6 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
     float* s_p = s_v + ldv;                              // [GQ][kWaSeg]
     float* s_acc = s_p + GQ * kWaSeg;                    // [kWaWarps][GQ][ldv] per-warp value sums; [0] holds the CTA's sum
     float* s_ml = s_acc + kWaWarps * GQ * ldv;           // [2][GQ] running maximum and denominator of this CTA
-    float* s_red = s_ml + 2 * GQ;                        // [32]
     pdl_wait();
     pdl_launch_dependents();
     const int pos = a.pos[seq];
@@ -61,18 +96,20 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
     float* tail_out = a.tail_out + (size_t)seq * a.tail_seq_stride;
     const float *pq = a.q + (size_t)seq * a.ld, *pk = a.k + (size_t)seq * a.ld, *pv = a.v + (size_t)seq * a.ld;
 
-    for (int i = tid; i < group * ldd; i += kWaThreads) {
-        const int g = i / ldd, d = i - g * ldd, ch = (kvh * group + g) * a.dim + d;
-        // the query as the storage type holds it, times the scale
-        s_q[i] = d < a.dim ? to_f(from_f<T>(conv_step(a.conv_q, ch, n_q, a.taps, tail + ch, n_ch, pq[ch]))) * a.scale : 0.0f;
-    }
-    for (int d = tid; d < ldd; d += kWaThreads) {
-        const int ch = kvh * a.dim + d;
-        s_k[d] = d < a.dim ? to_f(from_f<T>(conv_step(a.conv_k, ch, n_k, a.taps, tail + n_q + ch, n_ch, pk[ch]))) : 0.0f;
-    }
-    for (int d = tid; d < ldv; d += kWaThreads) {
-        const int ch = kvh * a.vdim + d;
-        s_v[d] = d < a.vdim ? to_f(from_f<T>(conv_step(a.conv_v, ch, n_v, a.taps, tail + n_q + n_k + ch, n_ch, pv[ch]))) : 0.0f;
+    for (int i = tid; i < (group + 1) * ldd + ldv; i += kWaThreads) {
+        // the convolved vectors as the storage type holds them; queries times the scale
+        float y = 0.0f;
+        if (i < group * ldd) {
+            const int g = i / ldd, d = i - g * ldd, ch = (kvh * group + g) * a.dim + d;
+            if (d < a.dim) y = to_f(from_f<T>(conv_step(a.conv_q, ch, n_q, a.taps, tail + ch, n_ch, pq[ch]))) * a.scale;
+        } else if (i < (group + 1) * ldd) {
+            const int d = i - group * ldd, ch = kvh * a.dim + d;
+            if (d < a.dim) y = to_f(from_f<T>(conv_step(a.conv_k, ch, n_k, a.taps, tail + n_q + ch, n_ch, pk[ch])));
+        } else {
+            const int d = i - (group + 1) * ldd, ch = kvh * a.vdim + d;
+            if (d < a.vdim) y = to_f(from_f<T>(conv_step(a.conv_v, ch, n_v, a.taps, tail + n_q + n_k + ch, n_ch, pv[ch])));
+        }
+        sm[i] = y;                                       // s_q, s_k and s_v lie back to back
     }
     __syncthreads();
 
@@ -80,9 +117,23 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
     T* ring_v = reinterpret_cast<T*>(a.ring_v) + (size_t)seq * a.ring_v_stride + (size_t)kvh * a.ring * ldv;
     const int first = max(0, pos - a.window + 1), n_keys = pos - first;      // cached keys; the new one comes on top
     const int per = (n_keys + n_rank - 1) / n_rank, j0 = min(n_keys, rank * per), j1 = min(n_keys, j0 + per);
+    const int slot0 = (first + j0) % a.ring;                                   // slot of this CTA's first key
     const int nvc = L.nvc, kpi = 32 / nvc, vc = lane & (nvc - 1), vk = lane / nvc;   // value chunk and key of this lane
+    const int kc = (lane & (LK - 1)) * 8, kg = lane / LK;                       // key piece and key of this lane
+    auto slot_of = [&](int j) { const int s = slot0 + j; return s >= a.ring ? s - a.ring : s; };
 
     for (int q0 = 0; q0 < group; q0 += GQ) {
+        float qf[GQ][8];
+#pragma unroll
+        for (int g = 0; g < GQ; ++g)
+#pragma unroll
+            for (int i = 0; i < 8; ++i) qf[g][i] = q0 + g < group && kc < ldd ? s_q[(q0 + g) * ldd + kc + i] : 0.0f;
+        int mine = 0;                                     // the query whose score this lane ends up with
+        {
+            float none[GQ] = {};
+            group_sums<GQ, LK>(none, lane, mine);
+        }
+        const float slope = head_slope(a, kvh * group + q0 + mine);
         float m[GQ], l[GQ], acc[GQ][8];
 #pragma unroll
         for (int g = 0; g < GQ; ++g) {
@@ -90,39 +141,35 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
 #pragma unroll
             for (int i = 0; i < 8; ++i) acc[g][i] = 0.0f;
         }
-        const bool has_new = rank == 0;
-        const int total = j1 - j0 + (has_new ? 1 : 0);   // key index total-1 of rank 0 is the new token
+        const int total = j1 - j0 + (rank == 0 ? 1 : 0), fresh = rank == 0 ? total - 1 : -1;   // rank 0 also takes the new token
         for (int sb = 0; sb < total; sb += kWaSeg) {
             const int ns = min(kWaSeg, total - sb);
-            // scores: eight lanes per key, 16 bytes of it per lane and step
-            for (int kk = warp * 4 + (lane >> 3); kk < ns; kk += kWaWarps * 4) {
-                const int j = sb + kk;
-                const bool fresh = has_new && j == total - 1;
-                const int p = fresh ? pos : first + j0 + j;
-                const T* krow = ring_k + (size_t)(p % a.ring) * ldd;
-                float s[GQ];
+            // scores. Every lane of a warp makes the same trips, so the exchanges are warp-wide.
+            for (int b = warp * KW; b < ns; b += kWaWarps * KW * KU) {
+                uint4 raw[KU][RAW];
 #pragma unroll
-                for (int g = 0; g < GQ; ++g) s[g] = 0.0f;
-                for (int c = (lane & 7) * 8; c < ldd; c += 64) {
-                    float kf[8];
-                    if (fresh) load8(s_k + c, kf); else load8(krow + c, kf);
-#pragma unroll
-                    for (int g = 0; g < GQ; ++g)
-                        if (q0 + g < group) {
-                            float qf[8];
-                            load8(s_q + (q0 + g) * ldd + c, qf);
-#pragma unroll
-                            for (int i = 0; i < 8; ++i) s[g] = fmaf(qf[i], kf[i], s[g]);
-                        }
+                for (int x = 0; x < KU; ++x) {
+                    const int kk = b + x * kWaWarps * KW + kg, j = sb + kk;
+                    if (kk < ns && j != fresh && kc < ldd) load_raw(ring_k + (size_t)slot_of(j) * ldd + kc, raw[x]);
                 }
-                const unsigned mask = 0xffu << (lane & 24);       // the eight lanes of this key
 #pragma unroll
-                for (int g = 0; g < GQ; ++g) {
-                    s[g] += __shfl_xor_sync(mask, s[g], 4);
-                    s[g] += __shfl_xor_sync(mask, s[g], 2);
-                    s[g] += __shfl_xor_sync(mask, s[g], 1);
-                    if ((lane & 7) == 0 && q0 + g < group)
-                        s_p[g * kWaSeg + kk] = s[g] - head_slope(a, kvh * group + q0 + g) * (float)(pos - p);
+                for (int x = 0; x < KU; ++x) {
+                    const int kk = b + x * kWaWarps * KW + kg, j = sb + kk;
+                    float s[GQ];
+#pragma unroll
+                    for (int g = 0; g < GQ; ++g) s[g] = 0.0f;
+                    if (kk < ns && kc < ldd) {
+                        float kf[8];
+                        if (j == fresh) load8(s_k + kc, kf); else raw_floats(raw[x], kf);
+#pragma unroll
+                        for (int g = 0; g < GQ; ++g)
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) s[g] = fmaf(qf[g][i], kf[i], s[g]);
+                    }
+                    int which;
+                    const float t = group_sums<GQ, LK>(s, lane, which);
+                    // distance to the new token, whose own is 0
+                    if (kk < ns && (lane & (LK / GQ - 1)) == 0) s_p[which * kWaSeg + kk] = t - slope * (float)(j == fresh ? 0 : n_keys - j0 - j);
                 }
             }
             __syncthreads();
@@ -153,21 +200,28 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
 #pragma unroll
                 for (int i = 0; i < 8; ++i) acc[g][i] *= f_old;
             }
-            for (int kk = warp * kpi + vk; kk < ns; kk += kWaWarps * kpi) {
-                const int j = sb + kk;
-                const bool fresh = has_new && j == total - 1;
-                const int p = fresh ? pos : first + j0 + j;
-                if (vc * 8 >= ldv) continue;
-                float vf[8];
-                if (fresh) load8(s_v + vc * 8, vf); else load8(ring_v + (size_t)(p % a.ring) * ldv + vc * 8, vf);
+            if (vc * 8 < ldv)
+                for (int b = warp * kpi + vk; b < ns; b += kWaWarps * kpi * VU) {
+                    uint4 raw[VU][RAW];
 #pragma unroll
-                for (int g = 0; g < GQ; ++g) {
-                    if (q0 + g >= group) continue;
-                    const float w = s_p[g * kWaSeg + kk] * f_new[g];
+                    for (int x = 0; x < VU; ++x) {
+                        const int kk = b + x * kWaWarps * kpi, j = sb + kk;
+                        if (kk < ns && j != fresh) load_raw(ring_v + (size_t)slot_of(j) * ldv + vc * 8, raw[x]);
+                    }
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) acc[g][i] = fmaf(w, vf[i], acc[g][i]);
+                    for (int x = 0; x < VU; ++x) {
+                        const int kk = b + x * kWaWarps * kpi, j = sb + kk;
+                        if (kk >= ns) continue;
+                        float vf[8];
+                        if (j == fresh) load8(s_v + vc * 8, vf); else raw_floats(raw[x], vf);
+#pragma unroll
+                        for (int g = 0; g < GQ; ++g) {
+                            const float w = q0 + g < group ? s_p[g * kWaSeg + kk] * f_new[g] : 0.0f;
+#pragma unroll
+                            for (int i = 0; i < 8; ++i) acc[g][i] = fmaf(w, vf[i], acc[g][i]);
+                        }
+                    }
                 }
-            }
             __syncthreads();
         }
         // value sums: across the key groups of a warp, then across warps
@@ -190,22 +244,21 @@ __global__ void __launch_bounds__(kWaThreads) window_decode_kernel(const WaDecod
             s_acc[i] = t;
         }
         cluster.sync();
-        if (rank == 0) {
-            T* out = reinterpret_cast<T*>(a.out) + (size_t)seq * a.ld_out;
-            for (int i = tid; i < GQ * ldv; i += kWaThreads) {
-                const int g = i / ldv, d = i - g * ldv;
-                if (q0 + g >= group || d >= a.vdim) continue;
-                float mx = a.sink > 0.0f ? 0.0f : -1e30f;     // the sink is a score of 0
-                for (int r = 0; r < n_rank; ++r) mx = fmaxf(mx, cluster.map_shared_rank(s_ml, r)[g]);
-                float den = a.sink * expf(-mx), num = 0.0f;
-                for (int r = 0; r < n_rank; ++r) {
-                    const float* ml = cluster.map_shared_rank(s_ml, r);
-                    const float f = expf(ml[g] - mx);
-                    den = fmaf(ml[GQ + g], f, den);
-                    num = fmaf(cluster.map_shared_rank(s_acc, r)[i], f, num);
-                }
-                out[(size_t)(kvh * group + q0 + g) * a.vdim + d] = from_f<T>(num / den);
+        // every CTA of the cluster finishes a slice of the outputs
+        T* out = reinterpret_cast<T*>(a.out) + (size_t)seq * a.ld_out;
+        for (int i = rank * kWaThreads + tid; i < GQ * ldv; i += n_rank * kWaThreads) {
+            const int g = i / ldv, d = i - g * ldv;
+            if (q0 + g >= group || d >= a.vdim) continue;
+            float mx = a.sink > 0.0f ? 0.0f : -1e30f;     // the sink is a score of 0
+            for (int r = 0; r < n_rank; ++r) mx = fmaxf(mx, cluster.map_shared_rank(s_ml, r)[g]);
+            float den = a.sink * expf(-mx), num = 0.0f;
+            for (int r = 0; r < n_rank; ++r) {
+                const float* ml = cluster.map_shared_rank(s_ml, r);
+                const float f = expf(ml[g] - mx);
+                den = fmaf(ml[GQ + g], f, den);
+                num = fmaf(cluster.map_shared_rank(s_acc, r)[i], f, num);
             }
+            out[(size_t)(kvh * group + q0 + g) * a.vdim + d] = from_f<T>(num / den);
         }
         cluster.sync();                                       // partials are read; the buffers may be reused
     }
@@ -229,74 +282,78 @@ struct WaChunkLaunch {
     int ldd, ldv, group, hist;
 };
 
-// Rows 0..hist-1 of lin_k / lin_v come from the ring, the M new rows from the convolution; queries get the storage type.
-// One CTA per row of the linear layout.
-template <typename T>
-__global__ void __launch_bounds__(256) window_prepare_kernel(const WaChunkLaunch L) {
+// Convolved rows in the storage type: queries to lin_q, keys and values behind the history in lin_k / lin_v. A thread owns
+// one channel of kPrepRows rows, with the convolution's inputs in registers. NT: taps rounded up to 4 or 16.
+constexpr int kPrepRows = 16, kPrepThreads = 128;
+
+template <typename T, int NT>
+__global__ void __launch_bounds__(kPrepThreads) window_prepare_kernel(const WaChunkLaunch L) {
     const WindowAttnArgs& a = L.a;
-    const int row = blockIdx.x, ldd = L.ldd, ldv = L.ldv, total = L.hist + a.M;
-    const int n_q = a.heads * a.dim, n_k = a.kv_heads * a.dim, n_v = a.kv_heads * a.vdim, n_ch = n_q + n_k + n_v;
-    T *lin_q = reinterpret_cast<T*>(a.lin_q), *lin_k = reinterpret_cast<T*>(a.lin_k), *lin_v = reinterpret_cast<T*>(a.lin_v);
-    if (row < L.hist) {
-        const int slot = (a.pos0 - L.hist + row) % a.ring;
-        for (int i = threadIdx.x; i < a.kv_heads * ldd; i += 256) {
-            const int h = i / ldd, d = i - h * ldd;
-            lin_k[((size_t)h * total + row) * ldd + d] = reinterpret_cast<const T*>(a.ring_k)[((size_t)h * a.ring + slot) * ldd + d];
-        }
-        for (int i = threadIdx.x; i < a.kv_heads * ldv; i += 256) {
-            const int h = i / ldv, d = i - h * ldv;
-            lin_v[((size_t)h * total + row) * ldv + d] = reinterpret_cast<const T*>(a.ring_v)[((size_t)h * a.ring + slot) * ldv + d];
-        }
-        return;
+    const int n_q = a.heads * a.dim, n_k = a.kv_heads * a.dim, n_v = a.kv_heads * a.vdim, n_ch = n_q + n_k + n_v, nt = a.taps - 1;
+    const int ch = blockIdx.x * kPrepThreads + threadIdx.x, t0 = blockIdx.y * kPrepRows, n_rows = min(kPrepRows, a.M - t0), total = L.hist + a.M;
+    if (ch >= n_ch) return;
+    const float *src, *w;
+    T* dst;                                                  // row t at dst + t * step
+    size_t step;
+    int local, nch, d, size, ld;
+    if (ch < n_q) {
+        local = ch; nch = n_q; size = a.dim; ld = L.ldd; src = a.q; w = a.conv_q;
+        dst = reinterpret_cast<T*>(a.lin_q) + (size_t)(local / size) * ld;
+        step = (size_t)a.heads * ld;
+    } else if (ch < n_q + n_k) {
+        local = ch - n_q; nch = n_k; size = a.dim; ld = L.ldd; src = a.k; w = a.conv_k;
+        dst = reinterpret_cast<T*>(a.lin_k) + ((size_t)(local / size) * total + L.hist) * ld;
+        step = ld;
+    } else {
+        local = ch - n_q - n_k; nch = n_v; size = a.vdim; ld = L.ldv; src = a.v; w = a.conv_v;
+        dst = reinterpret_cast<T*>(a.lin_v) + ((size_t)(local / size) * total + L.hist) * ld;
+        step = ld;
     }
-    const int t = row - L.hist, nt = a.taps - 1;
-    auto conv = [&](const float* src, const float* w, int nch, int ch, int tail_ch) {
+    d = local % size;
+    dst += d;
+    const int pad = d == size - 1 ? ld - size : 0;           // the last channel also zeroes the padding behind it
+    auto input = [&](int t) { return t >= 0 ? src[(size_t)t * a.ld + local] : t >= -nt ? a.tail_in[(size_t)(nt + t) * n_ch + ch] : 0.0f; };
+    float wt[NT], u[NT], in[kPrepRows];
+#pragma unroll
+    for (int j = 0; j < NT; ++j) {
+        wt[j] = j >= NT - a.taps ? w[(size_t)(j - NT + a.taps) * nch + local] : 0.0f;
+        u[j] = j > NT - a.taps ? input(t0 - NT + j) : 0.0f;
+    }
+#pragma unroll
+    for (int i = 0; i < kPrepRows; ++i) in[i] = i < n_rows ? input(t0 + i) : 0.0f;
+#pragma unroll
+    for (int i = 0; i < kPrepRows; ++i) {
+        if (i >= n_rows) break;
+#pragma unroll
+        for (int j = 0; j + 1 < NT; ++j) u[j] = u[j + 1];
+        u[NT - 1] = in[i];
         float y = 0.0f;
-        for (int j = 0; j < a.taps; ++j) {
-            const int u = t - nt + j;
-            const float v = u >= 0 ? src[(size_t)u * a.ld + ch] : a.tail_in[(size_t)(nt + u) * n_ch + tail_ch];
-            y = fmaf(w[(size_t)j * nch + ch], v, y);
-        }
-        return y;
-    };
-    for (int i = threadIdx.x; i < a.heads * ldd; i += 256) {
-        const int h = i / ldd, d = i - h * ldd, ch = h * a.dim + d;
-        lin_q[((size_t)t * a.heads + h) * ldd + d] = from_f<T>(d < a.dim ? conv(a.q, a.conv_q, n_q, ch, ch) : 0.0f);
+#pragma unroll
+        for (int j = 0; j < NT; ++j) y = fmaf(wt[j], u[j], y);
+        T* o = dst + (size_t)(t0 + i) * step;
+        o[0] = from_f<T>(y);
+        for (int k = 1; k <= pad; ++k) o[k] = from_f<T>(0.0f);
     }
-    for (int i = threadIdx.x; i < a.kv_heads * ldd; i += 256) {
-        const int h = i / ldd, d = i - h * ldd, ch = h * a.dim + d;
-        lin_k[((size_t)h * total + row) * ldd + d] = from_f<T>(d < a.dim ? conv(a.k, a.conv_k, n_k, ch, n_q + ch) : 0.0f);
-    }
-    for (int i = threadIdx.x; i < a.kv_heads * ldv; i += 256) {
-        const int h = i / ldv, d = i - h * ldv, ch = h * a.vdim + d;
-        lin_v[((size_t)h * total + row) * ldv + d] = from_f<T>(d < a.vdim ? conv(a.v, a.conv_v, n_v, ch, n_q + n_k + ch) : 0.0f);
-    }
-    if (t == a.M - 1)
-        for (int j = 0; j < nt; ++j) {
-            const int u = a.M - nt + j;
-            for (int ch = threadIdx.x; ch < n_ch; ch += 256) {
-                float v;
-                if (u < 0) v = a.tail_in[(size_t)(nt + u) * n_ch + ch];
-                else if (ch < n_q) v = a.q[(size_t)u * a.ld + ch];
-                else if (ch < n_q + n_k) v = a.k[(size_t)u * a.ld + ch - n_q];
-                else v = a.v[(size_t)u * a.ld + ch - n_q - n_k];
-                a.tail_out[(size_t)j * n_ch + ch] = v;
-            }
-        }
+    if (t0 + n_rows == a.M)
+        for (int j = 0; j < nt; ++j) a.tail_out[(size_t)j * n_ch + ch] = input(a.M - nt + j);
 }
 
-// The last min(M, ring) new rows go into the ring. One CTA per row.
-template <typename T>
+// Rows between the ring and the linear layout, 16 bytes per thread: TO_RING = 0 brings the history in front of the new rows,
+// TO_RING = 1 puts the last `rows` of them into the ring (a separate launch: the history is read first).
+template <typename T, bool TO_RING>
 __global__ void __launch_bounds__(256) window_ring_kernel(const WaChunkLaunch L, int rows) {
     const WindowAttnArgs& a = L.a;
-    const int t = a.M - rows + blockIdx.x, total = L.hist + a.M, slot = (a.pos0 + t) % a.ring, ldd = L.ldd, ldv = L.ldv;
-    for (int i = threadIdx.x; i < a.kv_heads * ldd; i += 256) {
-        const int h = i / ldd, d = i - h * ldd;
-        reinterpret_cast<T*>(a.ring_k)[((size_t)h * a.ring + slot) * ldd + d] = reinterpret_cast<const T*>(a.lin_k)[((size_t)h * total + L.hist + t) * ldd + d];
-    }
-    for (int i = threadIdx.x; i < a.kv_heads * ldv; i += 256) {
-        const int h = i / ldv, d = i - h * ldv;
-        reinterpret_cast<T*>(a.ring_v)[((size_t)h * a.ring + slot) * ldv + d] = reinterpret_cast<const T*>(a.lin_v)[((size_t)h * total + L.hist + t) * ldv + d];
+    constexpr int E = 16 / sizeof(T);
+    const int row = blockIdx.x, total = L.hist + a.M;
+    const int lin = TO_RING ? total - rows + row : row, slot = (a.pos0 - L.hist + lin) % a.ring;
+    const int kc = L.ldd / E, vc = L.ldv / E;
+    for (int i = threadIdx.x; i < a.kv_heads * (kc + vc); i += 256) {
+        const bool is_k = i < a.kv_heads * kc;
+        const int n = is_k ? kc : vc, x = is_k ? i : i - a.kv_heads * kc, h = x / n, c = x - h * n, ld = n * E;
+        T* l = reinterpret_cast<T*>(is_k ? a.lin_k : a.lin_v) + ((size_t)h * total + lin) * ld;
+        T* r = reinterpret_cast<T*>(is_k ? a.ring_k : a.ring_v) + ((size_t)h * a.ring + slot) * ld;
+        if (TO_RING) reinterpret_cast<uint4*>(r)[c] = reinterpret_cast<const uint4*>(l)[c];
+        else reinterpret_cast<uint4*>(l)[c] = reinterpret_cast<const uint4*>(r)[c];
     }
 }
 
@@ -366,28 +423,31 @@ static int window_attention(const WindowAttnArgs& a, cudaStream_t st, unsigned l
         L.a = a; L.ldd = ldd; L.ldv = ldv; L.group = group;
         L.nvc = 1;
         while (L.nvc * 8 < ldv) L.nvc *= 2;
-        // slices of about 256 keys, at most eight CTAs
+        // slices of at least 64 keys, at most eight CTAs, more than one only while the grid is small
         int cl = 1;
-        while (cl < 8 && a.ring > 256 * cl) cl *= 2;
+        while (cl < 8 && a.ring > 128 * cl && (long long)cl * a.kv_heads * a.M < 4 * 148) cl *= 2;
         auto go = [&](auto kernel, int GQ) {
-            const size_t smem = 4 * ((size_t)group * ldd + ldd + ldv + GQ * kWaSeg + (size_t)kWaWarps * GQ * ldv + 2 * GQ + 32);
+            const size_t smem = 4 * ((size_t)group * ldd + ldd + ldv + GQ * kWaSeg + (size_t)kWaWarps * GQ * ldv + 2 * GQ);
             if (smem > 220 * 1024) return -1;
             if (int rc = allow_smem(kernel, smem)) return rc;
             return launch_kernel(kernel, dim3(cl, a.kv_heads, a.M), dim3(kWaThreads), smem, st, a.use_pdl, cl, L);
         };
         *n_kernels += 1;
-        if (group == 1) return go(window_decode_kernel<T, 1>, 1);
-        if (group == 2) return go(window_decode_kernel<T, 2>, 2);
-        if (group <= 4) return go(window_decode_kernel<T, 4>, 4);
-        return go(window_decode_kernel<T, 8>, 8);
+        auto heads_at_once = [&](auto one, auto two, auto four) { return group == 1 ? go(one, 1) : group == 2 ? go(two, 2) : go(four, 4); };
+        if (ldd > 128) return heads_at_once(window_decode_kernel<T, 1, 32>, window_decode_kernel<T, 2, 32>, window_decode_kernel<T, 4, 32>);
+        if (ldd > 64) return heads_at_once(window_decode_kernel<T, 1, 16>, window_decode_kernel<T, 2, 16>, window_decode_kernel<T, 4, 16>);
+        return heads_at_once(window_decode_kernel<T, 1, 8>, window_decode_kernel<T, 2, 8>, window_decode_kernel<T, 4, 8>);
     }
     WaChunkLaunch L;
     L.a = a; L.ldd = ldd; L.ldv = ldv; L.group = group;
     L.hist = a.pos0 < a.window - 1 ? a.pos0 : a.window - 1;
-    window_prepare_kernel<T><<<L.hist + a.M, 256, 0, st>>>(L);
+    const dim3 grid((a.heads * a.dim + a.kv_heads * (a.dim + a.vdim) + kPrepThreads - 1) / kPrepThreads, (a.M + kPrepRows - 1) / kPrepRows);
+    if (a.taps <= 4) window_prepare_kernel<T, 4><<<grid, kPrepThreads, 0, st>>>(L);
+    else window_prepare_kernel<T, kMaxTaps><<<grid, kPrepThreads, 0, st>>>(L);
+    if (L.hist > 0) window_ring_kernel<T, false><<<L.hist, 256, 0, st>>>(L, L.hist);
     const int rows = a.M < a.ring ? a.M : a.ring;
-    window_ring_kernel<T><<<rows, 256, 0, st>>>(L, rows);
-    *n_kernels += 3;
+    window_ring_kernel<T, true><<<rows, 256, 0, st>>>(L, rows);
+    *n_kernels += L.hist > 0 ? 4 : 3;
     if (!a.f32 && window_flash_applicable(a)) return launch_window_flash(a, L.hist, st);
     const size_t smem = 4 * ((size_t)32 * (ldd + 1) + 32 * ldv + kWaQ * ldd);
     if (int rc = allow_smem(window_chunk_kernel<T>, smem)) return rc;

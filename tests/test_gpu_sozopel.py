@@ -102,7 +102,7 @@ def test_rows(width, taps, mixes, cuts):
         kernels.rows(x_in=dev(x[sl]), y0=dev(y0[sl]), y1=dev(y1[sl]), w0=dev(w0), w1=dev(w1), ld_y=width, x_out=x_out, width=width, M=n, eps=eps,
                      gain=1.7, conv_w=dev(cw.T.copy()), taps=taps, tail_in=state, tail_out=stage, mu=dev(mu) if mixes else None, n_mix=mixes,
                      prev_in=state[(taps - 1) * width:], prev_out=stage[(taps - 1) * width:], seq_stride=0, decode=int(n == 1), out=out,
-                     ld_out=width, f32=1)
+                     ld_out=width, row_inv=torch.empty(n, device="cuda"), f32=1)
         torch.cuda.synchronize()
         state = stage
         got[:, sl], got_x[sl] = host(out), host(x_out)
@@ -227,7 +227,7 @@ def test_linear_scan(kind, bonus, norm, heads, dim, vdim):
     o = o * gain.reshape(1, -1, vdim) if norm else o
     want = o.reshape(T, nv) * ora.silu(g)
     ldv = (vdim + 3) // 4 * 4
-    fixed = dict(ld=x.shape[1], q_scale=0.5, k_scale=0.7, heads=heads, dim=dim, vdim=vdim, decay_kind=kind, decay=dev(decay_h), up=dev(up, torch.bfloat16),
+    fixed = dict(ld=x.shape[1], q_scale=0.5, k_scale=0.7, heads=heads, dim=dim, vdim=vdim, decay_kind=kind, decay=dev(decay_h), up=dev(np.pad(up, ((0, 0), (0, -rank % 8))), torch.bfloat16),
                  bias=dev(bias), rank=rank, tau=tau, bonus=dev(u) if bonus else None, norm=dev(gain) if norm else None, norm_per_head=int(norm == "head"),
                  eps=eps, ld_out=nv, f32=1)
     for cuts in ([T], [1] * 30 + [2, 118], [64, 2, 3, 1, 70, 10]):
@@ -495,3 +495,12 @@ def test_trace_replay(model, compute, tmp_path):
     close(read(2), want[[52]], compute)
     close(read(3), want[[3]], compute)
     assert not (tmp_path / "1.f32").exists()
+
+
+def test_command_line_generates(model):
+    folder, cfg, W, tokens, _ = model("mixed")
+    prompt = tokens[:9].tolist()
+    r = subprocess.run([sys.executable, "-m", "tenzo_b200", "generate", "--model", str(folder), "--dtype", "float32", "--n", "6", "--tokens",
+                        ",".join(map(str, prompt))], capture_output=True, text=True, timeout=300, cwd=ROOT)
+    assert r.returncode == 0, r.stderr
+    assert [int(t) for t in r.stdout.split()] == ora.greedy(cfg, W, prompt, 6)
