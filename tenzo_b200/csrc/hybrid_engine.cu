@@ -347,17 +347,16 @@ void HybridEngine::run_rows(Pass& p, RowsArgs& a) {
     TZ_KERNEL(launch_rows(a, stream, &launches));
 }
 
-void HybridEngine::run_gemm(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c, int epilogue, const HybridLayer* y) {
+void HybridEngine::run_gemm(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c, const HybridLayer* mixes, const HybridLayer* act) {
     GemmArgs g;
     g.a = a; g.w = w.w; g.M = p.M; g.N = w.rows; g.ld_k = w.ld_k;
     g.seg_end[0] = w.rows;
-    if (y && y->n_mix) {
-        g.n_seg = y->n_seg;
-        std::copy(y->seg_end, y->seg_end + 8, g.seg_end);
+    if (mixes) {
+        g.n_seg = mixes->n_seg;
+        std::copy(mixes->seg_end, mixes->seg_end + 8, g.seg_end);
         g.a_seg_stride = (size_t)p.M * w.ld_k;
     }
-    g.epilogue = epilogue;
-    if (epilogue == TENZO_GEMM_XIELU) { g.act_pos = y->act_pos; g.act_neg = y->act_neg; }
+    if (act) { g.epilogue = TENZO_GEMM_XIELU; g.act_pos = act->act_pos; g.act_neg = act->act_neg; }
     g.c = c; g.ld_c = ld_c;
     g.f32 = f32; g.use_pdl = p.decode && use_pdl;
     g.workspace = gemm_ws; g.workspace_bytes = tenzo_cuda_gemm_workspace_bytes();
@@ -376,7 +375,7 @@ void HybridEngine::run_layer(Pass& p, int l) {
         ra.prev_out = p.decode ? carried : tail_stage + y.prev;
     }
     run_rows(p, ra);
-    run_gemm(p, r.in, y.in, r.proj, max_proj, TENZO_GEMM_STORE, y.n_mix ? &y : nullptr);
+    run_gemm(p, r.in, y.in, r.proj, max_proj, y.n_mix ? &y : nullptr);
 
     if (y.has_window) {
         const WindowMixer& m = y.win;
@@ -418,18 +417,18 @@ void HybridEngine::run_layer(Pass& p, int l) {
         TZ_KERNEL(launch_scan(a, stream, &launches));
     }
     if (y.has_window && y.has_scan) {
-        run_gemm(p, r.mix_a, y.win.o, r.ya, h, TENZO_GEMM_STORE, nullptr);
-        run_gemm(p, r.mix_b, y.scan.o, r.yb, h, TENZO_GEMM_STORE, nullptr);
+        run_gemm(p, r.mix_a, y.win.o, r.ya, h);
+        run_gemm(p, r.mix_b, y.scan.o, r.yb, h);
         p.add.y0 = r.ya; p.add.y1 = r.yb; p.add.w0 = y.left_out; p.add.w1 = y.right_out;
     } else {
-        run_gemm(p, r.mix_a, y.has_window ? y.win.o : y.scan.o, r.ya, h, TENZO_GEMM_STORE, nullptr);
+        run_gemm(p, r.mix_a, y.has_window ? y.win.o : y.scan.o, r.ya, h);
         p.add.y0 = r.ya;
     }
     if (y.has_mlp) {
         RowsArgs rb = row_args(p, y.norm2, y.canon2, y.tail2);
         run_rows(p, rb);
-        run_gemm(p, r.in, y.up, r.act, y.down.ld_k, TENZO_GEMM_XIELU, &y);
-        run_gemm(p, r.act, y.down, r.ya, h, TENZO_GEMM_STORE, nullptr);
+        run_gemm(p, r.in, y.up, r.act, y.down.ld_k, nullptr, &y);
+        run_gemm(p, r.act, y.down, r.ya, h);
         p.add.y0 = r.ya;
     }
 }
@@ -440,7 +439,7 @@ void HybridEngine::enqueue_step(bool with_logits, bool feed_back, int) {
     RowsArgs ra = row_args(p, final_gain, nullptr, 0);
     run_rows(p, ra);
     if (with_logits) {
-        run_gemm(p, dec.in, head, b_logits, V, TENZO_GEMM_STORE, nullptr);
+        run_gemm(p, dec.in, head, b_logits, V);
         TZ_KERNEL(launch_argmax(b_logits, V, batch, d_next, argmax_ws, stream));
         launches += 2;
     }
@@ -526,7 +525,7 @@ void HybridEngine::rows_logits(const int* want, int n_want, float* host) {
             i = j;
         }
         Pass p = {&chunk, n, 0, 0, 0, nullptr, nullptr};
-        run_gemm(p, logit_in, head, want_logits, V, TENZO_GEMM_STORE, nullptr);
+        run_gemm(p, logit_in, head, want_logits, V);
         TZ_CUDA(cudaMemcpyAsync(host + (size_t)a * V, want_logits, (size_t)n * V * 4, cudaMemcpyDeviceToHost, stream));
     }
     TZ_CUDA(cudaStreamSynchronize(stream));

@@ -101,7 +101,7 @@ private:
     void free_rows(Rows& r);
     RowsArgs row_args(Pass& p, float gain, const float* conv, size_t tail);
     void run_rows(Pass& p, RowsArgs& a);
-    void run_gemm(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c, int epilogue, const HybridLayer* seg);
+    void run_gemm(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c, const HybridLayer* mixes = nullptr, const HybridLayer* act = nullptr);
     void run_layer(Pass& p, int l);
     void upload_weight(DenseWeight& d, int row0, const SafeTensors& st, const std::string& name, int rows, int k);
     DenseWeight make_weight(int rows, int k);

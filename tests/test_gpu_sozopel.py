@@ -267,7 +267,7 @@ def config(layers, width=96, vocab=210, taps=4, eps=1e-5, n_pos=600):
 MODELS = {
     "attention_beside_gla": (config([parallel(4, 2, 24, 32, 3, 19, 3, 20, 28, 8.0, 130)]), 7),
     "retention": (config([retention(3, 20, 44), retention(2, 32, 16, ff=72)], width=80), 4),
-    "time_mixing": (config([wkv(3, 24), wkv(2, 48, ff=100)], width=72, taps=3), 12),
+    "time_mixing": (config([wkv(3, 24), wkv(2, 48, ff=333), wkv(1, 20, ff=140)], width=72, taps=3), 12),
     "mixed": (config([wkv(4, 16, ff=96), parallel(6, 3, 16, 48, 2, 31, 2, 40, 24, 20.0, None), retention(2, 24, 40), parallel(5, 1, 32, 16, 4, 70, 1, 16, 64, 5.0, 200)],
                      width=120, vocab=301, taps=2, eps=1e-3), 9),
     "no_reach_back": (config([parallel(2, 2, 16, 16, 1, 1, 2, 16, 16, 1.0, 64), wkv(1, 40), retention(1, 12, 20)], width=64, taps=1), 1),
