@@ -236,18 +236,22 @@ TENZO_API int tenzo_cuda_tl1_pack_rows2bit(const uint8_t* raw, int N, int K, uin
  * consecutive rows of one sequence; carried convolution inputs are read from *_in and their successors written to *_out,
  * a different buffer, because rows of the same launch still need the old ones. */
 
-/* Row kernel: x = source; x_out = x; u = x / sqrt(mean(x^2) + eps) * gain; y = u + conv(u); out = y, or with mu the mixes
- * out_s = y + (y of the row before - y) * mu_s. */
+/* Row kernel: x = source; x_out = x; u = x / sqrt(mean(x^2) + eps) * gain (* gain_w); y = u + conv(u); out = y, or with mu
+ * the mixes out_s = y + (y of the row before - y) * mu_s. */
 typedef struct {
-    const int *tokens, *pos;          /* not NULL: x = embed[token] + pos_table[pos] */
-    const void *embed, *pos_table;    /* bf16 [vocab][width], [n_pos][width] */
+    const int *tokens, *pos;          /* tokens not NULL: x = embed[token] (+ pos_table[pos]) */
+    const void *embed, *pos_table;    /* bf16 [vocab][width], [n_pos][width] or NULL */
     int vocab, n_pos;
-    const float *x_in;                /* otherwise x = x_in (+ y0) (+ 0.5 (y0 / rms(y0) * w0 + y1 / rms(y1) * w1) when y1) */
-    const float *y0, *y1, *w0, *w1;
+    const float *x_in;                /* otherwise x = x_in (+ y0), with w0 x_in + y0 / rms(y0) * w0, and with y1 the mean of the two */
+    const float *y0, *y1, *w0, *w1;   /* normed addends: x_in + 0.5 (y0 / rms(y0) * w0 + y1 / rms(y1) * w1) */
     int ld_y;
+    const int* y_slot;                /* [M][n_y] or NULL: y0 of row m is sum_j y_weight[m][j] * (row y_slot[m][j] of y0) */
+    const float* y_weight;
+    int n_y;
     float* x_out;                     /* [M][width] */
     int width, M;
     float eps, gain;
+    const float* gain_w;              /* [width] or NULL */
     const float* conv_w;              /* [taps][width]; NULL: no convolution */
     int taps;                         /* 1..16 */
     const float* tail_in;             /* [taps-1][width] per sequence: u of the tokens before, oldest first */
@@ -266,18 +270,29 @@ typedef struct {
 TENZO_API int tenzo_cuda_rows(const tenzo_rows_args* args, void* stream);
 
 /* c[m][n] = sum_k a[m][k] w[n][k]: a GEMV up to 8 rows, tcgen05 from 16 (bf16), tiled FMA for fp32. Rows of w in segment s
- * (n < seg_end[s]) multiply the matrix at a + s * a_seg_stride; on tcgen05 segments end at multiples of 128. */
-enum { TENZO_GEMM_STORE = 0, TENZO_GEMM_XIELU = 1 };
+ * (n < seg_end[s], or n / seg_rows == s) multiply the matrix at a + s * a_seg_stride; on tcgen05 segments end at multiples
+ * of 128.
+ * Grouped form (group_off): w holds n_group matrices [N][ld_k] back to back, and matrix g multiplies the rows
+ * group_off[g] .. group_off[g+1] - 1; M bounds group_off[n_group]. */
+enum { TENZO_GEMM_STORE = 0, TENZO_GEMM_XIELU = 1, TENZO_GEMM_GLU_RELU = 2, TENZO_GEMM_GLU_SILU = 3, TENZO_GEMM_CAST = 4, TENZO_GEMM_SOFTCAP = 5 };
 typedef struct {
     const void* a;                    /* storage type, rows of ld_k elements, padding finite */
     const void* w;                    /* bf16 [N][ld_k], padding zero; ld_k a multiple of 64 */
     int M, N, ld_k;
     int n_seg, seg_end[8];
     size_t a_seg_stride;              /* elements, a multiple of ld_k */
-    int epilogue;                     /* XIELU: z > 0: act_pos z^2 + z/2, else act_neg (exp(z) - 1 - z) + z/2 */
-    float act_pos, act_neg;
-    void* c;                          /* STORE: float [M][ld_c]; XIELU: storage type */
+    int seg_rows;                     /* > 0: N / seg_rows segments of equal size instead of seg_end */
+    int epilogue;                     /* XIELU: z > 0: act_pos z^2 + z/2, else act_neg (exp(z) - 1 - z) + z/2;
+                                         GLU: w rows 2i and 2i+1 are gate and up, column i of c is act(gate) * up;
+                                         CAST: c in the storage type; SOFTCAP: cap * tanh(z / cap) */
+    float act_pos, act_neg, cap;
+    void* c;                          /* STORE, SOFTCAP: float [M][ld_c]; others: storage type */
     int ld_c;
+    const int* group_off;             /* device [n_group + 1] or NULL */
+    int n_group;
+    const int* a_index;               /* device [M] or NULL: row m reads row a_index[m] of a (of a_rows); grouped form only */
+    int a_rows;
+    void* a_gather;                   /* [M][ld_k] scratch for a_index on tcgen05 */
     int f32, use_pdl;
     void* workspace;                  /* tenzo_cuda_gemm_workspace_bytes(), zeroed once; NULL keeps off the tensor cores */
     size_t workspace_bytes;
@@ -341,6 +356,84 @@ typedef struct {
 } tenzo_scan_args;
 TENZO_API int tenzo_cuda_linear_scan(const tenzo_scan_args* args, void* stream);
 TENZO_API size_t tenzo_cuda_linear_scan_part_floats(int M, int heads, int dim, int vdim);
+
+/* Gated delta rule. q, k, v pass a causal convolution of `taps` per channel and silu; q and k become unit vectors
+ * (x / sqrt(sum(x^2) + unit_eps)), q times q_scale; head h uses q/k head h / (heads / kv_heads). With
+ * g = exp(-exp(a_log) ln(1 + e^(a + dt_bias))) and beta = sigmoid(b): S' = g S_(t-1); u = beta (v - S'^T k); S_t = S' + k u^T;
+ * o = S_t^T q; out = o / sqrt(mean over the head(o^2) + eps) * norm * silu(g). */
+typedef struct {
+    const float *q, *k, *v, *g, *a, *b;   /* row stride ld; a and b: one value per head */
+    int ld;
+    const float *conv_q, *conv_k, *conv_v;   /* [taps][channels] */
+    int taps;                             /* 1..16 */
+    float* tail;                          /* [taps][q|k|v channels] per sequence: row p % taps is the input of position p, zero at the start */
+    size_t tail_seq_stride;
+    int heads, kv_heads, dim, vdim;       /* head sizes up to 256 */
+    float q_scale, unit_eps;
+    const float *a_log, *dt_bias;         /* [heads] */
+    const float* norm;                    /* [vdim] */
+    float eps;
+    float* state;                         /* [heads][dim][vdim rounded up to 4] per sequence */
+    size_t state_seq_stride;              /* a multiple of 4 */
+    const int* pos;                       /* decode: position of every row (device) */
+    int pos0;                             /* chunk: position of the first row */
+    int M, decode;
+    void* out;                            /* storage type [M][ld_out] */
+    int ld_out;
+    float* work;                          /* chunk: tenzo_cuda_delta_rule_work_floats(), 16-byte aligned */
+    int f32, use_pdl;
+} tenzo_delta_args;
+TENZO_API int tenzo_cuda_delta_rule(const tenzo_delta_args* args, void* stream);
+TENZO_API size_t tenzo_cuda_delta_rule_work_floats(int M, int heads, int kv_heads, int dim, int vdim);
+
+/* Causal sliding-window attention over a latent shared by all heads. A token's cache row is c = dkv[0..rank) / rms * norm and
+ * r = dkv[rank..rank+rot) rotated; head h's key is (W_uk,h c, r), its value W_uv,h c, its query q_h with the last `rot`
+ * elements rotated; score = scale * query.key. Rotation: elements i and i + rot/2 by position * freq[i].
+ * dim8, rot8, vdim8: sizes rounded up to 8; ld_c: rank rounded up to 64. */
+typedef struct {
+    const float *q, *dkv;                 /* row stride ld: [heads][dim + rot], [rank + rot]; dkv NULL: another layer's call put the */
+    int ld;                               /* rows of these tokens into the rings (and lin_c, lin_r) already */
+    const float* norm;                    /* [rank] */
+    float eps;
+    const double* freq;                   /* device [rot/2] */
+    int heads, dim, rot, vdim, rank;      /* head sizes up to 256, rank up to 1024 */
+    float scale;
+    int window;
+    const void* w_kv;                     /* bf16 [heads * dim8 key rows, then heads * vdim8 value rows][ld_c], padding zero */
+    void *ring_c, *ring_r;                /* storage type [ring][ld_c], [ring][rot8] per sequence, padding zero */
+    int ring;                             /* >= min(window, longest sequence): slot = position % ring */
+    size_t ring_c_stride, ring_r_stride;  /* elements between two sequences */
+    const int* pos;                       /* decode: position of every row (device) */
+    int pos0;                             /* chunk: position of the first row */
+    int M, decode;
+    void* out;                            /* storage type [M][ld_out], head h at h * vdim8 */
+    int ld_out;
+    void *lin_q, *lin_c, *lin_r, *kv;     /* chunk scratch, storage type: [M][heads][dim8 + rot8], [min(pos0, ring-1) + M][ld_c], [..][rot8], */
+                                          /* [min(pos0, window-1) + M][heads * (dim8 + vdim8)] */
+    float* q_abs;                         /* decode scratch: [M][heads][ld_c] */
+    void* lat;                            /* decode scratch, storage type: [heads][M][ld_c] */
+    void* workspace;                      /* of the matrix products, as in tenzo_gemm_args */
+    size_t workspace_bytes;
+    int f32, use_pdl;
+} tenzo_latent_attention_args;
+TENZO_API int tenzo_cuda_latent_attention(const tenzo_latent_attention_args* args, void* stream);
+
+/* Choice of experts: s = sigmoid(logits); the `top` largest s + correction of a row are chosen, weight = s. The pairs
+ * (row, choice) get places in order of their expert, rows ascending: the grouped form of tenzo_cuda_gemm takes group_off
+ * and row_of (its a_index), tenzo_cuda_rows adds the results back by slot and weight. */
+typedef struct {
+    const float* logits;                  /* row stride ld */
+    int ld;
+    const float* correction;              /* [experts] or NULL */
+    int experts, top, M;
+    int* chosen;                          /* [M][top] experts, best first */
+    float* weight;                        /* [M][top] */
+    int* slot;                            /* [M][top] place of the pair */
+    int* row_of;                          /* [M * top] row of the pair at a place */
+    int* group_off;                       /* [experts + 1] first place of every expert */
+    int use_pdl;
+} tenzo_route_args;
+TENZO_API int tenzo_cuda_route(const tenzo_route_args* args, void* stream);
 
 #ifdef __cplusplus
 }

@@ -77,13 +77,13 @@ def _fields(spec: str):
 
 
 class RowsArgs(C.Structure):
-    _fields_ = _fields("tokens:p pos:p embed:p pos_table:p vocab:i n_pos:i x_in:p y0:p y1:p w0:p w1:p ld_y:i x_out:p width:i M:i eps:f gain:f "
+    _fields_ = _fields("tokens:p pos:p embed:p pos_table:p vocab:i n_pos:i x_in:p y0:p y1:p w0:p w1:p ld_y:i y_slot:p y_weight:p n_y:i x_out:p width:i M:i eps:f gain:f gain_w:p "
                        "conv_w:p taps:i tail_in:p tail_out:p mu:p n_mix:i prev_in:p prev_out:p seq_stride:z decode:i out:p ld_out:i row_inv:p f32:i use_pdl:i")
 
 
 class GemmArgs(C.Structure):
-    _fields_ = _fields("a:p w:p M:i N:i ld_k:i n_seg:i seg_end:i8 a_seg_stride:z epilogue:i act_pos:f act_neg:f c:p ld_c:i f32:i use_pdl:i "
-                       "workspace:p workspace_bytes:z")
+    _fields_ = _fields("a:p w:p M:i N:i ld_k:i n_seg:i seg_end:i8 a_seg_stride:z seg_rows:i epilogue:i act_pos:f act_neg:f cap:f c:p ld_c:i "
+                       "group_off:p n_group:i a_index:p a_rows:i a_gather:p f32:i use_pdl:i workspace:p workspace_bytes:z")
 
 
 class WindowAttentionArgs(C.Structure):
@@ -96,6 +96,27 @@ class ScanArgs(C.Structure):
     _fields_ = _fields("q:p k:p v:p g:p ld:i q_scale:f k_scale:f heads:i dim:i vdim:i decay_kind:i decay:p low:p up:p bias:p rank:i tau:f "
                        "bonus:p norm:p norm_per_head:i eps:f state:p state_seq_stride:z M:i decode:i out:p ld_out:i w_rows:p o_rows:p part:p "
                        "f32:i use_pdl:i")
+
+
+class DeltaArgs(C.Structure):
+    _fields_ = _fields("q:p k:p v:p g:p a:p b:p ld:i conv_q:p conv_k:p conv_v:p taps:i tail:p tail_seq_stride:z heads:i kv_heads:i dim:i vdim:i "
+                       "q_scale:f unit_eps:f a_log:p dt_bias:p norm:p eps:f state:p state_seq_stride:z pos:p pos0:i M:i decode:i out:p ld_out:i "
+                       "work:p f32:i use_pdl:i")
+
+
+class LatentAttentionArgs(C.Structure):
+    _fields_ = _fields("q:p dkv:p ld:i norm:p eps:f freq:p heads:i dim:i rot:i vdim:i rank:i scale:f window:i w_kv:p ring_c:p ring_r:p ring:i "
+                       "ring_c_stride:z ring_r_stride:z pos:p pos0:i M:i decode:i out:p ld_out:i lin_q:p lin_c:p lin_r:p kv:p q_abs:p lat:p "
+                       "workspace:p workspace_bytes:z f32:i use_pdl:i")
+
+
+class RouteArgs(C.Structure):
+    _fields_ = _fields("logits:p ld:i correction:p experts:i top:i M:i chosen:p weight:p slot:p row_of:p group_off:p use_pdl:i")
+
+
+# flat calls that take one struct: name -> struct
+STRUCT_CALLS = {"rows": RowsArgs, "gemm": GemmArgs, "window_attention": WindowAttentionArgs, "linear_scan": ScanArgs, "delta_rule": DeltaArgs,
+                "latent_attention": LatentAttentionArgs, "route": RouteArgs}
 
 
 ENGINE_SYMBOLS = [
@@ -120,6 +141,7 @@ KERNEL_SYMBOLS = [
     "tenzo_cuda_lm_head_static_max_batch", "tenzo_cuda_lm_head_take_timeouts", "tenzo_cuda_repetition_penalty",
     "tenzo_cuda_topk_candidates", "tenzo_cuda_topk_max_candidates", "tenzo_cuda_rows", "tenzo_cuda_gemm", "tenzo_cuda_gemm_workspace_bytes",
     "tenzo_cuda_gemm_take_timeouts", "tenzo_cuda_window_attention", "tenzo_cuda_linear_scan", "tenzo_cuda_linear_scan_part_floats",
+    "tenzo_cuda_delta_rule", "tenzo_cuda_delta_rule_work_floats", "tenzo_cuda_latent_attention", "tenzo_cuda_route",
 ]
 HAL_SYMBOLS = ["tenzo_hal_initialize", "tenzo_hal_bitlinear_tl1_host", "tenzo_hal_rmsnorm_host", "tenzo_hal_gemm_f32_host", "tenzo_hal_call_count"]
 
@@ -224,12 +246,13 @@ def declare_kernel_abi(L):
     L.tenzo_cuda_lm_head_scratch_bytes.restype, L.tenzo_cuda_lm_head_scratch_bytes.argtypes = sz, [i32]
     L.tenzo_cuda_embedding_i8.restype, L.tenzo_cuda_embedding_i8.argtypes = i32, [vp, vp, i32, vp, i32, vp, i32, i32, vp]
     L.tenzo_cuda_tl1_pack_rows2bit.restype, L.tenzo_cuda_tl1_pack_rows2bit.argtypes = i32, [vp, i32, i32, vp, vp]
-    for name, args in (("rows", RowsArgs), ("gemm", GemmArgs), ("window_attention", WindowAttentionArgs), ("linear_scan", ScanArgs)):
+    for name, args in STRUCT_CALLS.items():
         fn = getattr(L, "tenzo_cuda_" + name)
         fn.restype, fn.argtypes = i32, [C.POINTER(args), vp]
     L.tenzo_cuda_gemm_workspace_bytes.restype, L.tenzo_cuda_gemm_workspace_bytes.argtypes = sz, []
     L.tenzo_cuda_gemm_take_timeouts.restype, L.tenzo_cuda_gemm_take_timeouts.argtypes = i32, []
     L.tenzo_cuda_linear_scan_part_floats.restype, L.tenzo_cuda_linear_scan_part_floats.argtypes = sz, [i32, i32, i32, i32]
+    L.tenzo_cuda_delta_rule_work_floats.restype, L.tenzo_cuda_delta_rule_work_floats.argtypes = sz, [i32, i32, i32, i32, i32]
     L.tenzo_hal_initialize.restype, L.tenzo_hal_initialize.argtypes = i32, []
     L.tenzo_hal_bitlinear_tl1_host.restype = i32
     L.tenzo_hal_bitlinear_tl1_host.argtypes = [c_f32p, c_u8p, c_f32p, sz, sz, sz, f32]

@@ -23,9 +23,10 @@ CORE = ["engine_core.cu", "capi.cu", "sampler.cu", "model_registry.cu"]
 FAMILIES = {
     "bitnet": ["tl1_gemv.cu", "tl1_umma.cu", "norm_quant.cu", "attention.cu", "attention_fast.cu", "lm_head.cu", "lm_head_umma.cu",
                "decode_persistent.cu", "engine.cu", "capi_bitnet.cu", "cuda_runtime_hal.cu", "model_loader.cu"],
-    "hybrid": ["rows.cu", "gemm.cu", "gemm_umma.cu", "window_attention.cu", "window_attention_mma.cu", "linear_scan.cu", "hybrid_engine.cu"],
+    "hybrid": ["rows.cu", "gemm.cu", "gemm_umma.cu", "window_attention.cu", "window_attention_mma.cu", "linear_attention.cu", "linear_scan.cu",
+               "delta_rule.cu", "latent_attention.cu", "route.cu", "hybrid_engine.cu", "hybrid_sozopel.cu", "hybrid_tigitar.cu"],
 }
-ARCHITECTURES = {"BitNet": "bitnet", "Sozopel": "hybrid"}      # "architecture" of a model folder's config.json
+ARCHITECTURES = {"BitNet": "bitnet", "Sozopel": "hybrid", "Tigitar": "hybrid"}      # "architecture" of a model folder's config.json
 SOURCES = CORE + FAMILIES["bitnet"] + FAMILIES["hybrid"]
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",

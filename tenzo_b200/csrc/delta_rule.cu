@@ -1,0 +1,411 @@
+// Gated delta rule (DeltaArgs): short convolutions with silu on q, k, v, unit q and k, one decay and one step size per head,
+// and a matrix state that is decayed, corrected towards v along k, then read. State, decays, step sizes and sums are fp32.
+//
+// With S the state before a token, a = S^T k and b = S^T q give everything of that token in one pass over the state:
+// u = beta (v - g a), o = g b + (k.q) u, and the new state is g S + k u^T.
+//
+// Decode: one CTA per (head, sequence), its part of the state fetched before the kernel waits for its producer. Inputs of the
+// convolutions are kept in rows by position modulo taps, so that heads that share q and k can read the older rows while
+// one of them stores the newest.
+// Chunk: rows are taken eight at a time. Within a block the values u solve a unit lower triangular system whose matrix
+// (step sizes, decays between the rows, k.k) does not depend on the state; a preparation kernel inverts it for every block
+// and head in parallel, next to the convolved rows. One kernel then walks the blocks: sixteen products with the state, the
+// 8 x 8 solutions, the outputs, the update. Decays appear only as products over a range of rows, never as quotients.
+#include "hybrid_common.cuh"
+
+namespace tz {
+
+constexpr int kDeltaThreads = 256, kDeltaPre = 16;       // decode: float4 pieces of the state a thread holds
+constexpr int kDeltaBlock = 8, kDeltaCols = 16, kDeltaStages = 4;
+constexpr int kDeltaCoef = 2 * kDeltaBlock * kDeltaBlock + 2 * kDeltaBlock;   // inverse * beta, read-out, decays from the start, to the end
+
+__device__ __forceinline__ float softplus_f(float z) { return softplus_neg(-z); }
+__device__ __forceinline__ float head_log_decay(const DeltaArgs& a, int head, float z) { return -expf(a.a_log[head]) * softplus_f(z + a.dt_bias[head]); }
+
+// ---- decode --------------------------------------------------------------------------------------------------------------
+// convolution and silu of one channel at position pos; rows of the tail that no token of the sequence has written are zero
+__device__ __forceinline__ float conv_at(const float* w, int ch, int n_ch, int taps, const float* tail, int tail_ld, int pos, float cur) {
+    float y = w[(size_t)(taps - 1) * n_ch + ch] * cur;
+    for (int j = 1; j < taps; ++j) y = fmaf(w[(size_t)(taps - 1 - j) * n_ch + ch], tail[(size_t)((pos + taps - j) % taps) * tail_ld], y);
+    return silu_f(y);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(kDeltaThreads) delta_decode_kernel(const DeltaArgs a) {
+    extern __shared__ float sm[];
+    __shared__ float s_red[4][8];
+    const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    const int ldv = (a.vdim + 3) & ~3, nc = ldv / 4;
+    int nc2 = 1;
+    while (nc2 < nc) nc2 *= 2;
+    const int col = tid & (nc2 - 1), rg = tid / nc2, n_rg = kDeltaThreads / nc2;
+    const bool live = col < nc;
+    float4* S = reinterpret_cast<float4*>(a.state + (size_t)seq * a.state_seq_stride + (size_t)head * a.dim * ldv) + col;
+    float4 pre[kDeltaPre];
+#pragma unroll
+    for (int i = 0; i < kDeltaPre; ++i) {
+        const int r = rg + i * n_rg;
+        if (live && r < a.dim) pre[i] = S[(size_t)r * nc];
+    }
+    float* s_q = sm;                                     // [dim]
+    float* s_k = s_q + a.dim;                            // [dim]
+    float* s_u = sm + ((2 * a.dim + 3) & ~3);            // [ldv]
+    float* s_a = s_u + ldv;                              // [n_rg][ldv]
+    float* s_b = s_a + n_rg * ldv;
+    const int group = a.heads / a.kv_heads, kvh = head / group;
+    const int n_q = a.kv_heads * a.dim, n_v = a.heads * a.vdim, n_ch = 2 * n_q + n_v;
+    pdl_wait();
+    pdl_launch_dependents();
+    const size_t row = (size_t)seq * a.ld;
+    const int pos = a.pos[seq];
+    float* tail = a.tail + (size_t)seq * a.tail_seq_stride;
+    float* newest = tail + (size_t)(pos % a.taps) * n_ch;
+    float q = 0.0f, k = 0.0f, v = 0.0f;
+    if (tid < a.dim) {                                   // head sizes are at most one thread per element
+        const int ch = kvh * a.dim + tid;
+        const float uq = a.q[row + ch], uk = a.k[row + ch];
+        q = conv_at(a.conv_q, ch, n_q, a.taps, tail + ch, n_ch, pos, uq);
+        k = conv_at(a.conv_k, ch, n_q, a.taps, tail + n_q + ch, n_ch, pos, uk);
+        if (head % group == 0) {
+            newest[ch] = uq;
+            newest[n_q + ch] = uk;
+        }
+    }
+    if (tid < a.vdim) {
+        const int ch = head * a.vdim + tid;
+        const float uv = a.v[row + ch];
+        v = conv_at(a.conv_v, ch, n_v, a.taps, tail + 2 * n_q + ch, n_ch, pos, uv);
+        newest[2 * n_q + ch] = uv;
+    }
+    const float g = expf(head_log_decay(a, head, a.a[row + head])), beta = sigmoid_f(a.b[row + head]);
+    const float qq = warp_sum(q * q), kk = warp_sum(k * k), qk = warp_sum(q * k);
+    if (lane == 0) { s_red[0][warp] = qq; s_red[1][warp] = kk; s_red[2][warp] = qk; }
+    __syncthreads();
+    float sums[3];
+#pragma unroll
+    for (int i = 0; i < 3; ++i) {
+        sums[i] = 0.0f;
+#pragma unroll
+        for (int w = 0; w < kDeltaThreads / 32; ++w) sums[i] += s_red[i][w];
+    }
+    const float iq = a.q_scale / sqrtf(sums[0] + a.unit_eps), ik = 1.0f / sqrtf(sums[1] + a.unit_eps), kq = sums[2] * iq * ik;
+    if (tid < a.dim) { s_q[tid] = q * iq; s_k[tid] = k * ik; }
+    __syncthreads();
+    if (live) {
+        float pa[4] = {}, pb[4] = {};
+        auto step = [&](int r, const float4& s4) {
+            const float kr = s_k[r], qr = s_q[r], s[4] = {s4.x, s4.y, s4.z, s4.w};
+#pragma unroll
+            for (int j = 0; j < 4; ++j) {
+                pa[j] = fmaf(kr, s[j], pa[j]);
+                pb[j] = fmaf(qr, s[j], pb[j]);
+            }
+        };
+#pragma unroll
+        for (int i = 0; i < kDeltaPre; ++i)
+            if (rg + i * n_rg < a.dim) step(rg + i * n_rg, pre[i]);
+        for (int r = rg + kDeltaPre * n_rg; r < a.dim; r += n_rg) step(r, S[(size_t)r * nc]);
+        *reinterpret_cast<float4*>(s_a + rg * ldv + col * 4) = make_float4(pa[0], pa[1], pa[2], pa[3]);
+        *reinterpret_cast<float4*>(s_b + rg * ldv + col * 4) = make_float4(pb[0], pb[1], pb[2], pb[3]);
+    }
+    __syncthreads();
+    float o = 0.0f;
+    if (tid < ldv) {
+        float sa = 0.0f, sb = 0.0f;
+        for (int r = 0; r < n_rg; ++r) {
+            sa += s_a[r * ldv + tid];
+            sb += s_b[r * ldv + tid];
+        }
+        const float u = tid < a.vdim ? beta * (v - g * sa) : 0.0f;
+        s_u[tid] = u;
+        if (tid < a.vdim) o = fmaf(g, sb, kq * u);
+    }
+    const float oo = warp_sum(o * o);
+    if (lane == 0) s_red[3][warp] = oo;
+    __syncthreads();
+    if (tid < a.vdim) {
+        float t = 0.0f;
+#pragma unroll
+        for (int w = 0; w < kDeltaThreads / 32; ++w) t += s_red[3][w];
+        const float y = o * (1.0f / sqrtf(t / (float)a.vdim + a.eps)) * a.norm[tid];
+        reinterpret_cast<T*>(a.out)[(size_t)seq * a.ld_out + head * a.vdim + tid] = from_f<T>(y * silu_f(a.g[row + head * a.vdim + tid]));
+    }
+    if (live) {
+        const float4 u = *reinterpret_cast<const float4*>(s_u + col * 4);
+        auto update = [&](int r, const float4& s) {
+            const float kr = s_k[r];
+            S[(size_t)r * nc] = make_float4(fmaf(g, s.x, kr * u.x), fmaf(g, s.y, kr * u.y), fmaf(g, s.z, kr * u.z), fmaf(g, s.w, kr * u.w));
+        };
+#pragma unroll
+        for (int i = 0; i < kDeltaPre; ++i)
+            if (rg + i * n_rg < a.dim) update(rg + i * n_rg, pre[i]);
+        for (int r = rg + kDeltaPre * n_rg; r < a.dim; r += n_rg) update(r, S[(size_t)r * nc]);
+    }
+}
+
+// ---- chunk ---------------------------------------------------------------------------------------------------------------
+struct DeltaLaunch {
+    DeltaArgs a;
+    int dp, vp;                  // padded head sizes: 32 KJ, a multiple of kDeltaCols
+    float *kq, *v, *coef, *o;    // [block][kv_head][8 k, 8 q][dp], [block][head][8][vp], [block][head][kDeltaCoef], [M][heads*vdim]
+};
+
+// One CTA per (block of rows, kv head), one warp per row.
+__global__ void __launch_bounds__(kDeltaThreads) delta_prepare_kernel(const DeltaLaunch L) {
+    extern __shared__ float sm[];
+    __shared__ float s_kk[8][9], s_qk[8][9], s_sys[8][64], s_gl[8][8], s_beta[8][8];
+    const DeltaArgs& a = L.a;
+    const int b = blockIdx.x, kvh = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, dp = L.dp;
+    const int t = b * kDeltaBlock + warp, group = a.heads / a.kv_heads;
+    const int n_q = a.kv_heads * a.dim, n_v = a.heads * a.vdim, n_ch = 2 * n_q + n_v;
+    const bool in = t < a.M;
+    float* s_k = sm;                                     // [8][dp]
+    float* s_q = sm + 8 * dp;
+    // convolved channel of this warp's row: `src` the channel's projection, `first` its place among the tail's channels
+    auto convolved = [&](const float* src, const float* w, int ch, int nch, int first) {
+        float y = 0.0f;
+        for (int j = 0; j < a.taps; ++j) {
+            const int r = t - j, p = a.pos0 + r;
+            const float u = r >= 0 ? src[(size_t)r * a.ld + ch] : p >= 0 ? a.tail[(size_t)(p % a.taps) * n_ch + first + ch] : 0.0f;
+            y = fmaf(w[(size_t)(a.taps - 1 - j) * nch + ch], u, y);
+        }
+        return silu_f(y);
+    };
+    float qq = 0.0f, kk = 0.0f;
+    for (int d = lane; d < dp; d += 32) {
+        const bool ok = in && d < a.dim;
+        const float q = ok ? convolved(a.q, a.conv_q, kvh * a.dim + d, n_q, 0) : 0.0f;
+        const float k = ok ? convolved(a.k, a.conv_k, kvh * a.dim + d, n_q, n_q) : 0.0f;
+        s_q[warp * dp + d] = q;
+        s_k[warp * dp + d] = k;
+        qq = fmaf(q, q, qq);
+        kk = fmaf(k, k, kk);
+    }
+    qq = warp_sum(qq);
+    kk = warp_sum(kk);
+    const float iq = a.q_scale / sqrtf(qq + a.unit_eps), ik = 1.0f / sqrtf(kk + a.unit_eps);
+    float* out = L.kq + ((size_t)b * a.kv_heads + kvh) * 16 * dp;
+    for (int d = lane; d < dp; d += 32) {
+        const float q = s_q[warp * dp + d] * iq, k = s_k[warp * dp + d] * ik;
+        s_q[warp * dp + d] = q;
+        s_k[warp * dp + d] = k;
+        out[warp * dp + d] = k;
+        out[(8 + warp) * dp + d] = q;
+    }
+    for (int i = lane; i < group * L.vp; i += 32) {
+        const int h = kvh * group + i / L.vp, d = i % L.vp;
+        L.v[(((size_t)b * a.heads + h) * 8 + warp) * L.vp + d] = in && d < a.vdim ? convolved(a.v, a.conv_v, h * a.vdim + d, n_v, 2 * n_q) : 0.0f;
+    }
+    __syncthreads();
+    for (int j = 0; j <= warp; ++j) {                    // row `warp` against the rows up to it
+        float kkj = 0.0f, qkj = 0.0f;
+        for (int d = lane; d < dp; d += 32) {
+            const float kj = s_k[j * dp + d];
+            kkj = fmaf(s_k[warp * dp + d], kj, kkj);
+            qkj = fmaf(s_q[warp * dp + d], kj, qkj);
+        }
+        kkj = warp_sum(kkj);
+        qkj = warp_sum(qkj);
+        if (lane == 0) { s_kk[warp][j] = kkj; s_qk[warp][j] = qkj; }
+    }
+    __syncthreads();
+    for (int hh = warp; hh < group; hh += 8) {
+        const int h = kvh * group + hh;
+        float* c = L.coef + ((size_t)b * a.heads + h) * kDeltaCoef;
+        if (lane < 8) {
+            const int r = b * kDeltaBlock + lane;        // rows past the end change nothing
+            s_gl[warp][lane] = r < a.M ? head_log_decay(a, h, a.a[(size_t)r * a.ld + h]) : 0.0f;
+            s_beta[warp][lane] = r < a.M ? sigmoid_f(a.b[(size_t)r * a.ld + h]) : 0.0f;
+        }
+        __syncwarp();
+        for (int e = lane; e < 64; e += 32) {
+            const int i = e >> 3, j = e & 7;
+            float s = 0.0f;
+            for (int m = j + 1; m <= i; ++m) s += s_gl[warp][m];
+            const float d = expf(s);
+            s_sys[warp][e] = j < i ? s_beta[warp][i] * d * s_kk[i][j] : 0.0f;
+            c[64 + e] = j <= i ? d * s_qk[i][j] : 0.0f;
+        }
+        __syncwarp();
+        if (lane < 8) {                                  // column `lane` of the inverse of (1 + system), times beta
+            float x[8];
+#pragma unroll
+            for (int i = 0; i < 8; ++i) {
+                float y = i == lane ? 1.0f : 0.0f;
+#pragma unroll
+                for (int j = 0; j < i; ++j) y = fmaf(-s_sys[warp][i * 8 + j], x[j], y);
+                x[i] = y;
+                c[i * 8 + lane] = y * s_beta[warp][lane];
+            }
+            float from = 0.0f, to = 0.0f;
+            for (int m = 0; m <= lane; ++m) from += s_gl[warp][m];
+            for (int m = lane + 1; m < 8; ++m) to += s_gl[warp][m];
+            c[128 + lane] = expf(from);
+            c[136 + lane] = expf(to);
+        }
+        __syncwarp();
+    }
+}
+
+// Sixteen value columns of one head, four per warp; eight lanes share a column, lane l holding the state's rows
+// 4 (l + 8 j) .. + 3, and stand for the block's eight rows once the products are summed.
+template <int KJ>
+__global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
+    constexpr int DP = 32 * KJ, V = 16 * DP, C = V + 8 * kDeltaCols, FLOATS = C + kDeltaCoef;
+    extern __shared__ __align__(16) float smem[];
+    const DeltaArgs& a = L.a;
+    const int head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, l = lane & 7, cl = (tid >> 5) * 4 + (lane >> 3), c = blockIdx.x * kDeltaCols + cl;
+    const int group = a.heads / a.kv_heads, kvh = head / group, ldv = (a.vdim + 3) & ~3, nv = a.heads * a.vdim;
+    const int n_blocks = (a.M + kDeltaBlock - 1) / kDeltaBlock;
+    const bool live = c < a.vdim;
+    auto stage = [&](int b) {
+        if (b < n_blocks) {
+            float* dst = smem + (b % kDeltaStages) * FLOATS;
+            const float* kq = L.kq + ((size_t)b * a.kv_heads + kvh) * 16 * DP;
+            for (int i = tid; i < 4 * DP; i += 128) cp16(dst + 4 * i, kq + 4 * i);
+            if (tid < 32) cp16(dst + V + 4 * tid, L.v + (((size_t)b * a.heads + head) * 8 + tid / 4) * L.vp + blockIdx.x * kDeltaCols + (tid & 3) * 4);
+            else if (tid < 32 + kDeltaCoef / 4) cp16(dst + C + 4 * (tid - 32), L.coef + ((size_t)b * a.heads + head) * kDeltaCoef + 4 * (tid - 32));
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    };
+    for (int b = 0; b + 1 < kDeltaStages; ++b) stage(b);
+    float s[KJ * 4];
+#pragma unroll
+    for (int j = 0; j < KJ * 4; ++j) {
+        const int d = 4 * (l + 8 * (j >> 2)) + (j & 3);
+        s[j] = live && d < a.dim ? a.state[((size_t)head * a.dim + d) * ldv + c] : 0.0f;
+    }
+    for (int b = 0; b < n_blocks; ++b) {
+        asm volatile("cp.async.wait_group %0;" ::"n"(kDeltaStages - 2) : "memory");
+        __syncthreads();                                 // the block is here, and the stage before it is free
+        stage(b + kDeltaStages - 1);
+        const float* buf = smem + (b % kDeltaStages) * FLOATS;
+        const float *sk = buf + 4 * l, *sq = sk + 8 * DP, *co = buf + C;
+        float pa[8], pb[8];
+#pragma unroll
+        for (int t = 0; t < 8; ++t) {
+            float x = 0.0f, y = 0.0f;
+#pragma unroll
+            for (int j = 0; j < KJ; ++j) {
+                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 32 * j), q4 = *reinterpret_cast<const float4*>(sq + t * DP + 32 * j);
+                x = fmaf(k4.x, s[4 * j], x); x = fmaf(k4.y, s[4 * j + 1], x); x = fmaf(k4.z, s[4 * j + 2], x); x = fmaf(k4.w, s[4 * j + 3], x);
+                y = fmaf(q4.x, s[4 * j], y); y = fmaf(q4.y, s[4 * j + 1], y); y = fmaf(q4.z, s[4 * j + 2], y); y = fmaf(q4.w, s[4 * j + 3], y);
+            }
+            pa[t] = x;
+            pb[t] = y;
+            if (KJ > 4) asm volatile("" ::: "memory");   // otherwise the loads of all rows are moved ahead, and spilled
+        }
+        int which;                                       // = l
+        const float at = group_sums<8, 8>(pa, lane, which), bt = group_sums<8, 8>(pb, lane, which);
+        const float from = co[128 + l], x = buf[V + l * kDeltaCols + cl] - from * at;
+        float u = 0.0f, o = from * bt;
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const float4 w = *reinterpret_cast<const float4*>(co + l * 8 + 4 * h);
+            u = fmaf(w.x, __shfl_sync(0xffffffffu, x, 4 * h, 8), u);
+            u = fmaf(w.y, __shfl_sync(0xffffffffu, x, 4 * h + 1, 8), u);
+            u = fmaf(w.z, __shfl_sync(0xffffffffu, x, 4 * h + 2, 8), u);
+            u = fmaf(w.w, __shfl_sync(0xffffffffu, x, 4 * h + 3, 8), u);
+        }
+        const float decay = co[128 + 7];
+#pragma unroll
+        for (int j = 0; j < KJ * 4; ++j) s[j] *= decay;
+        const float4 p0 = *reinterpret_cast<const float4*>(co + 64 + l * 8), p1 = *reinterpret_cast<const float4*>(co + 64 + l * 8 + 4);
+        const float p[8] = {p0.x, p0.y, p0.z, p0.w, p1.x, p1.y, p1.z, p1.w};
+#pragma unroll
+        for (int t = 0; t < 8; ++t) {
+            const float ut = __shfl_sync(0xffffffffu, u, t, 8), w = ut * co[136 + t];
+            o = fmaf(p[t], ut, o);
+            if (KJ > 4) asm volatile("" ::: "memory");
+#pragma unroll
+            for (int j = 0; j < KJ; ++j) {
+                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 32 * j);
+                s[4 * j] = fmaf(k4.x, w, s[4 * j]);
+                s[4 * j + 1] = fmaf(k4.y, w, s[4 * j + 1]);
+                s[4 * j + 2] = fmaf(k4.z, w, s[4 * j + 2]);
+                s[4 * j + 3] = fmaf(k4.w, w, s[4 * j + 3]);
+            }
+        }
+        const int row = b * kDeltaBlock + l;
+        if (live && row < a.M) L.o[(size_t)row * nv + head * a.vdim + c] = o;
+    }
+#pragma unroll
+    for (int j = 0; j < KJ * 4; ++j) {
+        const int d = 4 * (l + 8 * (j >> 2)) + (j & 3);
+        if (live && d < a.dim) a.state[((size_t)head * a.dim + d) * ldv + c] = s[j];
+    }
+    // the convolutions' last inputs; the preparation kernel has read the older ones
+    if (blockIdx.x == 0) {
+        const int n_q = a.kv_heads * a.dim, n_ch = 2 * n_q + nv;
+        for (int t = max(0, a.M - a.taps); t < a.M; ++t) {
+            float* to = a.tail + (size_t)((a.pos0 + t) % a.taps) * n_ch;
+            const size_t row = (size_t)t * a.ld;
+            if (head % group == 0)
+                for (int d = tid; d < a.dim; d += 128) {
+                    to[kvh * a.dim + d] = a.q[row + kvh * a.dim + d];
+                    to[n_q + kvh * a.dim + d] = a.k[row + kvh * a.dim + d];
+                }
+            for (int d = tid; d < a.vdim; d += 128) to[2 * n_q + head * a.vdim + d] = a.v[row + head * a.vdim + d];
+        }
+    }
+}
+
+static size_t delta_work_floats(int M, int heads, int kv_heads, int dp, int vp, int vdim, DeltaLaunch* L, float* work) {
+    const size_t blocks = (M + kDeltaBlock - 1) / kDeltaBlock;
+    const size_t kq = blocks * kv_heads * 16 * dp, v = blocks * heads * 8 * vp, coef = blocks * heads * kDeltaCoef;
+    if (L) { L->kq = work; L->v = work + kq; L->coef = L->v + v; L->o = L->coef + coef; }
+    return kq + v + coef + (size_t)M * heads * vdim;
+}
+
+int launch_delta(const DeltaArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
+    if (a.M <= 0) return 0;
+    if (a.dim < 1 || a.dim > kMaxHeadDim || a.vdim < 1 || a.vdim > kMaxHeadDim || a.kv_heads < 1 || a.heads < 1 || a.heads % a.kv_heads ||
+        a.taps < 1 || a.taps > kMaxTaps || !a.norm) return -1;
+    if (a.decode) {
+        const int ldv = round_up(a.vdim, 4);
+        int nc2 = 1;
+        while (nc2 < ldv / 4) nc2 *= 2;
+        const size_t smem = 4 * (size_t)(round_up(2 * a.dim, 4) + ldv + 2 * (kDeltaThreads / nc2) * ldv);
+        *n_kernels += 1;
+        auto go = [&](auto kernel) {
+            if (int rc = allow_smem(kernel, smem)) return rc;
+            return launch_kernel(kernel, dim3(a.heads, a.M), dim3(kDeltaThreads), smem, st, a.use_pdl, 1, a);
+        };
+        return a.f32 ? go(delta_decode_kernel<float>) : go(delta_decode_kernel<bf16>);
+    }
+    DeltaLaunch L;
+    L.a = a;
+    L.dp = a.dim <= 32 ? 32 : a.dim <= 64 ? 64 : a.dim <= 128 ? 128 : 256;
+    L.vp = round_up(a.vdim, kDeltaCols);
+    delta_work_floats(a.M, a.heads, a.kv_heads, L.dp, L.vp, a.vdim, &L, a.work);
+    delta_prepare_kernel<<<dim3((a.M + kDeltaBlock - 1) / kDeltaBlock, a.kv_heads), kDeltaThreads, 64 * (size_t)L.dp, st>>>(L);
+    const dim3 grid(L.vp / kDeltaCols, a.heads);
+    auto go = [&](auto kernel) {
+        const size_t smem = 4 * (size_t)kDeltaStages * (16 * L.dp + 8 * kDeltaCols + kDeltaCoef);
+        if (int rc = allow_smem(kernel, smem)) return rc;
+        kernel<<<grid, 128, smem, st>>>(L);
+        return (int)cudaGetLastError();
+    };
+    const int rc = L.dp == 32 ? go(delta_block_kernel<1>) : L.dp == 64 ? go(delta_block_kernel<2>) : L.dp == 128 ? go(delta_block_kernel<4>) : go(delta_block_kernel<8>);
+    if (rc) return rc;
+    ScanArgs s;                                          // per head: o / rms(o) * norm * silu(g)
+    s.M = a.M; s.heads = a.heads; s.vdim = a.vdim; s.o_rows = L.o; s.eps = a.eps; s.norm = a.norm;
+    s.g = a.g; s.ld = a.ld; s.out = a.out; s.ld_out = a.ld_out; s.f32 = a.f32;
+    *n_kernels += 2;
+    return launch_scan_gate(s, st, n_kernels);
+}
+
+}  // namespace tz
+
+extern "C" int tenzo_cuda_delta_rule(const tenzo_delta_args* args, void* stream) {
+    if (!args) return TENZO_ERROR_INVALID_ARGUMENT;
+    tz::DeltaArgs a;
+    static_cast<tenzo_delta_args&>(a) = *args;
+    unsigned long long n = 0;
+    return tz::launch_delta(a, static_cast<cudaStream_t>(stream), &n);
+}
+
+extern "C" size_t tenzo_cuda_delta_rule_work_floats(int M, int heads, int kv_heads, int dim, int vdim) {
+    const int dp = dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256;
+    return tz::delta_work_floats(M, heads, kv_heads, dp, tz::round_up(vdim, tz::kDeltaCols), vdim, nullptr, nullptr);
+}

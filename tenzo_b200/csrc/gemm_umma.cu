@@ -39,20 +39,88 @@ __device__ __forceinline__ void umma_bf16(uint32_t tmem_d, uint64_t da, uint64_t
                  ::"r"(tmem_d), "l"(da), "l"(db), "r"(idesc), "r"(accumulate) : "memory");
 }
 
-__device__ __forceinline__ void gu_store16(const GemmArgs& a, int n, int m0, const float (&v)[16]) {
+// Sixteen rows of column n, rows m0 .. below m_end. All lanes of the warp call it (the two halves of a GLU pair are neighbours).
+__device__ __forceinline__ void gu_store16(const GemmArgs& a, int n, int m0, int m_end, const float (&v)[16]) {
+    if (a.epilogue == TENZO_GEMM_GLU_RELU || a.epilogue == TENZO_GEMM_GLU_SILU) {
+        const bool up = threadIdx.x & 1;                       // the even lane finishes eight rows, the odd one the others
+        float g[8], u[8];
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            const float other = __shfl_xor_sync(0xffffffffu, up ? v[i] : v[i + 8], 1);
+            g[i] = up ? other : v[i];
+            u[i] = up ? v[i + 8] : other;
+        }
+        if (n >= a.N) return;
+        bf16* c = reinterpret_cast<bf16*>(a.c) + n / 2;
+        const int m1 = m0 + (up ? 8 : 0);
+#pragma unroll
+        for (int i = 0; i < 8; ++i)
+            if (m1 + i < m_end) c[(size_t)(m1 + i) * a.ld_c] = __float2bfloat16_rn(glu_f(a.epilogue, g[i], u[i]));
+        return;
+    }
     if (n >= a.N) return;
-    if (a.epilogue == TENZO_GEMM_XIELU) {
+    if (a.epilogue == TENZO_GEMM_XIELU || a.epilogue == TENZO_GEMM_CAST) {
         bf16* c = reinterpret_cast<bf16*>(a.c) + n;
+        const bool act = a.epilogue == TENZO_GEMM_XIELU;
 #pragma unroll
         for (int i = 0; i < 16; ++i)
-            if (m0 + i < a.M) c[(size_t)(m0 + i) * a.ld_c] = __float2bfloat16_rn(xielu_f(v[i], a.act_pos, a.act_neg));
+            if (m0 + i < m_end) c[(size_t)(m0 + i) * a.ld_c] = __float2bfloat16_rn(act ? xielu_f(v[i], a.act_pos, a.act_neg) : v[i]);
     } else {
         float* c = reinterpret_cast<float*>(a.c) + n;
+        const bool cap = a.epilogue == TENZO_GEMM_SOFTCAP;
 #pragma unroll
         for (int i = 0; i < 16; ++i)
-            if (m0 + i < a.M) c[(size_t)(m0 + i) * a.ld_c] = v[i];
+            if (m0 + i < m_end) c[(size_t)(m0 + i) * a.ld_c] = cap ? soft_cap_f(v[i], a.cap) : v[i];
     }
 }
+
+// A unit of work: a weight tile against a tile of activation rows, over a part of K.
+struct GuUnit {
+    int row_w, row_a, n0;        // first row of the weight tile and of the activation tile in their tensor maps; its first column
+    int m0, m_end;               // first output row, end of the rows that may be stored
+    int split, tile;
+};
+// Unit u of the launch, false past the last one. Every role walks its units in ascending order; in the grouped form the
+// number of row tiles of a group is read as the walk reaches it.
+struct GuWalk {
+    int g = 0, base = 0, lo = 0, hi = -1;
+    __device__ __forceinline__ bool at(const GuLaunch& L, int u, GuUnit& o) {
+        const GemmArgs& a = L.a;
+        if (!a.group_off) {
+            if (u >= L.n_tiles * L.m_tiles * L.n_split) return false;
+            // consecutive units share the activation rows
+            const int nt = (u / L.n_split) % L.n_tiles, mt = u / (L.n_split * L.n_tiles);
+            o.split = u % L.n_split;
+            o.tile = mt * L.n_tiles + nt;
+            o.n0 = o.row_w = nt * kGuRows;
+            int seg = 0;
+            if (a.seg_rows > 0) seg = o.row_w / a.seg_rows;
+            else
+                while (seg + 1 < a.n_seg && o.row_w >= a.seg_end[seg]) ++seg;
+            o.row_a = seg * L.a_seg_rows + mt * L.n_box;
+            o.m0 = mt * L.n_box;
+            o.m_end = a.M;
+            return true;
+        }
+        for (;; ++g, hi = -1) {
+            if (g >= a.n_group) return false;
+            if (hi < 0) {
+                lo = a.group_off[g];
+                hi = min(a.M, a.group_off[g + 1]);
+            }
+            const int n = (hi - lo + L.n_box - 1) / L.n_box * L.n_tiles;
+            if (u < base + n) break;
+            base += n;
+        }
+        const int nt = (u - base) % L.n_tiles, mt = (u - base) / L.n_tiles;
+        o.split = o.tile = 0;
+        o.n0 = nt * kGuRows;
+        o.row_w = g * a.N + o.n0;
+        o.row_a = o.m0 = lo + mt * L.n_box;
+        o.m_end = hi;
+        return true;
+    }
+};
 
 __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch L, const __grid_constant__ CUtensorMap wmap,
                                                                   const __grid_constant__ CUtensorMap amap) {
@@ -65,7 +133,6 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
     uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + GuSmem::n_bars);
     int* s_last = reinterpret_cast<int*>(tmem_slot + 1);
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-    const int n_units = L.n_tiles * L.m_tiles * L.n_split;
 
     if (tid == 0) {
         for (int s = 0; s < kGuStages; ++s) { mbar_init(&bar_full[s], 1); mbar_init(&bar_empty[s], 1); }
@@ -84,28 +151,22 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
     pdl_launch_dependents();
     bool timed_out = false;
 
-    // unit -> (weight tile, row tile, split): consecutive units share the activation rows
-    auto unit_split = [&](int u) { return u % L.n_split; };
-    auto unit_ntile = [&](int u) { return (u / L.n_split) % L.n_tiles; };
-    auto unit_mtile = [&](int u) { return u / (L.n_split * L.n_tiles); };
-    auto k_begin = [&](int u) { return unit_split(u) * L.chunks_per_split; };
-    auto k_end = [&](int u) { return min(L.chunks, k_begin(u) + L.chunks_per_split); };
+    GuWalk walk;
+    GuUnit t = {};
+    auto k_begin = [&]() { return t.split * L.chunks_per_split; };
+    auto k_end = [&]() { return min(L.chunks, k_begin() + L.chunks_per_split); };
 
     if (warp == 0) {
         if (lane == 0) {
             int it = 0;
-            for (int u = blockIdx.x; u < n_units && !timed_out; u += gridDim.x) {
-                const int row_w = unit_ntile(u) * kGuRows;
-                int seg = 0;
-                while (seg + 1 < L.a.n_seg && row_w >= L.a.seg_end[seg]) ++seg;
-                const int row_a = seg * L.a_seg_rows + unit_mtile(u) * N;
-                for (int j = k_begin(u); j < k_end(u); ++j, ++it) {
+            for (int u = blockIdx.x; !timed_out && walk.at(L, u, t); u += gridDim.x) {
+                for (int j = k_begin(); j < k_end(); ++j, ++it) {
                     const int s = it % kGuStages, use = it / kGuStages;
                     if (use > 0 && !mbar_spin_bounded(&bar_empty[s], (unsigned)(use - 1) & 1u)) { timed_out = true; break; }
                     unsigned char* sp = stages + (size_t)s * stage_bytes;
                     mbar_expect_tx(&bar_full[s], (unsigned)stage_bytes);
-                    tma_load_2d(sp, &wmap, j * kGuKc, row_w, &bar_full[s]);
-                    tma_load_2d(sp + kGuRows * 128, &amap, j * kGuKc, row_a, &bar_full[s]);
+                    tma_load_2d(sp, &wmap, j * kGuKc, t.row_w, &bar_full[s]);
+                    tma_load_2d(sp + kGuRows * 128, &amap, j * kGuKc, t.row_a, &bar_full[s]);
                 }
             }
             if (timed_out)                                     // shared memory must outlive the copies in flight
@@ -116,13 +177,13 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
             // d = f32, a = b = bf16, both K-major, N at bit 17 (>>3), M at bit 24 (>>4)
             const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(kGuRows >> 4) << 24);
             int it = 0, n = 0;
-            for (int u = blockIdx.x; u < n_units && !timed_out; u += gridDim.x, ++n) {
+            for (int u = blockIdx.x; !timed_out && walk.at(L, u, t); u += gridDim.x, ++n) {
                 const int half = n & 1, use_acc = n >> 1;
                 if (use_acc > 0 && !mbar_spin_bounded(&bar_acc_empty[half], (unsigned)(use_acc - 1) & 1u)) { timed_out = true; break; }
                 tc_fence_after();
                 const uint32_t d = tmem_base + (uint32_t)(half * L.tmem_half);
                 uint32_t acc = 0;
-                for (int j = k_begin(u); j < k_end(u); ++j, ++it) {
+                for (int j = k_begin(); j < k_end(); ++j, ++it) {
                     const int s = it % kGuStages, use = it / kGuStages;
                     if (!mbar_spin_bounded(&bar_full[s], (unsigned)use & 1u)) { timed_out = true; break; }
                     tc_fence_after();
@@ -141,7 +202,7 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
     } else {
         const int q = warp & 3, row = 32 * q + lane;
         int n = 0;
-        for (int u = blockIdx.x; u < n_units; u += gridDim.x, ++n) {
+        for (int u = blockIdx.x; walk.at(L, u, t); u += gridDim.x, ++n) {
             const int half = n & 1, use_acc = n >> 1;
             bool ok = true;
             if (lane == 0) ok = mbar_spin_bounded(&bar_acc_full[half], (unsigned)use_acc & 1u);
@@ -150,10 +211,9 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
             if (!ok) timed_out = true;
             tc_fence_after();
             const uint32_t d = tmem_base + ((uint32_t)(32 * q) << 16) + (uint32_t)(half * L.tmem_half);
-            const int n_row = unit_ntile(u) * kGuRows + row, m0 = unit_mtile(u) * N;
-            const int tile = unit_mtile(u) * L.n_tiles + unit_ntile(u);
-            float* part = L.n_split > 1 ? L.partial + ((size_t)tile * L.n_split + unit_split(u)) * N * kGuRows : nullptr;
-            for (int c0 = 0; c0 < N; c0 += 16) {
+            const int n_row = t.n0 + row, m0 = t.m0, tile = t.tile;
+            float* part = L.n_split > 1 ? L.partial + ((size_t)tile * L.n_split + t.split) * N * kGuRows : nullptr;
+            for (int c0 = 0; c0 < N && m0 + c0 < t.m_end; c0 += 16) {
                 uint32_t r[16];
                 float v[16];
                 tmem_ld16(d + (uint32_t)c0, r);
@@ -163,7 +223,7 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
 #pragma unroll
                     for (int i = 0; i < 16; ++i) __stcg(part + (size_t)(c0 + i) * kGuRows + row, v[i]);
                 } else {
-                    gu_store16(L.a, n_row, m0 + c0, v);
+                    gu_store16(L.a, n_row, m0 + c0, t.m_end, v);
                 }
             }
             tc_fence_before();
@@ -181,7 +241,7 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
                         for (int s = 0; s < L.n_split; ++s)
 #pragma unroll
                             for (int i = 0; i < 16; ++i) v[i] += __ldcg(base + ((size_t)s * N + c0 + i) * kGuRows);
-                        gu_store16(L.a, n_row, m0 + c0, v);
+                        gu_store16(L.a, n_row, m0 + c0, t.m_end, v);
                     }
                     if (tid == 64) L.counters[tile] = 0;      // ready for the next launch
                 }
@@ -203,6 +263,8 @@ constexpr size_t kGuWorkspaceBytes = kGuCounterBytes + (size_t)kGuSplitTiles * k
 
 bool gemm_umma_applicable(const GemmArgs& a) {
     if (a.f32 || a.M < kGemmUmmaMinRows || a.ld_k % kGuKc || !a.workspace) return false;
+    if (a.group_off) return !a.a_index || a.a_gather;
+    if (a.seg_rows > 0) return a.seg_rows % kGuRows == 0 && a.a_seg_stride % a.ld_k == 0;
     for (int s = 0; s + 1 < a.n_seg; ++s)
         if (a.seg_end[s] % kGuRows) return false;
     return a.n_seg == 1 || a.a_seg_stride % a.ld_k == 0;
@@ -211,16 +273,18 @@ bool gemm_umma_applicable(const GemmArgs& a) {
 int launch_gemm_umma(const GemmArgs& a, cudaStream_t st) {
     GuLaunch L;
     L.a = a;
-    L.n_box = std::min(kGuMaxN, round_up(a.M, 16));
+    // grouped: about a group's mean number of rows, so that most groups are one tile
+    L.n_box = std::min(kGuMaxN, round_up(a.group_off ? std::max(1, a.M / a.n_group) : a.M, 16));
     L.tmem_half = 32;
     while (L.tmem_half < L.n_box) L.tmem_half *= 2;
     L.n_tiles = (a.N + kGuRows - 1) / kGuRows;
     L.m_tiles = (a.M + L.n_box - 1) / L.n_box;
     L.chunks = a.ld_k / kGuKc;
-    L.a_seg_rows = a.n_seg > 1 ? (int)(a.a_seg_stride / a.ld_k) : 0;
-    const int tiles = L.n_tiles * L.m_tiles;
+    const int n_seg = a.seg_rows > 0 ? (a.N + a.seg_rows - 1) / a.seg_rows : a.n_seg;
+    L.a_seg_rows = n_seg > 1 ? (int)(a.a_seg_stride / a.ld_k) : 0;
+    const int tiles = a.group_off ? L.n_tiles * (L.m_tiles + a.n_group) : L.n_tiles * L.m_tiles;      // grouped: at most
     int split = 1;
-    if (tiles <= kGuSplitTiles / 2 && tiles * sizeof(unsigned) <= kGuCounterBytes)
+    if (!a.group_off && tiles <= kGuSplitTiles / 2 && tiles * sizeof(unsigned) <= kGuCounterBytes)
         split = std::max(1, std::min({kGuMaxSplit, kGuSplitTiles / tiles, L.chunks / 2}));
     L.chunks_per_split = (L.chunks + split - 1) / split;
     L.n_split = (L.chunks + L.chunks_per_split - 1) / L.chunks_per_split;
@@ -228,9 +292,9 @@ int launch_gemm_umma(const GemmArgs& a, cudaStream_t st) {
     L.partial = reinterpret_cast<float*>(static_cast<char*>(a.workspace) + kGuCounterBytes);
     if (L.n_split > 1 && kGuCounterBytes + (size_t)tiles * L.n_split * L.n_box * kGuRows * 4 > a.workspace_bytes) return -1;
     CUtensorMap wmap, amap;
-    if (int rc = encode_2d(&wmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.w, (uint64_t)a.ld_k, (uint64_t)a.N, (uint64_t)a.ld_k * 2, kGuKc, kGuRows,
+    if (int rc = encode_2d(&wmap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.w, (uint64_t)a.ld_k, (uint64_t)a.N * (a.group_off ? a.n_group : 1), (uint64_t)a.ld_k * 2, kGuKc, kGuRows,
                            CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
-    const uint64_t a_rows = a.n_seg > 1 ? (uint64_t)(a.n_seg - 1) * L.a_seg_rows + a.M : (uint64_t)a.M;
+    const uint64_t a_rows = n_seg > 1 ? (uint64_t)(n_seg - 1) * L.a_seg_rows + a.M : (uint64_t)a.M;
     if (int rc = encode_2d(&amap, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, a.a, (uint64_t)a.ld_k, a_rows, (uint64_t)a.ld_k * 2, kGuKc, (uint32_t)L.n_box,
                            CU_TENSOR_MAP_SWIZZLE_128B)) return rc;
     const size_t smem = GuSmem::bytes(L.n_box);

@@ -30,8 +30,53 @@ __device__ __forceinline__ float sigmoid_f(float z) { return 1.0f / (1.0f + expf
 __device__ __forceinline__ float silu_f(float z) { return z * sigmoid_f(z); }
 // ln(1 + e^-z), stable on both sides
 __device__ __forceinline__ float softplus_neg(float z) { return fmaxf(-z, 0.0f) + log1pf(expf(-fabsf(z))); }
+__device__ __forceinline__ float soft_cap_f(float z, float cap) { return cap * tanhf(z / cap); }
+__device__ __forceinline__ float glu_f(int epilogue, float gate, float up) {
+    return (epilogue == TENZO_GEMM_GLU_RELU ? fmaxf(gate, 0.0f) : silu_f(gate)) * up;
+}
 __device__ __forceinline__ float xielu_f(float z, float pos, float neg) {
     return 0.5f * z + (z > 0.0f ? pos * z * z : neg * (expm1f(z) - z));
+}
+
+// slope of head h's linear distance bias
+__device__ __forceinline__ float head_slope(float slope_base, int heads, int h) {
+    return slope_base == 0.0f ? 0.0f : exp2f(-slope_base * (float)(h + 1) / (float)heads);
+}
+
+// Sums of GQ values over groups of LK lanes: halves of the values travel while there are several, so that the total is
+// GQ - 1 + log2(LK / GQ) exchanges. The lane is left with the sum of value `which`.
+template <int GQ, int LK>
+__device__ __forceinline__ float group_sums(float (&s)[GQ], int lane, int& which) {
+    which = 0;
+    int m = LK / 2;
+#pragma unroll
+    for (int n = GQ; n > 1; n >>= 1, m >>= 1) {
+        const bool up = lane & m;
+#pragma unroll
+        for (int i = 0; i < n / 2; ++i) {
+            const float send = up ? s[i] : s[i + n / 2], keep = up ? s[i + n / 2] : s[i];
+            s[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
+        }
+        if (up) which += n / 2;
+    }
+#pragma unroll
+    for (; m > 0; m >>= 1) s[0] += __shfl_xor_sync(0xffffffffu, s[0], m);
+    return s[0];
+}
+
+// mma.sync pieces: 8 x 8 tiles of bf16 from shared memory, 16 x 8 x 16 products, 16-byte asynchronous copies
+__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
+}
+__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
+    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
+                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
+}
+__device__ __forceinline__ void cp16(void* dst, const void* src) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
 }
 
 template <typename K, typename A>

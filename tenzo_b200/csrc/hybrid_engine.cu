@@ -1,12 +1,15 @@
-// Hybrid decoders on the shared engine (hybrid_engine.h): configuration, weights, state and the walk through the layers.
+// Hybrid decoders on the shared engine (hybrid_engine.h): weights, state and the walk through the layers.
 //
 // One layer, M rows (decode: one per sequence; chunk: consecutive tokens of one sequence):
-//   rows     x += what the previous sublayer left, norm1, convolution (, token-shift mixes)
+//   rows     x += what the previous sublayer left (normed first, in some designs), norm1, convolution (, token-shift mixes)
 //   gemm     every projection of the mixer's input in one product
-//   window   convolution on q, k, v, ring update, attention          } whichever the mixer has
+//   window   convolution on q, k, v, ring update, attention          }
+//   latent   latent cache row, attention over latents or expanded     } whichever the mixer has
 //   scan     decays, recurrence, per-head norm, gate                  }
+//   delta    convolutions, delta rule, per-head norm, gate            }
 //   gemm     output projection(s)
-//   rows, gemm (+ activation), gemm    the feed-forward, when the layer has one
+//   rows, gemm (+ activation), gemm    the feed-forward, when the layer has one; a mixture of experts: rows, gemm (router),
+//                                      route, two grouped gemms
 // Residual sums happen at the start of the next row kernel.
 #include "hybrid_engine.h"
 
@@ -16,11 +19,9 @@
 
 namespace tz {
 
-static double softplus(double z) { return std::max(z, 0.0) + std::log1p(std::exp(-std::fabs(z))); }
-
-HybridEngine::HybridEngine(const Json& config, const OpenOptions& o) {
+HybridEngine::HybridEngine(const Json& config, const OpenOptions& o, Loader load) {
     try {
-        init(config, o);
+        init(config, o, load);
     } catch (...) {
         free_rows(dec);
         free_rows(chunk);
@@ -35,16 +36,10 @@ HybridEngine::~HybridEngine() {
     free_rows(chunk);
 }
 
-void HybridEngine::init(const Json& c, const OpenOptions& o) {
+void HybridEngine::init(const Json& c, const OpenOptions& o, Loader load) {
     f32 = o.compute == TENZO_COMPUTE_F32;
-    h = c.at("width").integer();
-    V = c.at("vocab").integer();
-    n_pos = c.at("max_positions").integer();
-    L = (int)c.at("layers").array().size();
-    eps = (float)c.at("norm").at("eps").number();
-    taps = c.at("canon").at("taps").integer();
-    if (h <= 0 || V <= 0 || n_pos <= 0 || L <= 0) throw std::invalid_argument("non-positive dimension");
-    if (taps < 1 || taps > kMaxTaps) throw std::invalid_argument("canon.taps is limited to 1..16");
+    init_core(o.opt.batch, o.opt.use_graph, o.opt.use_pdl);
+    (this->*load)(c, SafeTensors(o.dir + "/model.safetensors"));
     cfg = {};
     cfg.hidden_size = h;
     cfg.vocab_size = V;
@@ -52,9 +47,26 @@ void HybridEngine::init(const Json& c, const OpenOptions& o) {
     cfg.max_seq_len = n_pos;
     cfg.kv_mode = f32 ? "window_f32" : "window_bf16";
     cfg.device = "cuda";
-    init_core(o.opt.batch, o.opt.use_graph, o.opt.use_pdl);
     init_core_buffers();
-    load(c, o.dir);
+    tail_floats = std::max<size_t>(tail_floats, 4);
+    state_floats = std::max<size_t>(state_floats, 4);
+    for (const HybridLayer& y : layers) {
+        if (y.has_window) max_mix = std::max(max_mix, y.win.o.ld_k);
+        if (y.has_scan) max_mix = std::max(max_mix, y.scan.o.ld_k);
+        if (y.has_delta) max_mix = std::max(max_mix, y.delta.o.ld_k);
+        if (y.has_latent) {
+            max_mix = std::max(max_mix, y.lat.o.ld_k);
+            max_lat = std::max(max_lat, (size_t)y.lat.heads * caches[y.lat.cache].ld_c());
+        }
+        if (y.moe.experts) {
+            max_top = std::max(max_top, y.moe.top);
+            max_experts = std::max(max_experts, y.moe.experts);
+            max_expert_ff = std::max(max_expert_ff, y.moe.down.ld_k);
+            max_proj = std::max(max_proj, round_up(y.moe.experts, 8));
+        } else if (y.has_mlp) {
+            max_ff = std::max(max_ff, y.down.ld_k);
+        }
+    }
 
     const size_t B = batch, es = f32 ? 4 : 2;
     tails = (float*)dalloc(B * tail_floats * 4);
@@ -68,9 +80,23 @@ void HybridEngine::init(const Json& c, const OpenOptions& o) {
         m.ring_k = dalloc(B * m.ring_k_stride * es);
         m.ring_v = dalloc(B * m.ring_v_stride * es);
     }
+    int n_lin = 1;                                     // chunk buffers: 0 is shared by the caches that nobody borrows
+    for (LatentCache& k : caches) {
+        k.ring_c_stride = (size_t)k.ring * k.ld_c();
+        k.ring_r_stride = (size_t)k.ring * k.rot8();
+        k.ring_c = dalloc(B * k.ring_c_stride * es);
+        k.ring_r = dalloc(B * k.ring_r_stride * es);
+        k.lin = k.borrowed ? n_lin++ : 0;
+    }
+    lin_c.assign(caches.empty() ? 0 : n_lin, nullptr);
+    lin_r = lin_c;
     gemm_ws = dalloc(tenzo_cuda_gemm_workspace_bytes());
     argmax_ws = dalloc(argmax_scratch_bytes(batch));
     alloc_rows(dec, batch);
+    if (max_lat) {
+        dec.q_abs = (float*)dalloc(B * max_lat * 4);
+        dec.lat = dalloc(B * max_lat * es);
+    }
     b_x = dec.x;
     TZ_CUDA(cudaStreamSynchronize(stream));
 }
@@ -102,171 +128,40 @@ float* HybridEngine::conv_weights(const SafeTensors& st, const std::string& name
     return upload_floats(t);
 }
 
-void HybridEngine::read_window(WindowMixer& m, const Json& mix) {
-    m.heads = mix.at("heads").integer();
-    m.kv_heads = mix.at("kv_heads").integer();
-    m.dim = mix.at("dim").integer();
-    m.vdim = mix.at("vdim").integer();
-    m.taps = mix.at("conv").integer();
-    m.window = mix.at("mask").at("size").integer();
-    m.scale = (float)mix.at("scale").number();
-    if (m.heads < 1 || m.kv_heads < 1 || m.heads % m.kv_heads) throw std::invalid_argument("heads must be a multiple of kv_heads");
-    if (m.dim < 1 || m.dim > kMaxHeadDim || m.vdim < 1 || m.vdim > kMaxHeadDim) throw std::invalid_argument("attention head sizes are limited to 256");
-    if (m.taps < 1 || m.taps > kMaxTaps || m.window < 1) throw std::invalid_argument("bad convolution or window size");
-    m.ring = std::min(m.window, n_pos);
+size_t HybridEngine::take_tail(size_t floats) {
+    const size_t at = tail_floats;
+    tail_floats += (floats + 3) / 4 * 4;
+    return at;
 }
 
-static void read_scan(ScanMixer& m, const Json& mix, bool square) {
-    m.heads = mix.at("heads").integer();
-    m.dim = mix.at("dim").integer();
-    m.vdim = square ? m.dim : mix.at("vdim").integer();
-    if (m.heads < 1 || m.dim < 1 || m.dim > kMaxHeadDim || m.vdim < 1 || m.vdim > kMaxHeadDim)
-        throw std::invalid_argument("recurrent head sizes are limited to 256");
+size_t HybridEngine::take_state(size_t floats) {
+    const size_t at = state_floats;
+    state_floats += (floats + 3) / 4 * 4;
+    return at;
 }
 
-void HybridEngine::load(const Json& c, const std::string& dir) {
-    const SafeTensors st(dir + "/model.safetensors");
-    const int W = h;
-    embed = (bf16*)upload(st.bf16("embed", {V, W}).data, (size_t)V * W * 2);
-    pos_table = (bf16*)upload(st.bf16("pos", {n_pos, W}).data, (size_t)n_pos * W * 2);
-    final_gain = st.floats("final.norm", {})[0];
-    head = make_weight(V, W);
-    upload_weight(head, 0, st, "head", V, W);
-
-    size_t tail = 0, state = 0;
-    auto take = [](size_t& at, size_t n) {
-        const size_t a = at;
-        at += (n + 3) / 4 * 4;                    // 16-byte pieces
-        return a;
-    };
-    max_in = round_up(W, 64);
-    const auto& list = c.at("layers").array();
+void HybridEngine::start_layers(int n) {
+    L = n;
+    if (h <= 0 || V <= 0 || n_pos <= 0 || L <= 0) throw std::invalid_argument("non-positive dimension");
     layers.resize(L);
-    for (int l = 0; l < L; ++l) {
-        HybridLayer& y = layers[l];
-        const Json& e = list[l];
-        const std::string p = "l" + std::to_string(l) + ".", mp = p + "mix.", type = e.at("type").string();
-        const Json& mix = e.at("mixer");
-        y.norm1 = st.floats(p + "norm1", {})[0];
-        y.canon1 = conv_weights(st, p + "canon1", W, taps);
-        y.tail1 = take(tail, (size_t)(taps - 1) * W);
+    max_in = round_up(h, 64);
+}
 
-        // the fused input projection: (tensor, rows, where its column goes), pieces at multiples of `align` columns
-        struct Piece { std::string name; int rows; int* off; };
-        std::vector<Piece> pieces;
-        int align = 8;
-        auto scan_common = [&](const std::string& pre) {
-            ScanMixer& s = y.scan;
-            y.has_scan = true;
-            s.state = take(state, (size_t)s.heads * s.dim * round_up(s.vdim, 4));
-            s.o = make_weight(W, s.heads * s.vdim);
-            upload_weight(s.o, 0, st, pre + "o", W, s.heads * s.vdim);
-        };
-        auto low_rank = [&](const std::string& down, const std::string& up_name, const std::string& bias) {
-            ScanMixer& s = y.scan;
-            s.rank = (int)st.bf16(down, {-1, W}).shape[0];
-            const int n = s.heads * s.dim;
-            s.up = (bf16*)dalloc((size_t)n * round_up(s.rank, 8) * 2);
-            TZ_CUDA(cudaMemcpy2DAsync(s.up, (size_t)round_up(s.rank, 8) * 2, st.bf16(up_name, {n, s.rank}).data, (size_t)s.rank * 2, (size_t)s.rank * 2,
-                                      (size_t)n, cudaMemcpyHostToDevice, stream));
-            TZ_CUDA(cudaStreamSynchronize(stream));
-            s.bias = upload_floats(st.floats(bias, {n}));
-        };
-        if (type == "retention") {
-            ScanMixer& s = y.scan;
-            read_scan(s, mix, false);
-            s.k_scale = (float)std::pow((double)s.dim, -0.5);
-            s.decay_kind = TENZO_DECAY_CONST;
-            std::vector<float> d;
-            for (const Json& v : mix.at("decay").array()) d.push_back((float)v.number());
-            if ((int)d.size() != s.heads) throw std::invalid_argument("'decay' needs one entry per head");
-            s.decay = upload_floats(d);
-            scan_common(mp);
-            pieces = {{mp + "q", s.heads * s.dim, &s.off_q}, {mp + "k", s.heads * s.dim, &s.off_k},
-                      {mp + "v", s.heads * s.vdim, &s.off_v}, {mp + "g", s.heads * s.vdim, &s.off_g}};
-        } else if (type == "wkv") {
-            ScanMixer& s = y.scan;
-            read_scan(s, mix, true);
-            s.decay_kind = TENZO_DECAY_EXP_EXP;
-            low_rank(mp + "w1", mp + "w2", mp + "w0");
-            s.bonus = upload_floats(st.floats(mp + "u", {s.heads, s.dim}));
-            s.norm = upload_floats(st.floats(mp + "norm", {s.heads * s.vdim}));
-            s.norm_per_head = 1;
-            scan_common(mp);
-            const int n = s.heads * s.dim;
-            pieces = {{mp + "r", n, &s.off_q}, {mp + "k", n, &s.off_k}, {mp + "v", n, &s.off_v}, {mp + "g", n, &s.off_g}, {mp + "w1", s.rank, &s.off_low}};
-            align = 128;                           // each piece multiplies its own mix: a segment of the product
-            y.n_mix = 5;
-            std::vector<float> mu;
-            for (const char* m : {"r", "k", "v", "g", "w"}) {
-                const std::vector<float> v = st.floats(mp + "mu." + m, {W});
-                mu.insert(mu.end(), v.begin(), v.end());
-            }
-            y.mu = upload_floats(mu);
-            y.prev = take(tail, W);
-        } else if (type == "parallel") {
-            WindowMixer& m = y.win;
-            y.has_window = true;
-            read_window(m, mix.at("left"));
-            const std::string lp = mp + "left.", rp = mp + "right.";
-            m.conv_q = conv_weights(st, lp + "q.conv", m.heads * m.dim, m.taps);
-            m.conv_k = conv_weights(st, lp + "k.conv", m.kv_heads * m.dim, m.taps);
-            m.conv_v = conv_weights(st, lp + "v.conv", m.kv_heads * m.vdim, m.taps);
-            m.tail = take(tail, (size_t)(m.taps - 1) * m.channels());
-            m.o = make_weight(W, m.heads * m.vdim);
-            upload_weight(m.o, 0, st, lp + "o", W, m.heads * m.vdim);
-            ScanMixer& s = y.scan;
-            read_scan(s, mix.at("right"), false);
-            s.q_scale = (float)std::pow((double)s.dim, -0.5);
-            s.decay_kind = TENZO_DECAY_SIGMOID_ROOT;
-            s.tau = (float)mix.at("right").at("tau").number();
-            low_rank(rp + "a1", rp + "a2", rp + "a2.b");
-            s.norm = upload_floats(st.floats(rp + "norm", {s.vdim}));
-            scan_common(rp);
-            y.left_out = upload_floats(st.floats(lp + "out", {W}));
-            y.right_out = upload_floats(st.floats(rp + "out", {W}));
-            pieces = {{lp + "q", m.heads * m.dim, &m.off_q}, {lp + "k", m.kv_heads * m.dim, &m.off_k}, {lp + "v", m.kv_heads * m.vdim, &m.off_v},
-                      {rp + "q", s.heads * s.dim, &s.off_q}, {rp + "k", s.heads * s.dim, &s.off_k}, {rp + "v", s.heads * s.vdim, &s.off_v},
-                      {rp + "g", s.heads * s.vdim, &s.off_g}, {rp + "a1", s.rank, &s.off_low}};
-        } else {
-            throw std::invalid_argument("layer " + std::to_string(l) + ": unknown type '" + type + "'");
-        }
-        int n = 0;
-        y.n_seg = 0;
-        for (size_t i = 0; i < pieces.size(); ++i) {
-            *pieces[i].off = n;
-            n += i + 1 < pieces.size() ? round_up(pieces[i].rows, align) : pieces[i].rows;
-            if (y.n_mix) y.seg_end[y.n_seg++] = n;
-        }
-        if (!y.n_mix) y.seg_end[y.n_seg++] = n;
-        y.in = make_weight(n, W);
-        for (const Piece& q : pieces) upload_weight(y.in, *q.off, st, q.name, q.rows, W);
-        max_proj = std::max(max_proj, round_up(n, 8));
-        max_seg = std::max(max_seg, std::max(1, y.n_mix));
-        if (y.has_window) max_mix = std::max(max_mix, y.win.o.ld_k);
-        if (y.has_scan) max_mix = std::max(max_mix, y.scan.o.ld_k);
-
-        if (!e.at("mlp").is_null()) {
-            const Json& mlp = e.at("mlp");
-            if (mlp.at("kind").string() != "dense") throw std::invalid_argument("layer " + std::to_string(l) + ": unknown feed-forward '" + mlp.at("kind").string() + "'");
-            const int ff = mlp.at("ff").integer();
-            if (ff < 1) throw std::invalid_argument("non-positive dimension");
-            y.has_mlp = true;
-            y.norm2 = st.floats(p + "norm2", {})[0];
-            y.canon2 = conv_weights(st, p + "canon2", W, taps);
-            y.tail2 = take(tail, (size_t)(taps - 1) * W);
-            y.up = make_weight(ff, W);
-            upload_weight(y.up, 0, st, p + "mlp.up", ff, W);
-            y.down = make_weight(W, ff);
-            upload_weight(y.down, 0, st, p + "mlp.down", W, ff);
-            const std::vector<float> act = st.floats(p + "mlp.act", {2});
-            y.act_pos = (float)softplus(act[0]);
-            y.act_neg = (float)(0.5 + softplus(act[1]));
-            max_ff = std::max(max_ff, y.down.ld_k);
-        }
+// Every projection of a mixer's input as one product, pieces at multiples of `align` columns. With mixes each piece multiplies
+// its own one: a segment of the product.
+void HybridEngine::fuse_inputs(HybridLayer& y, const std::vector<Piece>& pieces, int align, const SafeTensors& st) {
+    int n = 0;
+    y.n_seg = 0;
+    for (size_t i = 0; i < pieces.size(); ++i) {
+        *pieces[i].off = n;
+        n += i + 1 < pieces.size() ? round_up(pieces[i].rows, align) : pieces[i].rows;
+        if (y.n_mix) y.seg_end[y.n_seg++] = n;
     }
-    tail_floats = std::max<size_t>(tail, 4);
-    state_floats = std::max<size_t>(state, 4);
+    if (!y.n_mix) y.seg_end[y.n_seg++] = n;
+    y.in = make_weight(n, h);
+    for (const Piece& q : pieces) upload_weight(y.in, *q.off, st, q.name, q.rows, h);
+    max_proj = std::max(max_proj, round_up(n, 8));
+    max_seg = std::max(max_seg, std::max(1, y.n_mix));
 }
 
 // ---- activations ------------------------------------------------------------------------------------------------------------
@@ -294,6 +189,17 @@ void HybridEngine::alloc_rows(Rows& r, int cap) {
     r.act = get(m * max_ff * es);
     r.ya = (float*)get(m * h * 4);
     r.yb = (float*)get(m * h * 4);
+    if (max_top) {
+        const size_t pairs = m * max_top;
+        r.chosen = (int*)get(pairs * 4);
+        r.slot = (int*)get(pairs * 4);
+        r.row_of = (int*)get(pairs * 4);
+        r.group_off = (int*)get((max_experts + 1) * 4);
+        r.weight = (float*)get(pairs * 4);
+        r.ye = (float*)get(pairs * h * 4);
+        r.act_e = get(pairs * max_expert_ff * es);
+        if (!f32) r.gathered = get(pairs * max_in * es);
+    }
     r.cap = cap;
 }
 
@@ -316,9 +222,9 @@ void HybridEngine::set_seq_len(int s, int len) {
 }
 
 // ---- one walk through the layers ---------------------------------------------------------------------------------------------
-RowsArgs HybridEngine::row_args(Pass& p, float gain, const float* conv, size_t tail) {
+RowsArgs HybridEngine::row_args(Pass& p, float gain, const float* gain_w, const float* conv, size_t tail) {
     RowsArgs a;
-    a.width = h; a.M = p.M; a.eps = eps; a.gain = gain;
+    a.width = h; a.M = p.M; a.eps = eps; a.gain = gain; a.gain_w = gain_w;
     a.conv_w = conv; a.taps = conv ? taps : 1;
     float* carried = tails + (size_t)p.seq * tail_floats + tail;
     a.tail_in = carried;
@@ -339,6 +245,7 @@ void HybridEngine::run_rows(Pass& p, RowsArgs& a) {
     } else {
         a.x_in = p.rows->x;
         a.y0 = p.add.y0; a.y1 = p.add.y1; a.w0 = p.add.w0; a.w1 = p.add.w1;
+        a.y_slot = p.add.slot; a.y_weight = p.add.weight; a.n_y = p.add.n_y;
         a.ld_y = h;
     }
     p.add = Pending();
@@ -347,27 +254,130 @@ void HybridEngine::run_rows(Pass& p, RowsArgs& a) {
     TZ_KERNEL(launch_rows(a, stream, &launches));
 }
 
-void HybridEngine::run_gemm(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c, const HybridLayer* mixes, const HybridLayer* act) {
+GemmArgs HybridEngine::gemm_args(Pass& p, const void* a, const DenseWeight& w, void* c, int ld_c) {
     GemmArgs g;
     g.a = a; g.w = w.w; g.M = p.M; g.N = w.rows; g.ld_k = w.ld_k;
     g.seg_end[0] = w.rows;
-    if (mixes) {
-        g.n_seg = mixes->n_seg;
-        std::copy(mixes->seg_end, mixes->seg_end + 8, g.seg_end);
-        g.a_seg_stride = (size_t)p.M * w.ld_k;
-    }
-    if (act) { g.epilogue = TENZO_GEMM_XIELU; g.act_pos = act->act_pos; g.act_neg = act->act_neg; }
     g.c = c; g.ld_c = ld_c;
     g.f32 = f32; g.use_pdl = p.decode && use_pdl;
     g.workspace = gemm_ws; g.workspace_bytes = tenzo_cuda_gemm_workspace_bytes();
-    TZ_KERNEL(launch_gemm(g, stream));
-    launches += p.M > 8 && p.M < kGemmUmmaMinRows && !f32 ? 2 : 1;
+    return g;
+}
+
+void HybridEngine::run_gemm(const GemmArgs& g) { TZ_KERNEL(launch_gemm(g, stream, &launches)); }
+
+void HybridEngine::run_window(Pass& p, HybridLayer& y) {
+    Rows& r = *p.rows;
+    const WindowMixer& m = y.win;
+    WindowAttnArgs a;
+    a.q = r.proj + m.off_q; a.k = r.proj + m.off_k; a.v = r.proj + m.off_v; a.ld = max_proj;
+    a.conv_q = m.conv_q; a.conv_k = m.conv_k; a.conv_v = m.conv_v; a.taps = m.taps;
+    float* carried = tails + (size_t)p.seq * tail_floats + m.tail;
+    a.tail_in = carried;
+    a.tail_out = p.decode ? carried : tail_stage + m.tail;
+    a.tail_seq_stride = tail_floats;
+    a.heads = m.heads; a.kv_heads = m.kv_heads; a.dim = m.dim; a.vdim = m.vdim; a.scale = m.scale;
+    a.window = m.window; a.ring = m.ring;
+    const size_t es = f32 ? 4 : 2;
+    a.ring_k = static_cast<char*>(m.ring_k) + (size_t)p.seq * m.ring_k_stride * es;
+    a.ring_v = static_cast<char*>(m.ring_v) + (size_t)p.seq * m.ring_v_stride * es;
+    a.ring_k_stride = m.ring_k_stride; a.ring_v_stride = m.ring_v_stride;
+    a.pos = p.pos; a.pos0 = p.pos0; a.M = p.M; a.decode = p.decode;
+    a.out = r.mix_a; a.ld_out = m.o.ld_k;
+    a.lin_q = lin_q; a.lin_k = lin_k; a.lin_v = lin_v;
+    a.f32 = f32; a.use_pdl = p.decode && use_pdl;
+    TZ_KERNEL(launch_window_attention(a, stream, &launches));
+}
+
+void HybridEngine::run_scan(Pass& p, HybridLayer& y) {
+    Rows& r = *p.rows;
+    const ScanMixer& m = y.scan;
+    ScanArgs a;
+    a.q = r.proj + m.off_q; a.k = r.proj + m.off_k; a.v = r.proj + m.off_v; a.g = r.proj + m.off_g; a.ld = max_proj;
+    a.q_scale = m.q_scale; a.k_scale = m.k_scale;
+    a.heads = m.heads; a.dim = m.dim; a.vdim = m.vdim;
+    a.decay_kind = m.decay_kind; a.decay = m.decay;
+    a.low = r.proj + m.off_low; a.up = m.up; a.bias = m.bias; a.rank = m.rank; a.tau = m.tau;
+    a.bonus = m.bonus; a.norm = m.norm; a.norm_per_head = m.norm_per_head; a.eps = eps;
+    a.state = states + (size_t)p.seq * state_floats + m.state;
+    a.state_seq_stride = state_floats;
+    a.M = p.M; a.decode = p.decode;
+    a.out = y.has_window ? r.mix_b : r.mix_a; a.ld_out = m.o.ld_k;
+    a.w_rows = w_rows; a.o_rows = o_rows; a.part = scan_part;
+    a.f32 = f32; a.use_pdl = p.decode && use_pdl;
+    TZ_KERNEL(launch_scan(a, stream, &launches));
+}
+
+void HybridEngine::run_delta(Pass& p, HybridLayer& y) {
+    Rows& r = *p.rows;
+    const DeltaMixer& m = y.delta;
+    DeltaArgs a;
+    a.q = r.proj + m.off_q; a.k = r.proj + m.off_k; a.v = r.proj + m.off_v; a.g = r.proj + m.off_g; a.a = r.proj + m.off_a; a.b = r.proj + m.off_b;
+    a.ld = max_proj;
+    a.conv_q = m.conv_q; a.conv_k = m.conv_k; a.conv_v = m.conv_v; a.taps = m.taps;
+    float* slot = states + (size_t)p.seq * state_floats;
+    a.tail = slot + m.tail; a.tail_seq_stride = state_floats;
+    a.heads = m.heads; a.kv_heads = m.kv_heads; a.dim = m.dim; a.vdim = m.vdim;
+    a.q_scale = (float)std::pow((double)m.dim, -0.5);
+    a.a_log = m.a_log; a.dt_bias = m.dt_bias; a.norm = m.norm; a.eps = eps;
+    a.state = slot + m.state; a.state_seq_stride = state_floats;
+    a.pos = p.pos; a.pos0 = p.pos0; a.M = p.M; a.decode = p.decode;
+    a.out = r.mix_a; a.ld_out = m.o.ld_k;
+    a.work = delta_work;
+    a.f32 = f32; a.use_pdl = p.decode && use_pdl;
+    TZ_KERNEL(launch_delta(a, stream, &launches));
+}
+
+void HybridEngine::run_latent(Pass& p, HybridLayer& y) {
+    Rows& r = *p.rows;
+    const LatentMixer& m = y.lat;
+    const LatentCache& k = caches[m.cache];
+    LatentAttnArgs a;
+    a.q = r.proj + m.off_q; a.dkv = m.owner ? r.proj + m.off_dkv : nullptr; a.ld = max_proj;
+    a.norm = m.norm; a.eps = eps; a.freq = k.freq;
+    a.heads = m.heads; a.dim = m.dim; a.rot = k.rot; a.vdim = m.vdim; a.rank = k.rank;
+    a.scale = m.scale; a.window = m.window; a.w_kv = m.kv;
+    const size_t es = f32 ? 4 : 2;
+    a.ring_c = static_cast<char*>(k.ring_c) + (size_t)p.seq * k.ring_c_stride * es;
+    a.ring_r = static_cast<char*>(k.ring_r) + (size_t)p.seq * k.ring_r_stride * es;
+    a.ring = k.ring; a.ring_c_stride = k.ring_c_stride; a.ring_r_stride = k.ring_r_stride;
+    a.pos = p.pos; a.pos0 = p.pos0; a.M = p.M; a.decode = p.decode;
+    a.out = r.mix_a; a.ld_out = m.o.ld_k;
+    a.lin_q = lin_q; a.lin_c = lin_c[k.lin]; a.lin_r = lin_r[k.lin]; a.kv = lat_kv;
+    a.q_abs = r.q_abs; a.lat = r.lat;
+    a.workspace = gemm_ws; a.workspace_bytes = tenzo_cuda_gemm_workspace_bytes();
+    a.f32 = f32; a.use_pdl = p.decode && use_pdl;
+    TZ_KERNEL(launch_latent_attention(a, stream, &launches));
+}
+
+// The chosen experts of every row; their outputs are weighted and summed by the next row kernel.
+void HybridEngine::run_experts(Pass& p, HybridLayer& y) {
+    Rows& r = *p.rows;
+    const ExpertMlp& m = y.moe;
+    run_gemm(gemm_args(p, r.in, m.router, r.proj, max_proj));
+    RouteArgs a;
+    a.logits = r.proj; a.ld = max_proj; a.correction = m.correction;
+    a.experts = m.experts; a.top = m.top; a.M = p.M;
+    a.chosen = r.chosen; a.weight = r.weight; a.slot = r.slot; a.row_of = r.row_of; a.group_off = r.group_off;
+    a.use_pdl = p.decode && use_pdl;
+    TZ_KERNEL(launch_route(a, stream, &launches));
+    GemmArgs g = gemm_args(p, r.in, m.up, r.act_e, m.down.ld_k);
+    g.M = p.M * m.top; g.N = 2 * m.ff; g.seg_end[0] = g.N;
+    g.epilogue = TENZO_GEMM_GLU_SILU;
+    g.group_off = r.group_off; g.n_group = m.experts;
+    g.a_index = r.row_of; g.a_rows = p.M; g.a_gather = r.gathered;
+    run_gemm(g);
+    g = gemm_args(p, r.act_e, m.down, r.ye, h);
+    g.M = p.M * m.top; g.N = h; g.seg_end[0] = g.N;
+    g.group_off = r.group_off; g.n_group = m.experts;
+    run_gemm(g);
+    p.add.y0 = r.ye; p.add.slot = r.slot; p.add.weight = r.weight; p.add.n_y = m.top;
 }
 
 void HybridEngine::run_layer(Pass& p, int l) {
     HybridLayer& y = layers[l];
     Rows& r = *p.rows;
-    RowsArgs ra = row_args(p, y.norm1, y.canon1, y.tail1);
+    RowsArgs ra = row_args(p, y.norm1, y.norm1_w, y.canon1, y.tail1);
     if (y.n_mix) {
         ra.mu = y.mu; ra.n_mix = y.n_mix;
         float* carried = tails + (size_t)p.seq * tail_floats + y.prev;
@@ -375,71 +385,58 @@ void HybridEngine::run_layer(Pass& p, int l) {
         ra.prev_out = p.decode ? carried : tail_stage + y.prev;
     }
     run_rows(p, ra);
-    run_gemm(p, r.in, y.in, r.proj, max_proj, y.n_mix ? &y : nullptr);
-
-    if (y.has_window) {
-        const WindowMixer& m = y.win;
-        WindowAttnArgs a;
-        a.q = r.proj + m.off_q; a.k = r.proj + m.off_k; a.v = r.proj + m.off_v; a.ld = max_proj;
-        a.conv_q = m.conv_q; a.conv_k = m.conv_k; a.conv_v = m.conv_v; a.taps = m.taps;
-        float* carried = tails + (size_t)p.seq * tail_floats + m.tail;
-        a.tail_in = carried;
-        a.tail_out = p.decode ? carried : tail_stage + m.tail;
-        a.tail_seq_stride = tail_floats;
-        a.heads = m.heads; a.kv_heads = m.kv_heads; a.dim = m.dim; a.vdim = m.vdim; a.scale = m.scale;
-        a.window = m.window; a.ring = m.ring;
-        const size_t es = f32 ? 4 : 2;
-        a.ring_k = static_cast<char*>(m.ring_k) + (size_t)p.seq * m.ring_k_stride * es;
-        a.ring_v = static_cast<char*>(m.ring_v) + (size_t)p.seq * m.ring_v_stride * es;
-        a.ring_k_stride = m.ring_k_stride; a.ring_v_stride = m.ring_v_stride;
-        a.pos = p.pos; a.pos0 = p.pos0; a.M = p.M; a.decode = p.decode;
-        a.out = r.mix_a; a.ld_out = m.o.ld_k;
-        a.lin_q = lin_q; a.lin_k = lin_k; a.lin_v = lin_v;
-        a.f32 = f32; a.use_pdl = p.decode && use_pdl;
-        TZ_KERNEL(launch_window_attention(a, stream, &launches));
+    GemmArgs in = gemm_args(p, r.in, y.in, r.proj, max_proj);
+    if (y.n_mix) {
+        in.n_seg = y.n_seg;
+        std::copy(y.seg_end, y.seg_end + 8, in.seg_end);
+        in.a_seg_stride = (size_t)p.M * y.in.ld_k;
     }
-    void* scan_out = y.has_window ? r.mix_b : r.mix_a;
-    if (y.has_scan) {
-        const ScanMixer& m = y.scan;
-        ScanArgs a;
-        a.q = r.proj + m.off_q; a.k = r.proj + m.off_k; a.v = r.proj + m.off_v; a.g = r.proj + m.off_g; a.ld = max_proj;
-        a.q_scale = m.q_scale; a.k_scale = m.k_scale;
-        a.heads = m.heads; a.dim = m.dim; a.vdim = m.vdim;
-        a.decay_kind = m.decay_kind; a.decay = m.decay;
-        a.low = r.proj + m.off_low; a.up = m.up; a.bias = m.bias; a.rank = m.rank; a.tau = m.tau;
-        a.bonus = m.bonus; a.norm = m.norm; a.norm_per_head = m.norm_per_head; a.eps = eps;
-        a.state = states + (size_t)p.seq * state_floats + m.state;
-        a.state_seq_stride = state_floats;
-        a.M = p.M; a.decode = p.decode;
-        a.out = scan_out; a.ld_out = m.o.ld_k;
-        a.w_rows = w_rows; a.o_rows = o_rows; a.part = scan_part;
-        a.f32 = f32; a.use_pdl = p.decode && use_pdl;
-        TZ_KERNEL(launch_scan(a, stream, &launches));
-    }
+    run_gemm(in);
+    if (y.has_window) run_window(p, y);
+    if (y.has_scan) run_scan(p, y);
+    if (y.has_delta) run_delta(p, y);
+    if (y.has_latent) run_latent(p, y);
     if (y.has_window && y.has_scan) {
-        run_gemm(p, r.mix_a, y.win.o, r.ya, h);
-        run_gemm(p, r.mix_b, y.scan.o, r.yb, h);
+        run_gemm(gemm_args(p, r.mix_a, y.win.o, r.ya, h));
+        run_gemm(gemm_args(p, r.mix_b, y.scan.o, r.yb, h));
         p.add.y0 = r.ya; p.add.y1 = r.yb; p.add.w0 = y.left_out; p.add.w1 = y.right_out;
     } else {
-        run_gemm(p, r.mix_a, y.has_window ? y.win.o : y.scan.o, r.ya, h);
+        run_gemm(gemm_args(p, r.mix_a, y.has_window ? y.win.o : y.has_scan ? y.scan.o : y.has_delta ? y.delta.o : y.lat.o, r.ya, h));
+        p.add.y0 = r.ya; p.add.w0 = y.post1_w;
+    }
+    if (!y.has_mlp) return;
+    RowsArgs rb = row_args(p, y.norm2, y.norm2_w, y.canon2, y.tail2);
+    run_rows(p, rb);
+    if (y.moe.experts) {
+        run_experts(p, y);
+    } else {
+        GemmArgs up = gemm_args(p, r.in, y.up, r.act, y.down.ld_k);
+        up.epilogue = y.up_epilogue; up.act_pos = y.act_pos; up.act_neg = y.act_neg;
+        run_gemm(up);
+        run_gemm(gemm_args(p, r.act, y.down, r.ya, h));
         p.add.y0 = r.ya;
     }
-    if (y.has_mlp) {
-        RowsArgs rb = row_args(p, y.norm2, y.canon2, y.tail2);
-        run_rows(p, rb);
-        run_gemm(p, r.in, y.up, r.act, y.down.ld_k, nullptr, &y);
-        run_gemm(p, r.act, y.down, r.ya, h);
-        p.add.y0 = r.ya;
-    }
+    p.add.w0 = y.post2_w;
+}
+
+// Leaves the normalised rows in p.rows->in.
+void HybridEngine::run_final(Pass& p) {
+    RowsArgs ra = row_args(p, final_gain, final_gain_w, nullptr, 0);
+    run_rows(p, ra);
+}
+
+void HybridEngine::run_head(Pass& p, const void* rows, float* logits) {
+    GemmArgs g = gemm_args(p, rows, head, logits, V);
+    if (logit_cap > 0.0f) { g.epilogue = TENZO_GEMM_SOFTCAP; g.cap = logit_cap; }
+    run_gemm(g);
 }
 
 void HybridEngine::enqueue_step(bool with_logits, bool feed_back, int) {
     Pass p = {&dec, batch, 1, 0, 0, d_tokens, d_pos};
     for (int l = 0; l < L; ++l) run_layer(p, l);
-    RowsArgs ra = row_args(p, final_gain, nullptr, 0);
-    run_rows(p, ra);
+    run_final(p);
     if (with_logits) {
-        run_gemm(p, dec.in, head, b_logits, V);
+        run_head(p, dec.in, b_logits);
         TZ_KERNEL(launch_argmax(b_logits, V, batch, d_next, argmax_ws, stream));
         launches += 2;
     }
@@ -450,48 +447,70 @@ void HybridEngine::enqueue_layer(int l, int) {
     Pass p = {&dec, batch, 1, 0, 0, d_tokens, d_pos};
     p.embed = false;
     run_layer(p, l);
-    RowsArgs ra = row_args(p, 1.0f, nullptr, 0);
+    RowsArgs ra = row_args(p, 1.0f, nullptr, nullptr, 0);
     run_rows(p, ra);
 }
 
-void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
-    if (M > chunk.cap) {
-        int cap = 64;
-        while (cap < M) cap *= 2;
-        alloc_rows(chunk, cap);
-        chunk.cap = 0;                                 // until every buffer below exists too
-        const size_t m = cap, es = f32 ? 4 : 2;
-        auto get = [&](size_t bytes) -> void* {
-            void* p = nullptr;
-            TZ_CUDA(cudaMalloc(&p, bytes ? bytes : 16));
-            chunk.owned.push_back(p);
-            return p;
-        };
-        size_t lq = 0, lk = 0, lv = 0, w = 0, o = 0, part = 0;
-        for (const HybridLayer& y : layers) {
-            if (y.has_window) {
-                const WindowMixer& a = y.win;
-                lq = std::max(lq, m * a.heads * round_up(a.dim, 8));
-                lk = std::max(lk, (m + a.ring) * a.kv_heads * round_up(a.dim, 8));
-                lv = std::max(lv, (m + a.ring) * a.kv_heads * round_up(a.vdim, 8));
-            }
-            if (y.has_scan) {
-                const ScanMixer& s = y.scan;
-                if (s.decay_kind != TENZO_DECAY_CONST) w = std::max(w, m * s.heads * s.dim);
-                o = std::max(o, m * s.heads * s.vdim);
-                part = std::max(part, tenzo_cuda_linear_scan_part_floats(cap, s.heads, s.dim, s.vdim));
-            }
+// Activations and scratch of chunks of up to `rows` rows.
+void HybridEngine::grow_chunk(int rows) {
+    if (rows <= chunk.cap) return;
+    int cap = 64;
+    while (cap < rows) cap *= 2;
+    alloc_rows(chunk, cap);
+    chunk.cap = 0;                                     // until every buffer below exists too
+    const size_t m = cap, es = f32 ? 4 : 2;
+    auto get = [&](size_t bytes) -> void* {
+        void* p = nullptr;
+        TZ_CUDA(cudaMalloc(&p, bytes ? bytes : 16));
+        chunk.owned.push_back(p);
+        return p;
+    };
+    size_t lq = 0, lk = 0, lv = 0, w = 0, o = 0, part = 0, work = 0, kv = 0;
+    for (const HybridLayer& y : layers) {
+        if (y.has_window) {
+            const WindowMixer& a = y.win;
+            lq = std::max(lq, m * a.heads * round_up(a.dim, 8));
+            lk = std::max(lk, (m + a.ring) * a.kv_heads * round_up(a.dim, 8));
+            lv = std::max(lv, (m + a.ring) * a.kv_heads * round_up(a.vdim, 8));
         }
-        chunk_tokens = (int*)get(m * 4);
-        chunk_pos = (int*)get(m * 4);
-        lin_q = get(lq * es);
-        lin_k = get(lk * es);
-        lin_v = get(lv * es);
-        w_rows = (float*)get(w * 4);
-        o_rows = (float*)get(o * 4);
-        scan_part = (float*)get(part * 4);
-        chunk.cap = cap;
+        if (y.has_scan) {
+            const ScanMixer& s = y.scan;
+            if (s.decay_kind != TENZO_DECAY_CONST) w = std::max(w, m * s.heads * s.dim);
+            o = std::max(o, m * s.heads * s.vdim);
+            part = std::max(part, tenzo_cuda_linear_scan_part_floats(cap, s.heads, s.dim, s.vdim));
+        }
+        if (y.has_delta) work = std::max(work, tenzo_cuda_delta_rule_work_floats(cap, y.delta.heads, y.delta.kv_heads, y.delta.dim, y.delta.vdim));
+        if (y.has_latent) {
+            const LatentMixer& a = y.lat;
+            lq = std::max(lq, m * a.heads * (a.dim8() + caches[a.cache].rot8()));
+            kv = std::max(kv, (m + std::min(a.window, n_pos)) * a.heads * (a.dim8() + a.vdim8()));
+        }
     }
+    chunk_tokens = (int*)get(m * 4);
+    chunk_pos = (int*)get(m * 4);
+    lin_q = get(lq * es);
+    lin_k = get(lk * es);
+    lin_v = get(lv * es);
+    w_rows = (float*)get(w * 4);
+    o_rows = (float*)get(o * 4);
+    scan_part = (float*)get(part * 4);
+    delta_work = (float*)get(work * 4);
+    lat_kv = get(kv * es);
+    for (size_t i = 0; i < lin_c.size(); ++i) {
+        size_t c = 0, r = 0;
+        for (const LatentCache& k : caches)
+            if (k.lin == (int)i) {
+                c = std::max(c, (m + k.ring) * k.ld_c());
+                r = std::max(r, (m + k.ring) * k.rot8());
+            }
+        lin_c[i] = get(c * es);
+        lin_r[i] = get(r * es);
+    }
+    chunk.cap = cap;
+}
+
+void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
+    grow_chunk(M);
     const int pos0 = seq_len[seq];
     std::vector<int> hp(M);
     for (int i = 0; i < M; ++i) hp[i] = pos0 + i;
@@ -499,8 +518,7 @@ void HybridEngine::chunk_rows(int seq, const int* tokens, int M) {
     TZ_CUDA(cudaMemcpyAsync(chunk_pos, hp.data(), (size_t)M * 4, cudaMemcpyHostToDevice, stream));
     Pass p = {&chunk, M, 0, seq, pos0, chunk_tokens, chunk_pos};
     for (int l = 0; l < L; ++l) run_layer(p, l);
-    RowsArgs ra = row_args(p, final_gain, nullptr, 0);
-    run_rows(p, ra);                                   // leaves the normalised rows for rows_logits in chunk.in
+    run_final(p);                                      // for rows_logits
     TZ_CUDA(cudaMemcpyAsync(tails + (size_t)seq * tail_floats, tail_stage, tail_floats * 4, cudaMemcpyDeviceToDevice, stream));
     TZ_CUDA(cudaMemcpyAsync(dec.x + (size_t)seq * h, chunk.x + (size_t)(M - 1) * h, (size_t)h * 4, cudaMemcpyDeviceToDevice, stream));
     TZ_CUDA(cudaStreamSynchronize(stream));
@@ -525,7 +543,7 @@ void HybridEngine::rows_logits(const int* want, int n_want, float* host) {
             i = j;
         }
         Pass p = {&chunk, n, 0, 0, 0, nullptr, nullptr};
-        run_gemm(p, logit_in, head, want_logits, V);
+        run_head(p, logit_in, want_logits);
         TZ_CUDA(cudaMemcpyAsync(host + (size_t)a * V, want_logits, (size_t)n * V * 4, cudaMemcpyDeviceToHost, stream));
     }
     TZ_CUDA(cudaStreamSynchronize(stream));
@@ -544,8 +562,5 @@ void HybridEngine::check_device_status(bool force) {
     if (!force && batch == 1 && (++status_poll & 31) != 0) return;
     if (tenzo_cuda_gemm_take_timeouts() > 0) throw std::runtime_error("a matrix product gave up waiting for a tile copy; results are invalid");
 }
-
-static EngineCore* open_sozopel(const Json& config, const OpenOptions& o) { return new HybridEngine(config, o); }
-static const ModelRegistration registration({"Sozopel", open_sozopel});
 
 }  // namespace tz

@@ -341,6 +341,14 @@ __global__ void __launch_bounds__(256) scan_gate_kernel(const ScanArgs a) {
     }
 }
 
+int launch_scan_gate(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
+    const unsigned ctas = (unsigned)(((size_t)a.M * a.heads + 7) / 8);
+    if (a.f32) scan_gate_kernel<float><<<ctas, 256, 0, st>>>(a);
+    else scan_gate_kernel<bf16><<<ctas, 256, 0, st>>>(a);
+    *n_kernels += 1;
+    return (int)cudaGetLastError();
+}
+
 int launch_scan(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
     if (a.M <= 0) return 0;
     if (a.dim < 1 || a.dim > kMaxHeadDim || a.vdim < 1 || a.vdim > kMaxHeadDim || a.heads < 1) return -1;
@@ -387,11 +395,8 @@ int launch_scan(const ScanArgs& a, cudaStream_t st, unsigned long long* n_kernel
     const int rc = a.dim <= 32 ? sized(std::integral_constant<int, 2>()) : a.dim <= 64 ? sized(std::integral_constant<int, 4>())
                  : a.dim <= 128 ? sized(std::integral_constant<int, 8>()) : sized(std::integral_constant<int, 16>());
     if (rc) return rc;
-    const unsigned gate_ctas = (unsigned)(((size_t)a.M * a.heads + 7) / 8);
-    if (a.f32) scan_gate_kernel<float><<<gate_ctas, 256, 0, st>>>(p);
-    else scan_gate_kernel<bf16><<<gate_ctas, 256, 0, st>>>(p);
-    *n_kernels += 4;
-    return (int)cudaGetLastError();
+    *n_kernels += 3;
+    return launch_scan_gate(p, st, n_kernels);
 }
 
 }  // namespace tz

@@ -1,8 +1,9 @@
-// Row kernels of the hybrid decoders: residual update, RMS norm with one gain, causal convolution over time on every
-// channel, and the token-shift mixes of a time-mixing layer (tenzo_rows_args).
+// Row kernels of the hybrid decoders: residual update, RMS norm with one gain or a gain per channel, causal convolution over
+// time on every channel, and the token-shift mixes of a time-mixing layer (tenzo_rows_args).
 //
-// Decode: one CTA per sequence does all of it; a thread keeps its columns in registers, with the convolution's weights and
-// the carried inputs fetched before the kernel waits for its producer (the launch that wrote them lies a whole step back).
+// Decode, and rows that carry nothing from one to the next: one CTA per row does all of it; a thread keeps its columns in
+// registers, with the convolution's weights and the carried inputs fetched before the kernel waits for its producer (the
+// launch that wrote them lies a whole step back).
 // Chunk (and decode of rows wider than that): one kernel updates the residual and leaves each row's inverse RMS, a second
 // one walks tiles of rows per channel with the convolution's inputs in registers.
 #include "hybrid_common.cuh"
@@ -26,22 +27,37 @@ __device__ __forceinline__ float2 block_sum2(float2 v, float2* scratch) {
 struct RowSource {                              // where a row's residual comes from
     const RowsArgs& a;
     const bf16 *e = nullptr, *p = nullptr;
-    const float *x = nullptr, *y0 = nullptr, *y1 = nullptr;
+    const float *x = nullptr, *y0 = nullptr, *y1 = nullptr, *yw = nullptr;
+    const int* ys = nullptr;
+    bool normed = false;                        // the addends are normed
     __device__ __forceinline__ RowSource(const RowsArgs& args, int t) : a(args) {
         if (a.tokens) {
-            const int tok = min(max(a.tokens[t], 0), a.vocab - 1), pos = min(max(a.pos[t], 0), a.n_pos - 1);
+            const int tok = min(max(a.tokens[t], 0), a.vocab - 1);
             e = static_cast<const bf16*>(a.embed) + (size_t)tok * a.width;
-            p = static_cast<const bf16*>(a.pos_table) + (size_t)pos * a.width;
+            if (a.pos_table) p = static_cast<const bf16*>(a.pos_table) + (size_t)min(max(a.pos[t], 0), a.n_pos - 1) * a.width;
         } else {
             x = a.x_in + (size_t)t * a.width;
-            y0 = a.y0 ? a.y0 + (size_t)t * a.ld_y : nullptr;
             y1 = a.y1 ? a.y1 + (size_t)t * a.ld_y : nullptr;
+            normed = a.w0 != nullptr;
+            if (a.y_slot) {
+                ys = a.y_slot + (size_t)t * a.n_y;
+                yw = a.y_weight + (size_t)t * a.n_y;
+                y0 = a.y0;
+            } else if (a.y0) {
+                y0 = a.y0 + (size_t)t * a.ld_y;
+            }
         }
     }
-    // without the two normed addends
+    __device__ __forceinline__ float first(int c) const {
+        if (!ys) return y0[c];
+        float v = 0.0f;
+        for (int j = 0; j < a.n_y; ++j) v = fmaf(yw[j], y0[(size_t)ys[j] * a.ld_y + c], v);
+        return v;
+    }
+    // without normed addends
     __device__ __forceinline__ float plain(int c) const {
-        if (e) return to_f(e[c]) + to_f(p[c]);
-        return y0 && !y1 ? x[c] + y0[c] : x[c];
+        if (e) return p ? to_f(e[c]) + to_f(p[c]) : to_f(e[c]);
+        return y0 && !normed ? x[c] + first(c) : x[c];
     }
 };
 
@@ -75,20 +91,24 @@ __global__ void __launch_bounds__(kStepThreads) rows_step_kernel(const RowsArgs 
         x[i] = l[i] = r[i] = 0.0f;
         if (c >= width) continue;
         x[i] = src.plain(c);
-        if (src.y1) {
-            l[i] = src.y0[c];
-            r[i] = src.y1[c];
+        if (src.normed) {
+            l[i] = src.first(c);
             q.x = fmaf(l[i], l[i], q.x);
-            q.y = fmaf(r[i], r[i], q.y);
+            if (src.y1) {
+                r[i] = src.y1[c];
+                q.y = fmaf(r[i], r[i], q.y);
+            }
         }
     }
-    if (src.y1) {
+    if (src.normed) {
         q = block_sum2(q, s_red[0]);
         const float i0 = 1.0f / sqrtf(q.x / (float)width + a.eps), i1 = 1.0f / sqrtf(q.y / (float)width + a.eps);
 #pragma unroll
         for (int i = 0; i < CPT; ++i) {
             const int c = threadIdx.x + i * kStepThreads;
-            if (c < width) x[i] += 0.5f * (l[i] * i0 * a.w0[c] + r[i] * i1 * a.w1[c]);
+            if (c >= width) continue;
+            const float v = l[i] * i0 * a.w0[c];
+            x[i] += src.y1 ? 0.5f * (v + r[i] * i1 * a.w1[c]) : v;
         }
     }
     q = make_float2(0.0f, 0.0f);
@@ -106,7 +126,7 @@ __global__ void __launch_bounds__(kStepThreads) rows_step_kernel(const RowsArgs 
     for (int i = 0; i < CPT; ++i) {
         const int c = threadIdx.x + i * kStepThreads;
         if (c >= width) continue;
-        const float h = x[i] * inv * a.gain;
+        const float h = x[i] * inv * (a.gain_w ? a.gain * a.gain_w[c] : a.gain);
         float z = 0.0f;
 #pragma unroll
         for (int j = 0; j < kStepTaps - 1; ++j) z = fmaf(w[i][j], u[i][j], z);
@@ -134,10 +154,10 @@ __global__ void __launch_bounds__(kNormThreads) rows_norm_kernel(const RowsArgs 
     const RowSource src(a, t);
     float i0 = 0.0f, i1 = 0.0f;
     float2 q = make_float2(0.0f, 0.0f);
-    if (src.y1) {
+    if (src.normed) {
 #pragma unroll 4
         for (int c = threadIdx.x; c < width; c += kNormThreads) {
-            const float u = src.y0[c], v = src.y1[c];
+            const float u = src.first(c), v = src.y1 ? src.y1[c] : 0.0f;
             q.x = fmaf(u, u, q.x);
             q.y = fmaf(v, v, q.y);
         }
@@ -150,7 +170,10 @@ __global__ void __launch_bounds__(kNormThreads) rows_norm_kernel(const RowsArgs 
 #pragma unroll 4
     for (int c = threadIdx.x; c < width; c += kNormThreads) {
         float x = src.plain(c);
-        if (src.y1) x += 0.5f * (src.y0[c] * i0 * a.w0[c] + src.y1[c] * i1 * a.w1[c]);
+        if (src.normed) {
+            const float v = src.first(c) * i0 * a.w0[c];
+            x += src.y1 ? 0.5f * (v + src.y1[c] * i1 * a.w1[c]) : v;
+        }
         xo[c] = x;
         q.x = fmaf(x, x, q.x);
     }
@@ -169,11 +192,12 @@ __global__ void __launch_bounds__(kConvThreads) rows_conv_kernel(const RowsArgs 
     const int t0 = blockIdx.y * (DECODE ? 1 : kConvRows), n_rows = DECODE ? 1 : min(kConvRows, a.M - t0);
     const size_t off = DECODE ? (size_t)t0 * a.seq_stride : 0;
     const float* tail_in = a.tail_in + off;
+    const float gain = a.gain_w ? a.gain * a.gain_w[c] : a.gain;
     // input of the convolution at row t: from the launch, or from the carried rows before it
     auto input = [&](int t) {
         const int rel = DECODE ? t - t0 : t;
         if (rel < 0) return rel >= -nt ? tail_in[(size_t)(nt + rel) * width + c] : 0.0f;
-        return a.x_out[(size_t)t * width + c] * a.row_inv[t] * a.gain;
+        return a.x_out[(size_t)t * width + c] * a.row_inv[t] * gain;
     };
     const bool lead = a.mu && !DECODE && t0 > 0;                 // the shift starts from the row before, recomputed
     const int start = lead ? -1 : 0;
@@ -223,7 +247,9 @@ __global__ void __launch_bounds__(kConvThreads) rows_conv_kernel(const RowsArgs 
 int launch_rows(const RowsArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
     if (a.M <= 0) return 0;
     if (a.taps < 1 || a.taps > kMaxTaps || a.width <= 0 || a.n_mix > 8) return -1;
-    if (a.decode && a.width <= kStepThreads * kStepMaxCols && a.taps <= kStepTaps) {
+    if ((a.y_slot && (!a.y_weight || a.n_y < 1)) || (a.y1 && !a.w0)) return -1;
+    const bool alone = a.decode || (!a.conv_w && !a.mu);          // no row looks at another one of the launch
+    if (alone && a.width <= kStepThreads * kStepMaxCols && a.taps <= kStepTaps) {
         auto go = [&](auto kernel) { return launch_kernel(kernel, dim3(a.M), dim3(kStepThreads), 0, st, a.use_pdl, 1, a); };
         *n_kernels += 1;
         const int cols = (a.width + kStepThreads - 1) / kStepThreads;

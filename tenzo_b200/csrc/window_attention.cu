@@ -15,14 +15,7 @@ namespace cg = cooperative_groups;
 
 namespace tz {
 
-int launch_window_flash(const WindowAttnArgs& a, int hist, cudaStream_t st);     // window_attention_mma.cu: bf16, tensor cores
-bool window_flash_applicable(const WindowAttnArgs& a);
-
 constexpr int kWaThreads = 256, kWaWarps = 8, kWaSeg = 256;
-
-__device__ __forceinline__ float head_slope(const WindowAttnArgs& a, int h) {
-    return a.slope_base == 0.0f ? 0.0f : exp2f(-a.slope_base * (float)(h + 1) / (float)a.heads);
-}
 
 // y = sum_j w[j] u_(t-taps+1+j) for one channel; `cur` is u_t, older values from the tail
 __device__ __forceinline__ float conv_step(const float* w, int ch, int n_ch, int taps, const float* tail, int tail_ld, float cur) {
@@ -47,27 +40,6 @@ __device__ __forceinline__ void raw_floats(const uint4 (&r)[2], float (&f)[8]) {
     const uint32_t b[8] = {r[0].x, r[0].y, r[0].z, r[0].w, r[1].x, r[1].y, r[1].z, r[1].w};
 #pragma unroll
     for (int i = 0; i < 8; ++i) f[i] = __uint_as_float(b[i]);
-}
-
-// Sums of GQ values over groups of LK lanes: halves of the values travel while there are several, so that the total is
-// GQ - 1 + log2(LK / GQ) exchanges. The lane is left with the sum of value `which`.
-template <int GQ, int LK>
-__device__ __forceinline__ float group_sums(float (&s)[GQ], int lane, int& which) {
-    which = 0;
-    int m = LK / 2;
-#pragma unroll
-    for (int n = GQ; n > 1; n >>= 1, m >>= 1) {
-        const bool up = lane & m;
-#pragma unroll
-        for (int i = 0; i < n / 2; ++i) {
-            const float send = up ? s[i] : s[i + n / 2], keep = up ? s[i + n / 2] : s[i];
-            s[i] = keep + __shfl_xor_sync(0xffffffffu, send, m);
-        }
-        if (up) which += n / 2;
-    }
-#pragma unroll
-    for (; m > 0; m >>= 1) s[0] += __shfl_xor_sync(0xffffffffu, s[0], m);
-    return s[0];
 }
 
 // GQ query heads at a time (1, 2 or 4); LK lanes share a key, eight elements each. A lane's piece of the queries is in
@@ -133,7 +105,7 @@ __global__ void __launch_bounds__(kWaThreads, 2) window_decode_kernel(const WaDe
             float none[GQ] = {};
             group_sums<GQ, LK>(none, lane, mine);
         }
-        const float slope = head_slope(a, kvh * group + q0 + mine);
+        const float slope = head_slope(a.slope_base, a.heads, kvh * group + q0 + mine);
         float m[GQ], l[GQ], acc[GQ][8];
 #pragma unroll
         for (int g = 0; g < GQ; ++g) {
@@ -357,64 +329,6 @@ __global__ void __launch_bounds__(256) window_ring_kernel(const WaChunkLaunch L,
     }
 }
 
-// Plain FMA attention: a CTA takes eight consecutive queries of one head, a warp one of them; 32 keys at a time in shared
-// memory, lanes over keys for the scores and over value columns for the sums.
-constexpr int kWaQ = 8, kWaMaxCols = kMaxHeadDim / 32;
-
-template <typename T>
-__global__ void __launch_bounds__(kWaThreads) window_chunk_kernel(const WaChunkLaunch L) {
-    extern __shared__ float sm[];
-    const WindowAttnArgs& a = L.a;
-    const int ldd = L.ldd, ldv = L.ldv, total = L.hist + a.M, h = blockIdx.y, kvh = h / L.group;
-    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-    const int kstride = ldd + 1;                            // odd: lanes hit different banks
-    float* s_k = sm;                                        // [32][ldd + 1]
-    float* s_v = s_k + 32 * kstride;                        // [32][ldv]
-    float* s_q = s_v + 32 * ldv;                            // [kWaQ][ldd]
-    const int t = blockIdx.x * kWaQ + warp, i = L.hist + t;  // linear index of this warp's query
-    const bool live = t < a.M;
-    for (int d = lane; d < ldd; d += 32)
-        s_q[warp * ldd + d] = live ? to_f(reinterpret_cast<const T*>(a.lin_q)[((size_t)t * a.heads + h) * ldd + d]) * a.scale : 0.0f;
-    const float slope = head_slope(a, h);
-    float m = a.sink > 0.0f ? 0.0f : -1e30f, l = a.sink, acc[kWaMaxCols];   // the sink is a score of 0
-#pragma unroll
-    for (int c = 0; c < kWaMaxCols; ++c) acc[c] = 0.0f;
-    const int i_last = L.hist + min(a.M, (int)(blockIdx.x + 1) * kWaQ) - 1;
-    const int first = max(0, L.hist + (int)blockIdx.x * kWaQ - a.window + 1);
-    for (int k0 = first; k0 <= i_last; k0 += 32) {
-        __syncthreads();
-        for (int e = threadIdx.x; e < 32 * ldd; e += kWaThreads) {
-            const int r = e / ldd, d = e - r * ldd;
-            s_k[r * kstride + d] = k0 + r < total ? to_f(reinterpret_cast<const T*>(a.lin_k)[((size_t)kvh * total + k0 + r) * ldd + d]) : 0.0f;
-        }
-        for (int e = threadIdx.x; e < 32 * ldv; e += kWaThreads) {
-            const int r = e / ldv;
-            s_v[e] = k0 + r < total ? to_f(reinterpret_cast<const T*>(a.lin_v)[((size_t)kvh * total + k0) * ldv + e]) : 0.0f;
-        }
-        __syncthreads();
-        const int j = k0 + lane, dist = i - j;
-        float s = 0.0f;
-        for (int d = 0; d < ldd; ++d) s = fmaf(s_q[warp * ldd + d], s_k[lane * kstride + d], s);
-        s = live && dist >= 0 && dist < a.window ? s - slope * (float)dist : -INFINITY;
-        const float mn = fmaxf(m, warp_max(s)), f = expf(m - mn), p = expf(s - mn);
-        l = l * f + warp_sum(p);
-        m = mn;
-#pragma unroll
-        for (int c = 0; c < kWaMaxCols; ++c) acc[c] *= f;
-        for (int r = 0; r < 32; ++r) {
-            const float pr = __shfl_sync(0xffffffffu, p, r);
-#pragma unroll
-            for (int c = 0; c < kWaMaxCols; ++c)
-                if (c * 32 + lane < ldv) acc[c] = fmaf(pr, s_v[r * ldv + c * 32 + lane], acc[c]);
-        }
-    }
-    if (!live) return;
-    T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.ld_out + (size_t)h * a.vdim;
-#pragma unroll
-    for (int c = 0; c < kWaMaxCols; ++c)
-        if (c * 32 + lane < a.vdim) out[c * 32 + lane] = from_f<T>(acc[c] / l);
-}
-
 template <typename T>
 static int window_attention(const WindowAttnArgs& a, cudaStream_t st, unsigned long long* n_kernels) {
     const int ldd = round_up(a.dim, 8), ldv = round_up(a.vdim, 8), group = a.heads / a.kv_heads;
@@ -448,11 +362,15 @@ static int window_attention(const WindowAttnArgs& a, cudaStream_t st, unsigned l
     const int rows = a.M < a.ring ? a.M : a.ring;
     window_ring_kernel<T, true><<<rows, 256, 0, st>>>(L, rows);
     *n_kernels += L.hist > 0 ? 4 : 3;
-    if (!a.f32 && window_flash_applicable(a)) return launch_window_flash(a, L.hist, st);
-    const size_t smem = 4 * ((size_t)32 * (ldd + 1) + 32 * ldv + kWaQ * ldd);
-    if (int rc = allow_smem(window_chunk_kernel<T>, smem)) return rc;
-    window_chunk_kernel<T><<<dim3((a.M + kWaQ - 1) / kWaQ, a.heads), kWaThreads, smem, st>>>(L);
-    return (int)cudaGetLastError();
+    LinearAttn n;
+    n.q = a.lin_q;
+    n.k = a.lin_k; n.k_row = ldd; n.k_head = (size_t)(L.hist + a.M) * ldd;
+    n.v = a.lin_v; n.v_row = ldv; n.v_head = (size_t)(L.hist + a.M) * ldv;
+    n.d1 = ldd; n.dv = ldv; n.vdim = a.vdim;
+    n.heads = a.heads; n.group = group; n.M = a.M; n.hist = L.hist; n.window = a.window;
+    n.scale = a.scale; n.slope_base = a.slope_base; n.sink = a.sink;
+    n.out = a.out; n.ld_out = a.ld_out; n.out_head = a.vdim; n.f32 = a.f32;
+    return launch_linear_attention(n, st);
 }
 
 int launch_window_attention(const WindowAttnArgs& a, cudaStream_t st, unsigned long long* n_kernels) {

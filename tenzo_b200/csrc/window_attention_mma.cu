@@ -1,4 +1,5 @@
-// Sliding-window attention over the linear layout of a chunk with bf16 storage, on tensor cores (mma.sync m16n8k16).
+// Sliding-window attention over the linear layout of a chunk (LinearAttn) with bf16 storage, on tensor cores (mma.sync
+// m16n8k16).
 //
 // A CTA takes 64 consecutive queries of one head, a warp 16 of them; tiles of 64 keys stream through two shared-memory
 // stages. Scores and softmax are fp32. The weights enter the second product as the sum of two bf16 values (the rounded
@@ -10,23 +11,10 @@ namespace tz {
 constexpr int kWfQ = 64, kWfK = 64, kWfThreads = 128;
 
 struct WfLaunch {
-    WindowAttnArgs a;
-    int ldd, ldv, group, hist, dp, vp;       // dp / vp: head sizes padded to 32 / 16
+    LinearAttn a;
+    int dp, vp;                              // head sizes padded to 32 / 16
 };
 
-__device__ __forceinline__ void ldsm4(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void ldsm4t(uint32_t (&r)[4], uint32_t addr) {
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0,%1,%2,%3}, [%4];" : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
-}
-__device__ __forceinline__ void mma_bf16(float (&c)[4], const uint32_t (&a)[4], uint32_t b0, uint32_t b1) {
-    asm volatile("mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0,%1,%2,%3}, {%4,%5,%6,%7}, {%8,%9}, {%0,%1,%2,%3};"
-                 : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3]) : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-__device__ __forceinline__ void cp16(void* dst, const void* src) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(smem_addr(dst)), "l"(src) : "memory");
-}
 // two floats as bf16 (x in the low half), and what the rounding dropped
 __device__ __forceinline__ uint32_t pack_split(float x, float y, uint32_t& rest) {
     const bf16 bx = __float2bfloat16_rn(x), by = __float2bfloat16_rn(y);
@@ -39,13 +27,14 @@ __device__ __forceinline__ uint32_t pack_split(float x, float y, uint32_t& rest)
 template <int KT, int VT>
 __global__ void __launch_bounds__(kWfThreads) window_flash_kernel(const WfLaunch L) {
     extern __shared__ __align__(16) unsigned char smem[];
-    const WindowAttnArgs& a = L.a;
-    const int ldd = L.ldd, ldv = L.ldv, ks = L.dp + 8, vs = L.vp + 8, total = L.hist + a.M;
-    const int h = blockIdx.y, kvh = h / L.group, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
+    const LinearAttn& a = L.a;
+    const int d1 = a.d1 / 8, ldd = a.d1 + a.d2, ldv = a.dv, ks = L.dp + 8, vs = L.vp + 8, total = a.hist + a.M;
+    const int h = blockIdx.y, kvh = h / a.group, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
     bf16* s_k = reinterpret_cast<bf16*>(smem);               // [2][64][ks]
     bf16* s_v = s_k + 2 * kWfK * ks;                         // [2][64][vs]
-    const bf16* gk = reinterpret_cast<const bf16*>(a.lin_k) + (size_t)kvh * total * ldd;
-    const bf16* gv = reinterpret_cast<const bf16*>(a.lin_v) + (size_t)kvh * total * ldv;
+    const bf16* gk = static_cast<const bf16*>(a.k) + (size_t)kvh * a.k_head;
+    const bf16* gk2 = static_cast<const bf16*>(a.k2);
+    const bf16* gv = static_cast<const bf16*>(a.v) + (size_t)kvh * a.v_head;
     for (int i = tid; i < 2 * kWfK * (ks + vs) / 8; i += kWfThreads) reinterpret_cast<uint4*>(smem)[i] = make_uint4(0, 0, 0, 0);   // padding
     __syncthreads();
 
@@ -56,10 +45,10 @@ __global__ void __launch_bounds__(kWfThreads) window_flash_kernel(const WfLaunch
 #pragma unroll
         for (int i = 0; i < 4; ++i) {
             const int t = row0 + g + (i & 1) * 8, c = kt * 16 + t4 * 2 + (i >> 1) * 8;
-            qf[kt][i] = t < a.M && c < ldd ? *reinterpret_cast<const uint32_t*>(reinterpret_cast<const bf16*>(a.lin_q) + ((size_t)t * a.heads + h) * ldd + c) : 0u;
+            qf[kt][i] = t < a.M && c < ldd ? *reinterpret_cast<const uint32_t*>(static_cast<const bf16*>(a.q) + ((size_t)t * a.heads + h) * ldd + c) : 0u;
         }
 
-    const int i_first = L.hist + q0, i_last = L.hist + min(a.M, q0 + kWfQ) - 1;      // linear places of the CTA's queries
+    const int i_first = a.hist + q0, i_last = a.hist + min(a.M, q0 + kWfQ) - 1;      // linear places of the CTA's queries
     const int k_first = max(0, i_first - a.window + 1) / kWfK * kWfK;
     const int n_tiles = (i_last - k_first) / kWfK + 1;
     auto fetch = [&](int tile) {
@@ -67,11 +56,12 @@ __global__ void __launch_bounds__(kWfThreads) window_flash_kernel(const WfLaunch
         bf16 *dk = s_k + (tile & 1) * kWfK * ks, *dv = s_v + (tile & 1) * kWfK * vs;
         for (int i = tid; i < kWfK * (ldd / 8); i += kWfThreads) {
             const int r = i / (ldd / 8), c = i - r * (ldd / 8);
-            cp16(dk + r * ks + c * 8, gk + (size_t)min(k0 + r, total - 1) * ldd + c * 8);
+            const size_t row = min(k0 + r, total - 1);
+            cp16(dk + r * ks + c * 8, c < d1 ? gk + row * a.k_row + c * 8 : gk2 + row * a.k2_row + (c - d1) * 8);
         }
         for (int i = tid; i < kWfK * (ldv / 8); i += kWfThreads) {
             const int r = i / (ldv / 8), c = i - r * (ldv / 8);
-            cp16(dv + r * vs + c * 8, gv + (size_t)min(k0 + r, total - 1) * ldv + c * 8);
+            cp16(dv + r * vs + c * 8, gv + (size_t)min(k0 + r, total - 1) * a.v_row + c * 8);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -91,7 +81,7 @@ __global__ void __launch_bounds__(kWfThreads) window_flash_kernel(const WfLaunch
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const int k0 = k_first + tile * kWfK, w_first = L.hist + row0, w_last = w_first + 15;
+        const int k0 = k_first + tile * kWfK, w_first = a.hist + row0, w_last = w_first + 15;
         // a warp skips tiles that none of its queries sees
         if (row0 < a.M && k0 <= w_last && k0 + kWfK - 1 > w_first - a.window) {
             const uint32_t bk = smem_addr(s_k + (tile & 1) * kWfK * ks), bv = smem_addr(s_v + (tile & 1) * kWfK * vs);
@@ -164,7 +154,7 @@ __global__ void __launch_bounds__(kWfThreads) window_flash_kernel(const WfLaunch
         const int t = row0 + g + r * 8;
         if (t >= a.M) continue;
         const float inv = 1.0f / (l[r] + (a.sink > 0.0f ? a.sink * exp2f(-m[r]) : 0.0f));
-        bf16* out = reinterpret_cast<bf16*>(a.out) + (size_t)t * a.ld_out + (size_t)h * a.vdim;
+        bf16* out = reinterpret_cast<bf16*>(a.out) + (size_t)t * a.ld_out + (size_t)h * a.out_head;
 #pragma unroll
         for (int v = 0; v < VT; ++v)
 #pragma unroll
@@ -175,12 +165,12 @@ __global__ void __launch_bounds__(kWfThreads) window_flash_kernel(const WfLaunch
     }
 }
 
-bool window_flash_applicable(const WindowAttnArgs& a) { return a.dim <= 128 && a.vdim <= 128 && a.M >= 16; }
+bool window_flash_applicable(const LinearAttn& a) { return a.d1 + a.d2 <= 256 && a.vdim <= 128 && a.M >= 16; }
 
-int launch_window_flash(const WindowAttnArgs& a, int hist, cudaStream_t st) {
+int launch_window_flash(const LinearAttn& a, cudaStream_t st) {
     WfLaunch L;
-    L.a = a; L.ldd = round_up(a.dim, 8); L.ldv = round_up(a.vdim, 8); L.group = a.heads / a.kv_heads; L.hist = hist;
-    L.dp = round_up(a.dim, 32); L.vp = round_up(a.vdim, 16);
+    L.a = a;
+    L.dp = round_up(a.d1 + a.d2, 32); L.vp = round_up(a.vdim, 16);
     const size_t smem = (size_t)2 * 2 * kWfK * (L.dp + 8 + L.vp + 8);
     const dim3 grid((a.M + kWfQ - 1) / kWfQ, a.heads);
     auto go = [&](auto kernel) {
@@ -189,7 +179,9 @@ int launch_window_flash(const WindowAttnArgs& a, int hist, cudaStream_t st) {
         return (int)cudaGetLastError();
     };
     if (L.dp <= 64) return L.vp <= 64 ? go(window_flash_kernel<4, 8>) : go(window_flash_kernel<4, 16>);
-    return L.vp <= 64 ? go(window_flash_kernel<8, 8>) : go(window_flash_kernel<8, 16>);
+    if (L.dp <= 128) return L.vp <= 64 ? go(window_flash_kernel<8, 8>) : go(window_flash_kernel<8, 16>);
+    if (L.dp <= 192) return L.vp <= 64 ? go(window_flash_kernel<12, 8>) : go(window_flash_kernel<12, 16>);
+    return L.vp <= 64 ? go(window_flash_kernel<16, 8>) : go(window_flash_kernel<16, 16>);
 }
 
 }  // namespace tz

@@ -167,28 +167,40 @@ def tl1_pack_rows2bit(raw, N, K):
 
 
 # ---- pieces of the hybrid decoders ------------------------------------------------------------------------------------
-def _struct_call(name: str, struct, defaults: dict, fields: dict):
+def _struct_call(name: str, defaults: dict, fields: dict):
     """One flat kernel call: keyword arguments are the struct's fields, tensors are passed by address."""
-    args = struct()
+    args = abi.STRUCT_CALLS[name]()
     for k, v in {**defaults, **fields}.items():
         setattr(args, k, v.data_ptr() if isinstance(v, torch.Tensor) else (C.c_int * 8)(*v) if isinstance(v, (list, tuple)) else v)
     _ok(getattr(load_library(), "tenzo_cuda_" + name)(C.byref(args), _stream()), "tenzo_cuda_" + name)
 
 
 def rows(**fields):
-    _struct_call("rows", abi.RowsArgs, {"gain": 1.0, "taps": 1}, fields)
+    _struct_call("rows", {"gain": 1.0, "taps": 1}, fields)
 
 
 def gemm(**fields):
-    _struct_call("gemm", abi.GemmArgs, {"n_seg": 1}, fields)
+    _struct_call("gemm", {"n_seg": 1}, fields)
 
 
 def window_attention(**fields):
-    _struct_call("window_attention", abi.WindowAttentionArgs, {"taps": 1, "scale": 1.0, "slope_base": 8.0, "sink": 1.0}, fields)
+    _struct_call("window_attention", {"taps": 1, "scale": 1.0, "slope_base": 8.0, "sink": 1.0}, fields)
 
 
 def linear_scan(**fields):
-    _struct_call("linear_scan", abi.ScanArgs, {"q_scale": 1.0, "k_scale": 1.0, "tau": 1.0}, fields)
+    _struct_call("linear_scan", {"q_scale": 1.0, "k_scale": 1.0, "tau": 1.0}, fields)
+
+
+def delta_rule(**fields):
+    _struct_call("delta_rule", {"taps": 1, "q_scale": 1.0, "unit_eps": 1e-6}, fields)
+
+
+def latent_attention(**fields):
+    _struct_call("latent_attention", {"scale": 1.0}, fields)
+
+
+def route(**fields):
+    _struct_call("route", {}, fields)
 
 
 def gemm_workspace() -> torch.Tensor:
@@ -197,3 +209,7 @@ def gemm_workspace() -> torch.Tensor:
 
 def linear_scan_part(M: int, heads: int, dim: int, vdim: int) -> torch.Tensor:
     return torch.empty(load_library().tenzo_cuda_linear_scan_part_floats(M, heads, dim, vdim), dtype=torch.float32, device="cuda")
+
+
+def delta_rule_work(M: int, heads: int, kv_heads: int, dim: int, vdim: int) -> torch.Tensor:
+    return torch.empty(load_library().tenzo_cuda_delta_rule_work_floats(M, heads, kv_heads, dim, vdim), dtype=torch.float32, device="cuda")

@@ -128,7 +128,7 @@ def prompt_tokens(seed: int, n: int, vocab: int) -> np.ndarray:
     return np.random.default_rng([seed, 99]).integers(0, vocab, n, dtype=np.int32)
 
 
-# ---- Sozopel folders ----------------------------------------------------------------------------------------------------
+# ---- folders of hybrid decoders ----------------------------------------------------------------------------------------------------
 def bf16_bits(x: np.ndarray) -> np.ndarray:
     """fp32 -> bf16 bit patterns, round to nearest even."""
     b = np.ascontiguousarray(x, np.float32).view(np.uint32)
@@ -206,30 +206,94 @@ def sozopel_tensors(cfg: dict, rank: int) -> dict:
     return t
 
 
-def write_sozopel(folder, cfg: dict, *, rank: int = 8, seed: int = 0, change=None) -> dict:
-    """A Sozopel model folder with random weights; `change(tensors)` may edit them first. Returns the fp32 tensors, already
-    rounded to what the file holds."""
+def tigitar_tensors(cfg: dict) -> dict:
+    """name -> (shape, spread, centre) of every tensor of a Tigitar configuration."""
+    W, V = cfg["width"], cfg["vocab"]
+    t = {"embed": ((V, W), 1.0, 0.0), "final.norm": ((W,), 0.1, 1.0), "head": ((V, W), W ** -0.5, 0.0)}
+
+    def lin(name, rows, cols, gain=1.0):
+        t[name] = ((rows, cols), gain * cols ** -0.5, 0.0)
+
+    for i, layer in enumerate(cfg["layers"]):
+        p, mix, mlp = f"l{i}.", layer["mixer"], layer["mlp"]
+        m = p + "mix."
+        for n in ("norm1", "norm1b") + (("norm2", "norm2b") if mlp else ()):
+            t[p + n] = ((W,), 0.2, 1.0)
+        if layer["type"] == "delta":
+            nk, nv, heads = mix["kv_heads"] * mix["dim"], mix["heads"] * mix["vdim"], mix["heads"]
+            for s, n in (("q", nk), ("k", nk), ("v", nv)):
+                lin(m + s, n, W)
+                t[m + s + ".conv"] = ((n, mix["conv"]), 0.5, 0.3)
+            lin(m + "g", nv, W)
+            for s in "ab":
+                lin(m + s, heads, W)
+            t[m + "A_log"] = ((heads,), 1.0, -2.0)
+            t[m + "dt_bias"] = ((heads,), 1.0, -1.0)
+            t[m + "norm"] = ((mix["vdim"],), 0.2, 1.0)
+            lin(m + "o", W, nv)
+        elif layer["type"] == "latent_attention":
+            heads, rank = mix["heads"], mix["kv_rank"]
+            lin(m + "q", heads * (mix["dim"] + mix["rot_dim"]), W, 1.5)
+            if "kv_from" not in mix:
+                lin(m + "dkv", rank + mix["rot_dim"], W)
+                t[m + "dkv.norm"] = ((rank,), 0.2, 1.0)
+            lin(m + "uk", heads * mix["dim"], rank, 1.5)
+            lin(m + "uv", heads * mix["vdim"], rank)
+            lin(m + "o", W, heads * mix["vdim"])
+        if mlp and mlp["kind"] == "dense":
+            lin(p + "mlp.gate", mlp["ff"], W)
+            lin(p + "mlp.up", mlp["ff"], W)
+            lin(p + "mlp.down", W, mlp["ff"])
+        elif mlp:
+            for e in range(mlp["router"]["experts"]):
+                for s in ("gate", "up"):
+                    lin(f"{p}mlp.e{e}.{s}", mlp["expert"]["ff"], W)
+                lin(f"{p}mlp.e{e}.down", W, mlp["expert"]["ff"])
+            lin(p + "mlp.router", mlp["router"]["experts"], W, 2.0)
+            t[p + "mlp.correction"] = ((mlp["router"]["experts"],), 0.2, 0.0)
+    return t
+
+
+def _write_folder(folder, architecture: str, cfg: dict, spec: dict, seed: int, change) -> dict:
     import json
     from pathlib import Path
     rng = np.random.default_rng(seed)
-    out = {name: (centre + spread * rng.standard_normal(shape)).astype(np.float32) for name, (shape, spread, centre) in sozopel_tensors(cfg, rank).items()}
+    out = {name: (centre + spread * rng.standard_normal(shape)).astype(np.float32) for name, (shape, spread, centre) in spec.items()}
     if change is not None:
         change(out)
     folder = Path(folder)
     folder.mkdir(parents=True, exist_ok=True)
-    (folder / "config.json").write_text(json.dumps(dict(cfg, architecture="Sozopel")))
+    (folder / "config.json").write_text(json.dumps(dict(cfg, architecture=architecture)))
     write_safetensors(folder / "model.safetensors", {n: np.asarray(a) for n, a in out.items()})
     return {n: (bf16_bits(a).astype(np.uint32) << 16).view(np.float32).reshape(np.shape(a)) for n, a in out.items()}
 
 
+def write_sozopel(folder, cfg: dict, *, rank: int = 8, seed: int = 0, change=None) -> dict:
+    """A Sozopel model folder with random weights; `change(tensors)` may edit them first. Returns the fp32 tensors, already
+    rounded to what the file holds."""
+    return _write_folder(folder, "Sozopel", cfg, sozopel_tensors(cfg, rank), seed, change)
+
+
+def write_tigitar(folder, cfg: dict, *, seed: int = 0, change=None) -> dict:
+    """The same for Tigitar."""
+    return _write_folder(folder, "Tigitar", cfg, tigitar_tensors(cfg), seed, change)
+
+
 def write_sozopel_pooled(folder, cfg: dict, *, rank: int, seed: int = 0):
     """write_sozopel for large models: values come from one pool of random numbers, tensors go to the file one by one."""
+    _write_pooled(folder, "Sozopel", cfg, sozopel_tensors(cfg, rank), seed)
+
+
+def write_tigitar_pooled(folder, cfg: dict, *, seed: int = 0):
+    _write_pooled(folder, "Tigitar", cfg, tigitar_tensors(cfg), seed)
+
+
+def _write_pooled(folder, architecture: str, cfg: dict, spec: dict, seed: int):
     import json
     import struct
     from pathlib import Path
     rng = np.random.default_rng(seed)
     pool = rng.standard_normal(1 << 22, dtype=np.float32)
-    spec = sozopel_tensors(cfg, rank)
     head, off = {}, 0
     for name, (shape, _, _) in spec.items():
         n = int(np.prod(shape))
@@ -238,7 +302,7 @@ def write_sozopel_pooled(folder, cfg: dict, *, rank: int, seed: int = 0):
     text = json.dumps(head).encode()
     text += b" " * (-len(text) % 8)
     folder = Path(folder)
-    (folder / "config.json").write_text(json.dumps(dict(cfg, architecture="Sozopel")))
+    (folder / "config.json").write_text(json.dumps(dict(cfg, architecture=architecture)))
     with open(folder / "model.safetensors", "wb") as f:
         f.write(struct.pack("<Q", len(text)) + text)
         for shape, spread, centre in spec.values():
