@@ -14,6 +14,7 @@
 
   sozopel       the Sozopel hybrid decoder beside BitNet at equal size: prompt and decode throughput at three widths, and
                 every kernel alone against its roofline (tenzo_b200/bench_hybrid.py).
+  tigitar       the same for the Tigitar decoder, beside Sozopel (tenzo_b200/bench_tigitar.py).
 
 Each prints one JSON line in the same format as the default workload.
 """
@@ -487,9 +488,14 @@ def run_sozopel(args):
     return bench_hybrid.run(args)
 
 
+def run_tigitar(args):
+    from . import bench_tigitar
+    return bench_tigitar.run(args)
+
+
 def run(args):
     fn = {"gemv": run_gemv, "lm_head": run_lm_head, "gemm": run_gemm, "attn": run_attn, "decode_batch": run_decode_batch, "decode_tp": run_decode_tp,
-          "sozopel": run_sozopel}.get(args.workload)
+          "sozopel": run_sozopel, "tigitar": run_tigitar}.get(args.workload)
     if fn is None:
         raise SystemExit(f"unknown workload {args.workload!r}")
     return fn(args)
