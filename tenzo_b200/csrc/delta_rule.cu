@@ -15,7 +15,7 @@
 
 namespace tz {
 
-constexpr int kDeltaThreads = 256, kDeltaPre = 16;       // decode: float4 pieces of the state a thread holds
+constexpr int kDeltaThreads = 256;
 constexpr int kDeltaBlock = 8, kDeltaCols = 16, kDeltaStages = 4;
 constexpr int kDeltaCoef = 2 * kDeltaBlock * kDeltaBlock + 2 * kDeltaBlock;   // inverse * beta, read-out, decays from the start, to the end
 
@@ -30,20 +30,22 @@ __device__ __forceinline__ float conv_at(const float* w, int ch, int n_ch, int t
     return silu_f(y);
 }
 
-template <typename T>
-__global__ void __launch_bounds__(kDeltaThreads) delta_decode_kernel(const DeltaArgs a) {
+// THREADS 256 or 512, whichever lets a thread hold its part of the state in kPre pieces for most sizes.
+template <typename T, int THREADS>
+__global__ void __launch_bounds__(THREADS, 1024 / THREADS) delta_decode_kernel(const DeltaArgs a) {
     extern __shared__ float sm[];
-    __shared__ float s_red[4][8];
+    constexpr int kPre = 8;                              // float4 pieces of the state that are fetched ahead
+    __shared__ float s_red[4][THREADS / 32];
     const int head = blockIdx.x, seq = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int ldv = (a.vdim + 3) & ~3, nc = ldv / 4;
     int nc2 = 1;
     while (nc2 < nc) nc2 *= 2;
-    const int col = tid & (nc2 - 1), rg = tid / nc2, n_rg = kDeltaThreads / nc2;
+    const int col = tid & (nc2 - 1), rg = tid / nc2, n_rg = THREADS / nc2;
     const bool live = col < nc;
     float4* S = reinterpret_cast<float4*>(a.state + (size_t)seq * a.state_seq_stride + (size_t)head * a.dim * ldv) + col;
-    float4 pre[kDeltaPre];
+    float4 pre[kPre];
 #pragma unroll
-    for (int i = 0; i < kDeltaPre; ++i) {
+    for (int i = 0; i < kPre; ++i) {
         const int r = rg + i * n_rg;
         if (live && r < a.dim) pre[i] = S[(size_t)r * nc];
     }
@@ -86,7 +88,7 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_decode_kernel(const Delta
     for (int i = 0; i < 3; ++i) {
         sums[i] = 0.0f;
 #pragma unroll
-        for (int w = 0; w < kDeltaThreads / 32; ++w) sums[i] += s_red[i][w];
+        for (int w = 0; w < THREADS / 32; ++w) sums[i] += s_red[i][w];
     }
     const float iq = a.q_scale / sqrtf(sums[0] + a.unit_eps), ik = 1.0f / sqrtf(sums[1] + a.unit_eps), kq = sums[2] * iq * ik;
     if (tid < a.dim) { s_q[tid] = q * iq; s_k[tid] = k * ik; }
@@ -102,9 +104,9 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_decode_kernel(const Delta
             }
         };
 #pragma unroll
-        for (int i = 0; i < kDeltaPre; ++i)
+        for (int i = 0; i < kPre; ++i)
             if (rg + i * n_rg < a.dim) step(rg + i * n_rg, pre[i]);
-        for (int r = rg + kDeltaPre * n_rg; r < a.dim; r += n_rg) step(r, S[(size_t)r * nc]);
+        for (int r = rg + kPre * n_rg; r < a.dim; r += n_rg) step(r, S[(size_t)r * nc]);
         *reinterpret_cast<float4*>(s_a + rg * ldv + col * 4) = make_float4(pa[0], pa[1], pa[2], pa[3]);
         *reinterpret_cast<float4*>(s_b + rg * ldv + col * 4) = make_float4(pb[0], pb[1], pb[2], pb[3]);
     }
@@ -126,7 +128,7 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_decode_kernel(const Delta
     if (tid < a.vdim) {
         float t = 0.0f;
 #pragma unroll
-        for (int w = 0; w < kDeltaThreads / 32; ++w) t += s_red[3][w];
+        for (int w = 0; w < THREADS / 32; ++w) t += s_red[3][w];
         const float y = o * (1.0f / sqrtf(t / (float)a.vdim + a.eps)) * a.norm[tid];
         reinterpret_cast<T*>(a.out)[(size_t)seq * a.ld_out + head * a.vdim + tid] = from_f<T>(y * silu_f(a.g[row + head * a.vdim + tid]));
     }
@@ -137,76 +139,100 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_decode_kernel(const Delta
             S[(size_t)r * nc] = make_float4(fmaf(g, s.x, kr * u.x), fmaf(g, s.y, kr * u.y), fmaf(g, s.z, kr * u.z), fmaf(g, s.w, kr * u.w));
         };
 #pragma unroll
-        for (int i = 0; i < kDeltaPre; ++i)
+        for (int i = 0; i < kPre; ++i)
             if (rg + i * n_rg < a.dim) update(rg + i * n_rg, pre[i]);
-        for (int r = rg + kDeltaPre * n_rg; r < a.dim; r += n_rg) update(r, S[(size_t)r * nc]);
+        for (int r = rg + kPre * n_rg; r < a.dim; r += n_rg) update(r, S[(size_t)r * nc]);
     }
 }
 
 // ---- chunk ---------------------------------------------------------------------------------------------------------------
 struct DeltaLaunch {
     DeltaArgs a;
-    int dp, vp;                  // padded head sizes: 32 KJ, a multiple of kDeltaCols
+    int dp, vp;                  // padded head sizes: delta_padded(), a multiple of kDeltaCols
     float *kq, *v, *coef, *o;    // [block][kv_head][8 k, 8 q][dp], [block][head][8][vp], [block][head][kDeltaCoef], [M][heads*vdim]
 };
 
-// One CTA per (block of rows, kv head), one warp per row.
+// One CTA per (block of rows, kv head). Convolutions: a thread per channel, the block's rows and the taps - 1 inputs before
+// them in registers; then a warp per row. NT: taps rounded up to 4 or 16.
+template <int NT>
 __global__ void __launch_bounds__(kDeltaThreads) delta_prepare_kernel(const DeltaLaunch L) {
     extern __shared__ float sm[];
     __shared__ float s_kk[8][9], s_qk[8][9], s_sys[8][64], s_gl[8][8], s_beta[8][8];
     const DeltaArgs& a = L.a;
     const int b = blockIdx.x, kvh = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, dp = L.dp;
-    const int t = b * kDeltaBlock + warp, group = a.heads / a.kv_heads;
+    const int t0 = b * kDeltaBlock, group = a.heads / a.kv_heads, taps = a.taps;
     const int n_q = a.kv_heads * a.dim, n_v = a.heads * a.vdim, n_ch = 2 * n_q + n_v;
-    const bool in = t < a.M;
     float* s_k = sm;                                     // [8][dp]
     float* s_q = sm + 8 * dp;
-    // convolved channel of this warp's row: `src` the channel's projection, `first` its place among the tail's channels
-    auto convolved = [&](const float* src, const float* w, int ch, int nch, int first) {
-        float y = 0.0f;
-        for (int j = 0; j < a.taps; ++j) {
-            const int r = t - j, p = a.pos0 + r;
-            const float u = r >= 0 ? src[(size_t)r * a.ld + ch] : p >= 0 ? a.tail[(size_t)(p % a.taps) * n_ch + first + ch] : 0.0f;
-            y = fmaf(w[(size_t)(a.taps - 1 - j) * nch + ch], u, y);
+    for (int i = tid; i < 2 * dp + group * L.vp; i += kDeltaThreads) {
+        // channel `ch` of `nch` with its input at src, its place among the tail's channels and its destination rows
+        const float *src, *w;
+        float* dst;
+        int ch, nch, first, ld;
+        bool ok;
+        if (i < 2 * dp) {
+            const int d = i < dp ? i : i - dp;
+            ok = d < a.dim; ch = kvh * a.dim + d; nch = n_q; ld = dp;
+            src = i < dp ? a.q : a.k; w = i < dp ? a.conv_q : a.conv_k; first = i < dp ? 0 : n_q;
+            dst = (i < dp ? s_q : s_k) + d;
+        } else {
+            const int x = i - 2 * dp, h = kvh * group + x / L.vp, d = x % L.vp;
+            ok = d < a.vdim; ch = h * a.vdim + d; nch = n_v; ld = L.vp;
+            src = a.v; w = a.conv_v; first = 2 * n_q;
+            dst = L.v + ((size_t)b * a.heads + h) * 8 * L.vp + d;
         }
-        return silu_f(y);
-    };
-    float qq = 0.0f, kk = 0.0f;
-    for (int d = lane; d < dp; d += 32) {
-        const bool ok = in && d < a.dim;
-        const float q = ok ? convolved(a.q, a.conv_q, kvh * a.dim + d, n_q, 0) : 0.0f;
-        const float k = ok ? convolved(a.k, a.conv_k, kvh * a.dim + d, n_q, n_q) : 0.0f;
-        s_q[warp * dp + d] = q;
-        s_k[warp * dp + d] = k;
-        qq = fmaf(q, q, qq);
-        kk = fmaf(k, k, kk);
-    }
-    qq = warp_sum(qq);
-    kk = warp_sum(kk);
-    const float iq = a.q_scale / sqrtf(qq + a.unit_eps), ik = 1.0f / sqrtf(kk + a.unit_eps);
-    float* out = L.kq + ((size_t)b * a.kv_heads + kvh) * 16 * dp;
-    for (int d = lane; d < dp; d += 32) {
-        const float q = s_q[warp * dp + d] * iq, k = s_k[warp * dp + d] * ik;
-        s_q[warp * dp + d] = q;
-        s_k[warp * dp + d] = k;
-        out[warp * dp + d] = k;
-        out[(8 + warp) * dp + d] = q;
-    }
-    for (int i = lane; i < group * L.vp; i += 32) {
-        const int h = kvh * group + i / L.vp, d = i % L.vp;
-        L.v[(((size_t)b * a.heads + h) * 8 + warp) * L.vp + d] = in && d < a.vdim ? convolved(a.v, a.conv_v, h * a.vdim + d, n_v, 2 * n_q) : 0.0f;
+        float wt[NT], u[NT + 7];                         // u[NT - 1 + r] is row t0 + r, wt[NT - 1] belongs to the row itself
+#pragma unroll
+        for (int j = 0; j < NT; ++j) wt[j] = ok && j >= NT - taps ? w[(size_t)(j - NT + taps) * nch + ch] : 0.0f;
+#pragma unroll
+        for (int j = 0; j < NT + 7; ++j) {
+            const int r = t0 + j - (NT - 1), p = a.pos0 + r;
+            u[j] = 0.0f;
+            if (ok && j >= NT - taps && r < a.M) {
+                if (r >= 0) u[j] = src[(size_t)r * a.ld + ch];
+                else if (p >= 0) u[j] = a.tail[(size_t)(p % taps) * n_ch + first + ch];
+            }
+        }
+#pragma unroll
+        for (int r = 0; r < 8; ++r) {
+            float y = 0.0f;
+#pragma unroll
+            for (int j = 0; j < NT; ++j) y = fmaf(wt[j], u[j + r], y);
+            dst[r * ld] = t0 + r < a.M ? silu_f(y) : 0.0f;
+        }
     }
     __syncthreads();
-    for (int j = 0; j <= warp; ++j) {                    // row `warp` against the rows up to it
-        float kkj = 0.0f, qkj = 0.0f;
+    float* out = L.kq + ((size_t)b * a.kv_heads + kvh) * 16 * dp;
+    {
+        float qq = 0.0f, kk = 0.0f;
         for (int d = lane; d < dp; d += 32) {
-            const float kj = s_k[j * dp + d];
-            kkj = fmaf(s_k[warp * dp + d], kj, kkj);
-            qkj = fmaf(s_q[warp * dp + d], kj, qkj);
+            qq = fmaf(s_q[warp * dp + d], s_q[warp * dp + d], qq);
+            kk = fmaf(s_k[warp * dp + d], s_k[warp * dp + d], kk);
         }
-        kkj = warp_sum(kkj);
-        qkj = warp_sum(qkj);
-        if (lane == 0) { s_kk[warp][j] = kkj; s_qk[warp][j] = qkj; }
+        const float iq = a.q_scale / sqrtf(warp_sum(qq) + a.unit_eps), ik = 1.0f / sqrtf(warp_sum(kk) + a.unit_eps);
+        for (int d = lane; d < dp; d += 32) {
+            const float q = s_q[warp * dp + d] * iq, k = s_k[warp * dp + d] * ik;
+            s_q[warp * dp + d] = q;
+            s_k[warp * dp + d] = k;
+            out[warp * dp + d] = k;
+            out[(8 + warp) * dp + d] = q;
+        }
+    }
+    __syncthreads();
+    {                                                    // row `warp` against all rows
+        float kkj[8] = {}, qkj[8] = {};
+        for (int d = lane; d < dp; d += 32) {
+            const float k = s_k[warp * dp + d], q = s_q[warp * dp + d];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) {
+                const float kj = s_k[j * dp + d];
+                kkj[j] = fmaf(k, kj, kkj[j]);
+                qkj[j] = fmaf(q, kj, qkj[j]);
+            }
+        }
+        int j;
+        const float kk = group_sums<8, 32>(kkj, lane, j), qk = group_sums<8, 32>(qkj, lane, j);
+        if ((lane & 3) == 0) { s_kk[warp][j] = kk; s_qk[warp][j] = qk; }
     }
     __syncthreads();
     for (int hh = warp; hh < group; hh += 8) {
@@ -247,17 +273,18 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_prepare_kernel(const Delt
     }
 }
 
-// Sixteen value columns of one head, four per warp; eight lanes share a column, lane l holding the state's rows
-// 4 (l + 8 j) .. + 3, and stand for the block's eight rows once the products are summed.
+// Sixteen value columns of one head, four per warp. Half a warp shares a pair of columns, lane l of it holding the state's rows
+// 4 (l + 16 j) .. + 3 of both; once the products are summed, eight lanes stand for the block's eight rows of one column.
 template <int KJ>
 __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
-    constexpr int DP = 32 * KJ, V = 16 * DP, C = V + 8 * kDeltaCols, FLOATS = C + kDeltaCoef;
+    constexpr int DP = 64 * KJ, V = 16 * DP, C = V + 8 * kDeltaCols, FLOATS = C + kDeltaCoef;
     extern __shared__ __align__(16) float smem[];
     const DeltaArgs& a = L.a;
-    const int head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, l = lane & 7, cl = (tid >> 5) * 4 + (lane >> 3), c = blockIdx.x * kDeltaCols + cl;
+    const int head = blockIdx.y, tid = threadIdx.x, lane = tid & 31, l = lane & 15, r = lane & 7;
+    const int cl = (tid >> 5) * 4 + (lane >> 3), c = blockIdx.x * kDeltaCols + cl;              // column whose row r this lane finishes
+    const int cs = blockIdx.x * kDeltaCols + (tid >> 5) * 4 + (lane >> 4) * 2;                  // first column of its part of the state
     const int group = a.heads / a.kv_heads, kvh = head / group, ldv = (a.vdim + 3) & ~3, nv = a.heads * a.vdim;
     const int n_blocks = (a.M + kDeltaBlock - 1) / kDeltaBlock;
-    const bool live = c < a.vdim;
     auto stage = [&](int b) {
         if (b < n_blocks) {
             float* dst = smem + (b % kDeltaStages) * FLOATS;
@@ -269,71 +296,77 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     for (int b = 0; b + 1 < kDeltaStages; ++b) stage(b);
-    float s[KJ * 4];
+    float s[2][KJ * 4];
+    auto place = [&](int x, int j) { return ((size_t)head * a.dim + 4 * (l + 16 * (j >> 2)) + (j & 3)) * ldv + cs + x; };
+    auto exists = [&](int x, int j) { return cs + x < a.vdim && 4 * (l + 16 * (j >> 2)) + (j & 3) < a.dim; };
 #pragma unroll
-    for (int j = 0; j < KJ * 4; ++j) {
-        const int d = 4 * (l + 8 * (j >> 2)) + (j & 3);
-        s[j] = live && d < a.dim ? a.state[((size_t)head * a.dim + d) * ldv + c] : 0.0f;
-    }
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+        for (int j = 0; j < KJ * 4; ++j) s[x][j] = exists(x, j) ? a.state[place(x, j)] : 0.0f;
     for (int b = 0; b < n_blocks; ++b) {
         asm volatile("cp.async.wait_group %0;" ::"n"(kDeltaStages - 2) : "memory");
         __syncthreads();                                 // the block is here, and the stage before it is free
         stage(b + kDeltaStages - 1);
         const float* buf = smem + (b % kDeltaStages) * FLOATS;
         const float *sk = buf + 4 * l, *sq = sk + 8 * DP, *co = buf + C;
-        float pa[8], pb[8];
+        float pa[16], pb[16];                            // [column][row]
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
-            float x = 0.0f, y = 0.0f;
+            float ka[2] = {}, qb[2] = {};
 #pragma unroll
             for (int j = 0; j < KJ; ++j) {
-                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 32 * j), q4 = *reinterpret_cast<const float4*>(sq + t * DP + 32 * j);
-                x = fmaf(k4.x, s[4 * j], x); x = fmaf(k4.y, s[4 * j + 1], x); x = fmaf(k4.z, s[4 * j + 2], x); x = fmaf(k4.w, s[4 * j + 3], x);
-                y = fmaf(q4.x, s[4 * j], y); y = fmaf(q4.y, s[4 * j + 1], y); y = fmaf(q4.z, s[4 * j + 2], y); y = fmaf(q4.w, s[4 * j + 3], y);
+                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 64 * j), q4 = *reinterpret_cast<const float4*>(sq + t * DP + 64 * j);
+                const float kf[4] = {k4.x, k4.y, k4.z, k4.w}, qf[4] = {q4.x, q4.y, q4.z, q4.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i)
+#pragma unroll
+                    for (int x = 0; x < 2; ++x) {
+                        ka[x] = fmaf(kf[i], s[x][4 * j + i], ka[x]);
+                        qb[x] = fmaf(qf[i], s[x][4 * j + i], qb[x]);
+                    }
             }
-            pa[t] = x;
-            pb[t] = y;
-            if (KJ > 4) asm volatile("" ::: "memory");   // otherwise the loads of all rows are moved ahead, and spilled
+            pa[t] = ka[0]; pa[8 + t] = ka[1];
+            pb[t] = qb[0]; pb[8 + t] = qb[1];
+            if (KJ > 2) asm volatile("" ::: "memory");   // otherwise the loads of all rows are moved ahead, and spilled
         }
-        int which;                                       // = l
-        const float at = group_sums<8, 8>(pa, lane, which), bt = group_sums<8, 8>(pb, lane, which);
-        const float from = co[128 + l], x = buf[V + l * kDeltaCols + cl] - from * at;
-        float u = 0.0f, o = from * bt;
+        int which;                                       // = l: column l / 8 of the pair, row l % 8
+        const float at = group_sums<16, 16>(pa, lane, which), bt = group_sums<16, 16>(pb, lane, which);
+        const float from = co[128 + r], x = buf[V + r * kDeltaCols + cl] - from * at;
+        const float4 i0 = *reinterpret_cast<const float4*>(co + r * 8), i1 = *reinterpret_cast<const float4*>(co + r * 8 + 4);
+        const float4 p0 = *reinterpret_cast<const float4*>(co + 64 + r * 8), p1 = *reinterpret_cast<const float4*>(co + 64 + r * 8 + 4);
+        const float inv[8] = {i0.x, i0.y, i0.z, i0.w, i1.x, i1.y, i1.z, i1.w}, p[8] = {p0.x, p0.y, p0.z, p0.w, p1.x, p1.y, p1.z, p1.w};
+        float u[2] = {}, o[2] = {from * bt, 0.0f};
 #pragma unroll
-        for (int h = 0; h < 2; ++h) {
-            const float4 w = *reinterpret_cast<const float4*>(co + l * 8 + 4 * h);
-            u = fmaf(w.x, __shfl_sync(0xffffffffu, x, 4 * h, 8), u);
-            u = fmaf(w.y, __shfl_sync(0xffffffffu, x, 4 * h + 1, 8), u);
-            u = fmaf(w.z, __shfl_sync(0xffffffffu, x, 4 * h + 2, 8), u);
-            u = fmaf(w.w, __shfl_sync(0xffffffffu, x, 4 * h + 3, 8), u);
-        }
-        const float decay = co[128 + 7];
+        for (int t = 0; t < 8; ++t) u[t & 1] = fmaf(inv[t], __shfl_sync(0xffffffffu, x, t, 8), u[t & 1]);
+        const float ur = u[0] + u[1], wr = ur * co[136 + r], decay = co[128 + 7];
 #pragma unroll
-        for (int j = 0; j < KJ * 4; ++j) s[j] *= decay;
-        const float4 p0 = *reinterpret_cast<const float4*>(co + 64 + l * 8), p1 = *reinterpret_cast<const float4*>(co + 64 + l * 8 + 4);
-        const float p[8] = {p0.x, p0.y, p0.z, p0.w, p1.x, p1.y, p1.z, p1.w};
+        for (int y = 0; y < 2; ++y)
+#pragma unroll
+            for (int j = 0; j < KJ * 4; ++j) s[y][j] *= decay;
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
-            const float ut = __shfl_sync(0xffffffffu, u, t, 8), w = ut * co[136 + t];
-            o = fmaf(p[t], ut, o);
-            if (KJ > 4) asm volatile("" ::: "memory");
+            o[t & 1] = fmaf(p[t], __shfl_sync(0xffffffffu, ur, t, 8), o[t & 1]);
+            const float w0 = __shfl_sync(0xffffffffu, wr, t, 16), w1 = __shfl_sync(0xffffffffu, wr, 8 + t, 16);
+            if (KJ > 2) asm volatile("" ::: "memory");
 #pragma unroll
             for (int j = 0; j < KJ; ++j) {
-                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 32 * j);
-                s[4 * j] = fmaf(k4.x, w, s[4 * j]);
-                s[4 * j + 1] = fmaf(k4.y, w, s[4 * j + 1]);
-                s[4 * j + 2] = fmaf(k4.z, w, s[4 * j + 2]);
-                s[4 * j + 3] = fmaf(k4.w, w, s[4 * j + 3]);
+                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 64 * j);
+                const float kf[4] = {k4.x, k4.y, k4.z, k4.w};
+#pragma unroll
+                for (int i = 0; i < 4; ++i) {
+                    s[0][4 * j + i] = fmaf(kf[i], w0, s[0][4 * j + i]);
+                    s[1][4 * j + i] = fmaf(kf[i], w1, s[1][4 * j + i]);
+                }
             }
         }
-        const int row = b * kDeltaBlock + l;
-        if (live && row < a.M) L.o[(size_t)row * nv + head * a.vdim + c] = o;
+        const int row = b * kDeltaBlock + r;
+        if (c < a.vdim && row < a.M) L.o[(size_t)row * nv + head * a.vdim + c] = o[0] + o[1];
     }
 #pragma unroll
-    for (int j = 0; j < KJ * 4; ++j) {
-        const int d = 4 * (l + 8 * (j >> 2)) + (j & 3);
-        if (live && d < a.dim) a.state[((size_t)head * a.dim + d) * ldv + c] = s[j];
-    }
+    for (int x = 0; x < 2; ++x)
+#pragma unroll
+        for (int j = 0; j < KJ * 4; ++j)
+            if (exists(x, j)) a.state[place(x, j)] = s[x][j];
     // the convolutions' last inputs; the preparation kernel has read the older ones
     if (blockIdx.x == 0) {
         const int n_q = a.kv_heads * a.dim, n_ch = 2 * n_q + nv;
@@ -350,6 +383,8 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
     }
 }
 
+static int delta_padded(int dim) { return dim <= 64 ? 64 : dim <= 128 ? 128 : 256; }
+
 static size_t delta_work_floats(int M, int heads, int kv_heads, int dp, int vp, int vdim, DeltaLaunch* L, float* work) {
     const size_t blocks = (M + kDeltaBlock - 1) / kDeltaBlock;
     const size_t kq = blocks * kv_heads * 16 * dp, v = blocks * heads * 8 * vp, coef = blocks * heads * kDeltaCoef;
@@ -365,20 +400,24 @@ int launch_delta(const DeltaArgs& a, cudaStream_t st, unsigned long long* n_kern
         const int ldv = round_up(a.vdim, 4);
         int nc2 = 1;
         while (nc2 < ldv / 4) nc2 *= 2;
-        const size_t smem = 4 * (size_t)(round_up(2 * a.dim, 4) + ldv + 2 * (kDeltaThreads / nc2) * ldv);
+        const int threads = (size_t)a.dim * nc2 <= 8 * 256 ? 256 : 512;
+        const size_t smem = 4 * (size_t)(round_up(2 * a.dim, 4) + ldv + 2 * (threads / nc2) * ldv);
         *n_kernels += 1;
         auto go = [&](auto kernel) {
             if (int rc = allow_smem(kernel, smem)) return rc;
-            return launch_kernel(kernel, dim3(a.heads, a.M), dim3(kDeltaThreads), smem, st, a.use_pdl, 1, a);
+            return launch_kernel(kernel, dim3(a.heads, a.M), dim3(threads), smem, st, a.use_pdl, 1, a);
         };
-        return a.f32 ? go(delta_decode_kernel<float>) : go(delta_decode_kernel<bf16>);
+        if (threads == 256) return a.f32 ? go(delta_decode_kernel<float, 256>) : go(delta_decode_kernel<bf16, 256>);
+        return a.f32 ? go(delta_decode_kernel<float, 512>) : go(delta_decode_kernel<bf16, 512>);
     }
     DeltaLaunch L;
     L.a = a;
-    L.dp = a.dim <= 32 ? 32 : a.dim <= 64 ? 64 : a.dim <= 128 ? 128 : 256;
+    L.dp = delta_padded(a.dim);
     L.vp = round_up(a.vdim, kDeltaCols);
     delta_work_floats(a.M, a.heads, a.kv_heads, L.dp, L.vp, a.vdim, &L, a.work);
-    delta_prepare_kernel<<<dim3((a.M + kDeltaBlock - 1) / kDeltaBlock, a.kv_heads), kDeltaThreads, 64 * (size_t)L.dp, st>>>(L);
+    const dim3 blocks((a.M + kDeltaBlock - 1) / kDeltaBlock, a.kv_heads);
+    if (a.taps <= 4) delta_prepare_kernel<4><<<blocks, kDeltaThreads, 64 * (size_t)L.dp, st>>>(L);
+    else delta_prepare_kernel<kMaxTaps><<<blocks, kDeltaThreads, 64 * (size_t)L.dp, st>>>(L);
     const dim3 grid(L.vp / kDeltaCols, a.heads);
     auto go = [&](auto kernel) {
         const size_t smem = 4 * (size_t)kDeltaStages * (16 * L.dp + 8 * kDeltaCols + kDeltaCoef);
@@ -386,7 +425,7 @@ int launch_delta(const DeltaArgs& a, cudaStream_t st, unsigned long long* n_kern
         kernel<<<grid, 128, smem, st>>>(L);
         return (int)cudaGetLastError();
     };
-    const int rc = L.dp == 32 ? go(delta_block_kernel<1>) : L.dp == 64 ? go(delta_block_kernel<2>) : L.dp == 128 ? go(delta_block_kernel<4>) : go(delta_block_kernel<8>);
+    const int rc = L.dp == 64 ? go(delta_block_kernel<1>) : L.dp == 128 ? go(delta_block_kernel<2>) : go(delta_block_kernel<4>);
     if (rc) return rc;
     ScanArgs s;                                          // per head: o / rms(o) * norm * silu(g)
     s.M = a.M; s.heads = a.heads; s.vdim = a.vdim; s.o_rows = L.o; s.eps = a.eps; s.norm = a.norm;
@@ -406,6 +445,5 @@ extern "C" int tenzo_cuda_delta_rule(const tenzo_delta_args* args, void* stream)
 }
 
 extern "C" size_t tenzo_cuda_delta_rule_work_floats(int M, int heads, int kv_heads, int dim, int vdim) {
-    const int dp = dim <= 32 ? 32 : dim <= 64 ? 64 : dim <= 128 ? 128 : 256;
-    return tz::delta_work_floats(M, heads, kv_heads, dp, tz::round_up(vdim, tz::kDeltaCols), vdim, nullptr, nullptr);
+    return tz::delta_work_floats(M, heads, kv_heads, tz::delta_padded(dim), tz::round_up(vdim, tz::kDeltaCols), vdim, nullptr, nullptr);
 }

@@ -9,6 +9,7 @@
 // the CTA that finishes a tile last adds the partials in split order (a counter decides, nobody waits), so results do
 // not depend on timing.
 #include <algorithm>
+#include <cmath>
 
 #include "hybrid_common.cuh"
 #include "umma.cuh"
@@ -175,13 +176,14 @@ __global__ void __launch_bounds__(kGuThreads, 1) gemm_umma_kernel(const GuLaunch
     } else if (warp == 1) {
         if (lane == 0) {
             // d = f32, a = b = bf16, both K-major, N at bit 17 (>>3), M at bit 24 (>>4)
-            const uint32_t idesc = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(N >> 3) << 17) | ((uint32_t)(kGuRows >> 4) << 24);
+            const uint32_t idesc0 = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(kGuRows >> 4) << 24);
             int it = 0, n = 0;
             for (int u = blockIdx.x; !timed_out && walk.at(L, u, t); u += gridDim.x, ++n) {
                 const int half = n & 1, use_acc = n >> 1;
                 if (use_acc > 0 && !mbar_spin_bounded(&bar_acc_empty[half], (unsigned)(use_acc - 1) & 1u)) { timed_out = true; break; }
                 tc_fence_after();
                 const uint32_t d = tmem_base + (uint32_t)(half * L.tmem_half);
+                const uint32_t idesc = idesc0 | ((uint32_t)(min(N, (t.m_end - t.m0 + 15) & ~15) >> 3) << 17);      // only rows that exist
                 uint32_t acc = 0;
                 for (int j = k_begin(); j < k_end(); ++j, ++it) {
                     const int s = it % kGuStages, use = it / kGuStages;
@@ -273,8 +275,9 @@ bool gemm_umma_applicable(const GemmArgs& a) {
 int launch_gemm_umma(const GemmArgs& a, cudaStream_t st) {
     GuLaunch L;
     L.a = a;
-    // grouped: about a group's mean number of rows, so that most groups are one tile
-    L.n_box = std::min(kGuMaxN, round_up(a.group_off ? std::max(1, a.M / a.n_group) : a.M, 16));
+    // grouped: equal tiles that cover a group somewhat larger than the mean
+    const int mean = a.group_off ? std::max(1, a.M / a.n_group) : 0, rows = a.group_off ? std::min(a.M, mean + 2 * (int)std::sqrt((double)mean)) : a.M;
+    L.n_box = a.group_off ? round_up((rows + (rows + kGuMaxN - 1) / kGuMaxN - 1) / ((rows + kGuMaxN - 1) / kGuMaxN), 16) : std::min(kGuMaxN, round_up(rows, 16));
     L.tmem_half = 32;
     while (L.tmem_half < L.n_box) L.tmem_half *= 2;
     L.n_tiles = (a.N + kGuRows - 1) / kGuRows;

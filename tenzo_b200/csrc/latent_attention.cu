@@ -4,8 +4,7 @@
 // Decode never expands the cache: a head's key matrix is moved to the query (q_h W_uk,h, latent_absorb_kernel), which then
 // scores the latents themselves, the weighted sum of latents is the heads' common value, and the value matrix follows as
 // a product with one segment per head. All heads of a sequence share every key, so a CTA takes 16 heads at once on
-// mma.sync (bf16; queries and weights enter as the sum of two bf16 values, so that rounding them costs nothing visible) or
-// eight with FMA arithmetic (fp32), and a thread-block cluster splits the keys.
+// mma.sync (bf16) or eight with FMA arithmetic (fp32), and a thread-block cluster splits the keys.
 // Chunk: history and new rows side by side, keys and values of all heads in one product, then attention over linear rows.
 // A layer that borrows another one's cache finds that layer's new rows already there, in both forms.
 #include <cooperative_groups.h>
@@ -136,7 +135,7 @@ __device__ __forceinline__ void latent_merge(const LatentLaunch& L, cg::cluster_
     const LatentAttnArgs& a = L.a;
     const int rank = (int)cluster.block_rank(), n_rank = (int)cluster.num_blocks();
     cluster.sync();
-    for (int i = rank * kLtThreads + threadIdx.x; i < nh * L.ld_c; i += n_rank * kLtThreads) {
+    for (int i = rank * (int)blockDim.x + threadIdx.x; i < nh * L.ld_c; i += n_rank * (int)blockDim.x) {
         const int h = i / L.ld_c, d = i - h * L.ld_c;
         if (h0 + h >= a.heads) continue;
         float mx = -1e30f;
@@ -204,22 +203,26 @@ __global__ void __launch_bounds__(kLtThreads) latent_decode_kernel(const LatentL
     latent_merge<T>(L, cluster, seq, h0, kLtFmaHeads, s_k, s_ml);
 }
 
-// bf16 cache on tensor cores: tiles of 64 keys, warps over keys for the scores and over 16-column blocks for the sums.
+// bf16 cache on tensor cores: tiles of 64 keys for 16 heads, 16 warps. Scores: a warp takes eight keys and half of the
+// elements, whose query fragments stay in its registers; softmax: a warp per head; sums: 16-column blocks over the warps.
+// The weights enter the second product as the sum of two bf16 values, so that rounding them costs nothing visible.
+constexpr int kLmThreads = 512;
+
 struct LatentSmem {
     int ks;                                              // elements of a padded row
-    size_t q, k, s, p, bytes;
+    size_t k, s, p, bytes;
     __host__ __device__ LatentSmem(int ld_c, int rot8) {
         ks = ld_c + (rot8 + 31) / 32 * 32 + 8;
-        q = 0;                                           // [2: value, rest][16][ks] bf16
-        k = q + (size_t)2 * kLtHeads * ks * 2;           // [2][64][ks] bf16; the sums at the end
-        s = k + (size_t)2 * kLtTile * ks * 2;            // [16][68] fp32 scores
-        p = s + (size_t)kLtHeads * 68 * 4;               // [2: value, rest][16][72] bf16 weights
+        k = 0;                                           // [2][64][ks] bf16, the queries [16][ks] at first in the second; the sums at the end
+        s = k + (size_t)2 * kLtTile * ks * 2;            // [2 halves][16][68] fp32 scores
+        p = s + (size_t)2 * kLtHeads * 68 * 4;           // [2: value, rest][16][72] bf16 weights
         bytes = p + (size_t)2 * kLtHeads * 72 * 2;
     }
 };
 
-template <int NP>
-__global__ void __launch_bounds__(kLtThreads) latent_decode_mma_kernel(const LatentLaunch L) {
+// NP: 16-column blocks of the latent per warp; PH: 32-element steps per half.
+template <int NP, int PH>
+__global__ void __launch_bounds__(kLmThreads, 1) latent_decode_mma_kernel(const LatentLaunch L) {
     extern __shared__ __align__(16) unsigned char smem[];
     __shared__ float s_f[kLtHeads], s_ml[2 * kLtHeads];
     const LatentAttnArgs& a = L.a;
@@ -227,38 +230,48 @@ __global__ void __launch_bounds__(kLtThreads) latent_decode_mma_kernel(const Lat
     cg::cluster_group cluster = cg::this_cluster();
     const int rank = (int)cluster.block_rank(), n_rank = (int)cluster.num_blocks();
     const int h0 = blockIdx.y * kLtHeads, seq = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
-    const int ks = o.ks, ldk = ks - 8, n_chunk = (L.ld_c + L.rot8) / 8, c_chunk = L.ld_c / 8;
-    bf16 *s_q = reinterpret_cast<bf16*>(smem + o.q), *s_k = reinterpret_cast<bf16*>(smem + o.k), *s_p = reinterpret_cast<bf16*>(smem + o.p);
+    const int ks = o.ks, ldk = ks - 8, n_chunk = (L.ld_c + L.rot8) / 8, c_chunk = L.ld_c / 8, n_step = ldk / 32;
+    const int kg = warp & 7, half = warp >> 3, p0 = half ? PH : 0, n_p = min(PH, n_step - p0);      // this warp's keys and steps
+    bf16 *s_k = reinterpret_cast<bf16*>(smem + o.k), *s_q = s_k + kLtTile * ks, *s_p = reinterpret_cast<bf16*>(smem + o.p);
     float* s_s = reinterpret_cast<float*>(smem + o.s);
-    for (int i = tid; i < 2 * kLtTile * ks / 8; i += kLtThreads) reinterpret_cast<uint4*>(s_k)[i] = make_uint4(0, 0, 0, 0);   // padding
+    for (int i = tid; i < kLtTile; i += kLmThreads)      // padding behind the rotated part
+        for (int x = 0; x < 2; ++x)
+            for (int c = L.ld_c + L.rot8; c < ks; c += 8) *reinterpret_cast<uint4*>(s_k + (size_t)(x * kLtTile + i) * ks + c) = make_uint4(0, 0, 0, 0);
     pdl_wait();
     pdl_launch_dependents();
     const int pos = a.pos[seq], n_keys = min(pos + 1, a.window), first = pos + 1 - n_keys;
     const bf16* rc = static_cast<const bf16*>(a.ring_c) + (size_t)seq * a.ring_c_stride;
     const bf16* rr = static_cast<const bf16*>(a.ring_r) + (size_t)seq * a.ring_r_stride;
     const int per = (n_keys + n_rank - 1) / n_rank, j0 = min(n_keys, rank * per), j1 = min(n_keys, j0 + per);
-    const int n_tiles = (j1 - j0 + kLtTile - 1) / kLtTile;
+    const int n_tiles = (j1 - j0 + kLtTile - 1) / kLtTile, slot0 = (first + j0) % a.ring;
     auto fetch = [&](int tile) {                         // a warp takes whole rows; rows past the end repeat the last one
         bf16* dst = s_k + (tile & 1) * kLtTile * ks;
-        for (int r = warp; r < kLtTile; r += kLtThreads / 32) {
-            const size_t slot = (first + min(j0 + tile * kLtTile + r, j1 - 1)) % a.ring;
+#pragma unroll
+        for (int i = 0; i < kLtTile * 32 / kLmThreads; ++i) {
+            const int r = warp + i * (kLmThreads / 32), k = slot0 + min(tile * kLtTile + r, j1 - j0 - 1);
+            const size_t slot = k >= a.ring ? k - a.ring : k;
             for (int c = lane; c < n_chunk; c += 32)
                 cp16(dst + r * ks + c * 8, c < c_chunk ? rc + slot * L.ld_c + c * 8 : rr + slot * L.rot8 + (c - c_chunk) * 8);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
-    __syncthreads();                                     // the padding is zero before copies land beside it
     if (n_tiles > 0) fetch(0);
-    for (int i = tid; i < kLtHeads * ldk; i += kLtThreads) {
+    for (int i = tid; i < kLtHeads * ldk; i += kLmThreads) {
         const int h = i / ldk, d = i - h * ldk;
-        const float v = latent_query(L, seq, h0 + h, d, pos);
-        const bf16 hi = __float2bfloat16_rn(v);
-        s_q[h * ks + d] = hi;
-        s_q[(kLtHeads + h) * ks + d] = __float2bfloat16_rn(v - __bfloat162float(hi));
+        s_q[h * ks + d] = __float2bfloat16_rn(latent_query(L, seq, h0 + h, d, pos));
     }
-    float m[2] = {-1e30f, -1e30f}, l[2] = {0.0f, 0.0f}, acc[NP][2][4] = {};      // m, l: heads 2 warp, 2 warp + 1
-    const int n_pair = L.ld_c / 16;
+    __syncthreads();
+    uint32_t q[PH][2][4];
     const uint32_t aq = smem_addr(s_q) + 2 * ((lane & 15) * ks + (lane >> 4) * 8), ap = smem_addr(s_p) + 2 * ((lane & 15) * 72 + (lane >> 4) * 8);
+#pragma unroll
+    for (int i = 0; i < PH; ++i)
+        if (i < n_p) {
+            ldsm4(q[i][0], aq + 2 * (p0 + i) * 32);
+            ldsm4(q[i][1], aq + 2 * ((p0 + i) * 32 + 16));
+        }
+    __syncthreads();                                     // the queries' place becomes the second stage
+    float m = -1e30f, l = 0.0f, acc[NP][2][4] = {};      // m, l: head `warp`
+    const int n_pair = L.ld_c / 16;
     for (int tile = 0; tile < n_tiles; ++tile) {
         if (tile + 1 < n_tiles) {
             fetch(tile + 1);
@@ -267,40 +280,32 @@ __global__ void __launch_bounds__(kLtThreads) latent_decode_mma_kernel(const Lat
             asm volatile("cp.async.wait_group 0;" ::: "memory");
         }
         __syncthreads();
-        const uint32_t bk = smem_addr(s_k + (tile & 1) * kLtTile * ks);
-        float sc[4][4] = {};
-        for (int kt = 0; kt < ldk; kt += 32) {
-            uint32_t b[4], q0[4], q1[4], r0[4], r1[4];
-            ldsm4(b, bk + 2 * ((warp * 8 + (lane & 7)) * ks + kt + (lane >> 3) * 8));
-            ldsm4(q0, aq + 2 * kt);
-            ldsm4(q1, aq + 2 * (kt + 16));
-            ldsm4(r0, aq + 2 * (kLtHeads * ks + kt));
-            ldsm4(r1, aq + 2 * (kLtHeads * ks + kt + 16));
-            mma_bf16(sc[0], q0, b[0], b[1]);
-            mma_bf16(sc[1], q1, b[2], b[3]);
-            mma_bf16(sc[2], r0, b[0], b[1]);
-            mma_bf16(sc[3], r1, b[2], b[3]);
-        }
-        const int left = j1 - j0 - tile * kLtTile;       // keys of this tile
+        const uint32_t bk = smem_addr(s_k + (tile & 1) * kLtTile * ks), kr = bk + 2 * ((kg * 8 + (lane & 7)) * ks + (lane >> 3) * 8 + p0 * 32);
+        float sc[2][4] = {};
 #pragma unroll
-        for (int i = 0; i < 4; ++i) {
-            const int key = warp * 8 + t4 * 2 + (i & 1);
-            s_s[(g + (i >> 1) * 8) * 68 + key] = key < left ? (sc[0][i] + sc[1][i]) + (sc[2][i] + sc[3][i]) : -INFINITY;
-        }
+        for (int i = 0; i < PH; ++i)
+            if (i < n_p) {
+                uint32_t b[4];
+                ldsm4(b, kr + 64 * i);
+                mma_bf16(sc[0], q[i][0], b[0], b[1]);
+                mma_bf16(sc[1], q[i][1], b[2], b[3]);
+            }
+#pragma unroll
+        for (int i = 0; i < 4; ++i) s_s[(half * kLtHeads + g + (i >> 1) * 8) * 68 + kg * 8 + t4 * 2 + (i & 1)] = sc[0][i] + sc[1][i];
         __syncthreads();
-#pragma unroll
-        for (int x = 0; x < 2; ++x) {
-            const int h = warp * 2 + x;
-            const float v0 = s_s[h * 68 + lane], v1 = s_s[h * 68 + 32 + lane];
-            const float mn = fmaxf(m[x], warp_max(fmaxf(v0, v1))), f = expf(m[x] - mn), p0 = expf(v0 - mn), p1 = expf(v1 - mn);
-            l[x] = l[x] * f + warp_sum(p0 + p1);
-            m[x] = mn;
-            const bf16 b0 = __float2bfloat16_rn(p0), b1 = __float2bfloat16_rn(p1);
-            s_p[h * 72 + lane] = b0;
-            s_p[h * 72 + 32 + lane] = b1;
-            s_p[(kLtHeads + h) * 72 + lane] = __float2bfloat16_rn(p0 - __bfloat162float(b0));
-            s_p[(kLtHeads + h) * 72 + 32 + lane] = __float2bfloat16_rn(p1 - __bfloat162float(b1));
-            if (lane == 0) s_f[h] = f;
+        {
+            const int left = j1 - j0 - tile * kLtTile;   // keys of this tile
+            const float *s0 = s_s + warp * 68, *s1 = s_s + (kLtHeads + warp) * 68;
+            const float v0 = lane < left ? s0[lane] + s1[lane] : -INFINITY, v1 = lane + 32 < left ? s0[lane + 32] + s1[lane + 32] : -INFINITY;
+            const float mn = fmaxf(m, warp_max(fmaxf(v0, v1))), f = expf(m - mn), e0 = expf(v0 - mn), e1 = expf(v1 - mn);
+            l = l * f + warp_sum(e0 + e1);
+            m = mn;
+            const bf16 b0 = __float2bfloat16_rn(e0), b1 = __float2bfloat16_rn(e1);
+            s_p[warp * 72 + lane] = b0;
+            s_p[warp * 72 + 32 + lane] = b1;
+            s_p[(kLtHeads + warp) * 72 + lane] = __float2bfloat16_rn(e0 - __bfloat162float(b0));
+            s_p[(kLtHeads + warp) * 72 + 32 + lane] = __float2bfloat16_rn(e1 - __bfloat162float(b1));
+            if (lane == 0) s_f[warp] = f;
         }
         __syncthreads();
         const float f0 = s_f[g], f1 = s_f[g + 8];
@@ -318,13 +323,13 @@ __global__ void __launch_bounds__(kLtThreads) latent_decode_mma_kernel(const Lat
             ldsm4(rest, ap + 2 * (kLtHeads * 72 + kt * 16));
 #pragma unroll
             for (int i = 0; i < NP; ++i) {
-                const int pair = warp + i * 8;
+                const int pair = warp + i * 16;
                 if (pair >= n_pair) break;
                 uint32_t b[4];
                 ldsm4t(b, bk + 2 * ((kt * 16 + (lane & 7) + ((lane >> 3) & 1) * 8) * ks + pair * 16 + (lane >> 4) * 8));
                 mma_bf16(acc[i][0], p, b[0], b[1]);
-                mma_bf16(acc[i][0], rest, b[0], b[1]);
                 mma_bf16(acc[i][1], p, b[2], b[3]);
+                mma_bf16(acc[i][0], rest, b[0], b[1]);
                 mma_bf16(acc[i][1], rest, b[2], b[3]);
             }
         }
@@ -333,17 +338,14 @@ __global__ void __launch_bounds__(kLtThreads) latent_decode_mma_kernel(const Lat
     float* s_acc = reinterpret_cast<float*>(s_k);         // [16][ld_c]
 #pragma unroll
     for (int i = 0; i < NP; ++i) {
-        const int pair = warp + i * 8;
+        const int pair = warp + i * 16;
         if (pair >= n_pair) break;
 #pragma unroll
         for (int x = 0; x < 2; ++x)
 #pragma unroll
             for (int e = 0; e < 4; ++e) s_acc[(g + (e >> 1) * 8) * L.ld_c + pair * 16 + x * 8 + t4 * 2 + (e & 1)] = acc[i][x][e];
     }
-    if (lane < 2) {
-        s_ml[warp * 2 + lane] = lane ? m[1] : m[0];
-        s_ml[kLtHeads + warp * 2 + lane] = lane ? l[1] : l[0];
-    }
+    if (lane == 0) { s_ml[warp] = m; s_ml[kLtHeads + warp] = l; }
     latent_merge<bf16>(L, cluster, seq, h0, kLtHeads, s_acc, s_ml);
 }
 
@@ -415,14 +417,16 @@ static int latent_decode(const LatentLaunch& L, cudaStream_t st, unsigned long l
     int cl = 1;                                          // slices of at least 64 keys, more than one only while SMs are free
     while (cl < 8 && a.ring > 64 * cl && (long long)2 * cl * tiles * a.M <= 148) cl *= 2;
     const dim3 grid(cl, tiles, a.M);
-    auto go = [&](auto kernel, size_t smem) {
+    auto go = [&](auto kernel, size_t smem, int threads = kLtThreads) {
         if (smem > 220 * 1024) return -1;
         if (int rc = allow_smem(kernel, smem)) return rc;
-        return launch_kernel(kernel, grid, dim3(kLtThreads), smem, st, a.use_pdl, cl, L);
+        return launch_kernel(kernel, grid, dim3(threads), smem, st, a.use_pdl, cl, L);
     };
     int rc;
     if (mma) {
-        rc = L.ld_c <= 128 ? go(latent_decode_mma_kernel<1>, o.bytes) : L.ld_c <= 256 ? go(latent_decode_mma_kernel<2>, o.bytes) : go(latent_decode_mma_kernel<4>, o.bytes);
+        const int steps = (o.ks - 8) / 32;               // of 32 elements, over two halves
+        rc = L.ld_c <= 256 ? (steps <= 6 ? go(latent_decode_mma_kernel<1, 3>, o.bytes, kLmThreads) : go(latent_decode_mma_kernel<1, 8>, o.bytes, kLmThreads))
+                           : (steps <= 18 ? go(latent_decode_mma_kernel<2, 9>, o.bytes, kLmThreads) : go(latent_decode_mma_kernel<2, 12>, o.bytes, kLmThreads));
     } else {
         const int ldk = L.ld_c + L.rot8;
         const size_t smem = 4 * ((size_t)kLtFmaHeads * ldk + kLtFmaTile * (ldk + 1));

@@ -4,6 +4,7 @@
 // Decode, and rows that carry nothing from one to the next: one CTA per row does all of it; a thread keeps its columns in
 // registers, with the convolution's weights and the carried inputs fetched before the kernel waits for its producer (the
 // launch that wrote them lies a whole step back).
+// Rows without convolution and mixes (designs that have none) take a kernel of 256 threads and 16-byte pieces instead.
 // Chunk (and decode of rows wider than that): one kernel updates the residual and leaves each row's inverse RMS, a second
 // one walks tiles of rows per channel with the convolution's inputs in registers.
 #include "hybrid_common.cuh"
@@ -145,6 +146,87 @@ __global__ void __launch_bounds__(kStepThreads) rows_step_kernel(const RowsArgs 
     }
 }
 
+// Rows without convolution and mixes, four columns at a time: NV pieces per thread, weights fetched ahead of the wait.
+constexpr int kPlainThreads = 256;
+
+__device__ __forceinline__ float sum4(const float4& a, const float4& b) { return fmaf(a.x, b.x, fmaf(a.y, b.y, fmaf(a.z, b.z, a.w * b.w))); }
+__device__ __forceinline__ float4 fma4(float s, const float4& a, const float4& b) {
+    return make_float4(fmaf(s, a.x, b.x), fmaf(s, a.y, b.y), fmaf(s, a.z, b.z), fmaf(s, a.w, b.w));
+}
+__device__ __forceinline__ void store4(float* p, const float4& v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void store4(bf16* p, const float4& v) {
+    const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = make_uint2(reinterpret_cast<const uint32_t&>(lo), reinterpret_cast<const uint32_t&>(hi));
+}
+
+template <typename T, int NV>
+__global__ void __launch_bounds__(kPlainThreads) rows_plain_kernel(const RowsArgs a) {
+    __shared__ float2 s_red[2][32];
+    const int t = blockIdx.x, width = a.width;
+    float4 w[NV], g[NV], x[NV], y[NV];
+    const float4 one = make_float4(1, 1, 1, 1), zero = make_float4(0, 0, 0, 0);
+    auto at = [&](int i) { return (threadIdx.x + i * kPlainThreads) * 4; };
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        w[i] = a.w0 && at(i) < width ? *reinterpret_cast<const float4*>(a.w0 + at(i)) : one;
+        g[i] = a.gain_w && at(i) < width ? *reinterpret_cast<const float4*>(a.gain_w + at(i)) : one;
+        x[i] = y[i] = zero;
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    if (a.tokens) {
+        const bf16* e = static_cast<const bf16*>(a.embed) + (size_t)min(max(a.tokens[t], 0), a.vocab - 1) * width;
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (at(i) < width) {
+                const uint2 u = *reinterpret_cast<const uint2*>(e + at(i));
+                bf16x2_to_f(u.x, x[i].x, x[i].y);
+                bf16x2_to_f(u.y, x[i].z, x[i].w);
+            }
+    } else {
+#pragma unroll
+        for (int i = 0; i < NV; ++i)
+            if (at(i) < width) x[i] = *reinterpret_cast<const float4*>(a.x_in + (size_t)t * width + at(i));
+        if (a.y_slot) {
+            for (int j = 0; j < a.n_y; ++j) {
+                const float s = a.y_weight[(size_t)t * a.n_y + j];
+                const float* src = a.y0 + (size_t)a.y_slot[(size_t)t * a.n_y + j] * a.ld_y;
+#pragma unroll
+                for (int i = 0; i < NV; ++i)
+                    if (at(i) < width) y[i] = fma4(s, *reinterpret_cast<const float4*>(src + at(i)), y[i]);
+            }
+        } else if (a.y0) {
+#pragma unroll
+            for (int i = 0; i < NV; ++i)
+                if (at(i) < width) y[i] = *reinterpret_cast<const float4*>(a.y0 + (size_t)t * a.ld_y + at(i));
+        }
+    }
+    float inv = 1.0f;
+    if (a.w0 && !a.tokens) {
+        float q = 0.0f;
+#pragma unroll
+        for (int i = 0; i < NV; ++i) q += sum4(y[i], y[i]);
+        q = block_sum2(make_float2(q, 0.0f), s_red[0]).x;
+        inv = 1.0f / sqrtf(q / (float)width + a.eps);
+    }
+    float q = 0.0f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+        x[i].x += y[i].x * inv * w[i].x; x[i].y += y[i].y * inv * w[i].y; x[i].z += y[i].z * inv * w[i].z; x[i].w += y[i].w * inv * w[i].w;
+        q += sum4(x[i], x[i]);
+        if (at(i) < width) *reinterpret_cast<float4*>(a.x_out + (size_t)t * width + at(i)) = x[i];
+    }
+    q = block_sum2(make_float2(q, 0.0f), s_red[1]).x;
+    inv = 1.0f / sqrtf(q / (float)width + a.eps);
+    T* out = reinterpret_cast<T*>(a.out) + (size_t)t * a.ld_out;
+#pragma unroll
+    for (int i = 0; i < NV; ++i)
+        if (at(i) < width) {
+            const float s = inv * a.gain;
+            store4(out + at(i), make_float4(x[i].x * s * g[i].x, x[i].y * s * g[i].y, x[i].z * s * g[i].z, x[i].w * s * g[i].w));
+        }
+}
+
 // Residual and inverse RMS of a row.
 __global__ void __launch_bounds__(kNormThreads) rows_norm_kernel(const RowsArgs a) {
     __shared__ float2 s_red[2][32];
@@ -249,6 +331,13 @@ int launch_rows(const RowsArgs& a, cudaStream_t st, unsigned long long* n_kernel
     if (a.taps < 1 || a.taps > kMaxTaps || a.width <= 0 || a.n_mix > 8) return -1;
     if ((a.y_slot && (!a.y_weight || a.n_y < 1)) || (a.y1 && !a.w0)) return -1;
     const bool alone = a.decode || (!a.conv_w && !a.mu);          // no row looks at another one of the launch
+    if (!a.conv_w && !a.mu && !a.y1 && !a.pos_table && a.width <= 16 * kPlainThreads && a.width % 4 == 0 && a.ld_out % 4 == 0 && a.ld_y % 4 == 0) {
+        auto go = [&](auto kernel) { return launch_kernel(kernel, dim3(a.M), dim3(kPlainThreads), 0, st, a.use_pdl, 1, a); };
+        *n_kernels += 1;
+        const int nv = (a.width + 4 * kPlainThreads - 1) / (4 * kPlainThreads);
+        if (a.f32) return nv == 1 ? go(rows_plain_kernel<float, 1>) : nv == 2 ? go(rows_plain_kernel<float, 2>) : nv == 3 ? go(rows_plain_kernel<float, 3>) : go(rows_plain_kernel<float, 4>);
+        return nv == 1 ? go(rows_plain_kernel<bf16, 1>) : nv == 2 ? go(rows_plain_kernel<bf16, 2>) : nv == 3 ? go(rows_plain_kernel<bf16, 3>) : go(rows_plain_kernel<bf16, 4>);
+    }
     if (alone && a.width <= kStepThreads * kStepMaxCols && a.taps <= kStepTaps) {
         auto go = [&](auto kernel) { return launch_kernel(kernel, dim3(a.M), dim3(kStepThreads), 0, st, a.use_pdl, 1, a); };
         *n_kernels += 1;
