@@ -16,18 +16,23 @@
 namespace tz {
 
 constexpr int kDeltaThreads = 256;
-constexpr int kDeltaBlock = 8, kDeltaCols = 16, kDeltaStages = 4;
+constexpr int kDeltaBlock = 8, kDeltaCols = 8, kDeltaStages = 4, kDeltaBlockThreads = 64;
 constexpr int kDeltaCoef = 2 * kDeltaBlock * kDeltaBlock + 2 * kDeltaBlock;   // inverse * beta, read-out, decays from the start, to the end
 
 __device__ __forceinline__ float softplus_f(float z) { return softplus_neg(-z); }
 __device__ __forceinline__ float head_log_decay(const DeltaArgs& a, int head, float z) { return -expf(a.a_log[head]) * softplus_f(z + a.dt_bias[head]); }
 
 // ---- decode --------------------------------------------------------------------------------------------------------------
-// convolution and silu of one channel at position pos; rows of the tail that no token of the sequence has written are zero
-__device__ __forceinline__ float conv_at(const float* w, int ch, int n_ch, int taps, const float* tail, int tail_ld, int pos, float cur) {
-    float y = w[(size_t)(taps - 1) * n_ch + ch] * cur;
-    for (int j = 1; j < taps; ++j) y = fmaf(w[(size_t)(taps - 1 - j) * n_ch + ch], tail[(size_t)((pos + taps - j) % taps) * tail_ld], y);
-    return silu_f(y);
+// The older inputs' part of one channel's convolution at position pos; rows of the tail that no token of the sequence has
+// written are zero.
+__device__ __forceinline__ float conv_before(const float* w, int ch, int n_ch, int taps, const float* tail, int tail_ld, int pos) {
+    float y = 0.0f;
+    int slot = pos % taps;
+    for (int j = 1; j < taps; ++j) {
+        slot = slot == 0 ? taps - 1 : slot - 1;
+        y = fmaf(w[(size_t)(taps - 1 - j) * n_ch + ch], tail[(size_t)slot * tail_ld], y);
+    }
+    return y;
 }
 
 // THREADS 256 or 512, whichever lets a thread hold its part of the state in kPre pieces for most sizes.
@@ -56,30 +61,48 @@ __global__ void __launch_bounds__(THREADS, 1024 / THREADS) delta_decode_kernel(c
     float* s_b = s_a + n_rg * ldv;
     const int group = a.heads / a.kv_heads, kvh = head / group;
     const int n_q = a.kv_heads * a.dim, n_v = a.heads * a.vdim, n_ch = 2 * n_q + n_v;
+    // the position and the convolutions' older inputs were written a whole step ago, like the state
+    const int pos = a.pos[seq], chq = kvh * a.dim + tid, chv = head * a.vdim + tid;
+    float* tail = a.tail + (size_t)seq * a.tail_seq_stride;
+    float* newest = tail + (size_t)(pos % a.taps) * n_ch;
+    const bool has_q = tid < a.dim, has_v = tid < a.vdim;  // head sizes are at most one thread per element
+    const size_t last = a.taps - 1;
+    float q = 0.0f, k = 0.0f, v = 0.0f, wq = 0.0f, wk = 0.0f, wv = 0.0f, gain = 0.0f, uq = 0.0f, uk = 0.0f, uv = 0.0f, gate = 0.0f;
+    if (has_q) {
+        wq = a.conv_q[last * n_q + chq];
+        wk = a.conv_k[last * n_q + chq];
+        q = conv_before(a.conv_q, chq, n_q, a.taps, tail + chq, n_ch, pos);
+        k = conv_before(a.conv_k, chq, n_q, a.taps, tail + n_q + chq, n_ch, pos);
+    }
+    if (has_v) {
+        wv = a.conv_v[last * n_v + chv];
+        gain = a.norm[tid];
+        v = conv_before(a.conv_v, chv, n_v, a.taps, tail + 2 * n_q + chv, n_ch, pos);
+    }
     pdl_wait();
     pdl_launch_dependents();
     const size_t row = (size_t)seq * a.ld;
-    const int pos = a.pos[seq];
-    float* tail = a.tail + (size_t)seq * a.tail_seq_stride;
-    float* newest = tail + (size_t)(pos % a.taps) * n_ch;
-    float q = 0.0f, k = 0.0f, v = 0.0f;
-    if (tid < a.dim) {                                   // head sizes are at most one thread per element
-        const int ch = kvh * a.dim + tid;
-        const float uq = a.q[row + ch], uk = a.k[row + ch];
-        q = conv_at(a.conv_q, ch, n_q, a.taps, tail + ch, n_ch, pos, uq);
-        k = conv_at(a.conv_k, ch, n_q, a.taps, tail + n_q + ch, n_ch, pos, uk);
-        if (head % group == 0) {
-            newest[ch] = uq;
-            newest[n_q + ch] = uk;
-        }
+    if (has_q) {
+        uq = a.q[row + chq];
+        uk = a.k[row + chq];
     }
-    if (tid < a.vdim) {
-        const int ch = head * a.vdim + tid;
-        const float uv = a.v[row + ch];
-        v = conv_at(a.conv_v, ch, n_v, a.taps, tail + 2 * n_q + ch, n_ch, pos, uv);
-        newest[2 * n_q + ch] = uv;
+    if (has_v) {
+        uv = a.v[row + chv];
+        gate = a.g[row + chv];
     }
     const float g = expf(head_log_decay(a, head, a.a[row + head])), beta = sigmoid_f(a.b[row + head]);
+    if (has_q) {
+        q = silu_f(fmaf(wq, uq, q));
+        k = silu_f(fmaf(wk, uk, k));
+        if (head % group == 0) {
+            newest[chq] = uq;
+            newest[n_q + chq] = uk;
+        }
+    }
+    if (has_v) {
+        v = silu_f(fmaf(wv, uv, v));
+        newest[2 * n_q + chv] = uv;
+    }
     const float qq = warp_sum(q * q), kk = warp_sum(k * k), qk = warp_sum(q * k);
     if (lane == 0) { s_red[0][warp] = qq; s_red[1][warp] = kk; s_red[2][warp] = qk; }
     __syncthreads();
@@ -91,7 +114,7 @@ __global__ void __launch_bounds__(THREADS, 1024 / THREADS) delta_decode_kernel(c
         for (int w = 0; w < THREADS / 32; ++w) sums[i] += s_red[i][w];
     }
     const float iq = a.q_scale / sqrtf(sums[0] + a.unit_eps), ik = 1.0f / sqrtf(sums[1] + a.unit_eps), kq = sums[2] * iq * ik;
-    if (tid < a.dim) { s_q[tid] = q * iq; s_k[tid] = k * ik; }
+    if (has_q) { s_q[tid] = q * iq; s_k[tid] = k * ik; }
     __syncthreads();
     if (live) {
         float pa[4] = {}, pb[4] = {};
@@ -118,19 +141,19 @@ __global__ void __launch_bounds__(THREADS, 1024 / THREADS) delta_decode_kernel(c
             sa += s_a[r * ldv + tid];
             sb += s_b[r * ldv + tid];
         }
-        const float u = tid < a.vdim ? beta * (v - g * sa) : 0.0f;
+        const float u = has_v ? beta * (v - g * sa) : 0.0f;
         s_u[tid] = u;
-        if (tid < a.vdim) o = fmaf(g, sb, kq * u);
+        if (has_v) o = fmaf(g, sb, kq * u);
     }
     const float oo = warp_sum(o * o);
     if (lane == 0) s_red[3][warp] = oo;
     __syncthreads();
-    if (tid < a.vdim) {
+    if (has_v) {
         float t = 0.0f;
 #pragma unroll
         for (int w = 0; w < THREADS / 32; ++w) t += s_red[3][w];
-        const float y = o * (1.0f / sqrtf(t / (float)a.vdim + a.eps)) * a.norm[tid];
-        reinterpret_cast<T*>(a.out)[(size_t)seq * a.ld_out + head * a.vdim + tid] = from_f<T>(y * silu_f(a.g[row + head * a.vdim + tid]));
+        const float y = o * (1.0f / sqrtf(t / (float)a.vdim + a.eps)) * gain;
+        reinterpret_cast<T*>(a.out)[(size_t)seq * a.ld_out + chv] = from_f<T>(y * silu_f(gate));
     }
     if (live) {
         const float4 u = *reinterpret_cast<const float4*>(s_u + col * 4);
@@ -273,10 +296,10 @@ __global__ void __launch_bounds__(kDeltaThreads) delta_prepare_kernel(const Delt
     }
 }
 
-// Sixteen value columns of one head, four per warp. Half a warp shares a pair of columns, lane l of it holding the state's rows
+// Eight value columns of one head, four per warp. Half a warp shares a pair of columns, lane l of it holding the state's rows
 // 4 (l + 16 j) .. + 3 of both; once the products are summed, eight lanes stand for the block's eight rows of one column.
 template <int KJ>
-__global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
+__global__ void __launch_bounds__(kDeltaBlockThreads) delta_block_kernel(const DeltaLaunch L) {
     constexpr int DP = 64 * KJ, V = 16 * DP, C = V + 8 * kDeltaCols, FLOATS = C + kDeltaCoef;
     extern __shared__ __align__(16) float smem[];
     const DeltaArgs& a = L.a;
@@ -289,9 +312,10 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
         if (b < n_blocks) {
             float* dst = smem + (b % kDeltaStages) * FLOATS;
             const float* kq = L.kq + ((size_t)b * a.kv_heads + kvh) * 16 * DP;
-            for (int i = tid; i < 4 * DP; i += 128) cp16(dst + 4 * i, kq + 4 * i);
-            if (tid < 32) cp16(dst + V + 4 * tid, L.v + (((size_t)b * a.heads + head) * 8 + tid / 4) * L.vp + blockIdx.x * kDeltaCols + (tid & 3) * 4);
-            else if (tid < 32 + kDeltaCoef / 4) cp16(dst + C + 4 * (tid - 32), L.coef + ((size_t)b * a.heads + head) * kDeltaCoef + 4 * (tid - 32));
+#pragma unroll
+            for (int i = 0; i < 4 * DP / kDeltaBlockThreads; ++i) cp16(dst + 4 * (tid + i * kDeltaBlockThreads), kq + 4 * (tid + i * kDeltaBlockThreads));
+            if (tid < 16) cp16(dst + V + 4 * tid, L.v + (((size_t)b * a.heads + head) * 8 + tid / 2) * L.vp + blockIdx.x * kDeltaCols + (tid & 1) * 4);
+            else if (tid < 16 + kDeltaCoef / 4) cp16(dst + C + 4 * (tid - 16), L.coef + ((size_t)b * a.heads + head) * kDeltaCoef + 4 * (tid - 16));
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
@@ -310,12 +334,14 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
         const float* buf = smem + (b % kDeltaStages) * FLOATS;
         const float *sk = buf + 4 * l, *sq = sk + 8 * DP, *co = buf + C;
         float pa[16], pb[16];                            // [column][row]
+        float4 kr[KJ > 2 ? 1 : 8][KJ];                   // the block's keys, for the update, where registers allow it
 #pragma unroll
         for (int t = 0; t < 8; ++t) {
             float ka[2] = {}, qb[2] = {};
 #pragma unroll
             for (int j = 0; j < KJ; ++j) {
                 const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 64 * j), q4 = *reinterpret_cast<const float4*>(sq + t * DP + 64 * j);
+                if (KJ <= 2) kr[KJ > 2 ? 0 : t][j] = k4;
                 const float kf[4] = {k4.x, k4.y, k4.z, k4.w}, qf[4] = {q4.x, q4.y, q4.z, q4.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i)
@@ -350,7 +376,7 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
             if (KJ > 2) asm volatile("" ::: "memory");
 #pragma unroll
             for (int j = 0; j < KJ; ++j) {
-                const float4 k4 = *reinterpret_cast<const float4*>(sk + t * DP + 64 * j);
+                const float4 k4 = KJ <= 2 ? kr[KJ > 2 ? 0 : t][j] : *reinterpret_cast<const float4*>(sk + t * DP + 64 * j);
                 const float kf[4] = {k4.x, k4.y, k4.z, k4.w};
 #pragma unroll
                 for (int i = 0; i < 4; ++i) {
@@ -374,11 +400,11 @@ __global__ void __launch_bounds__(128) delta_block_kernel(const DeltaLaunch L) {
             float* to = a.tail + (size_t)((a.pos0 + t) % a.taps) * n_ch;
             const size_t row = (size_t)t * a.ld;
             if (head % group == 0)
-                for (int d = tid; d < a.dim; d += 128) {
+                for (int d = tid; d < a.dim; d += kDeltaBlockThreads) {
                     to[kvh * a.dim + d] = a.q[row + kvh * a.dim + d];
                     to[n_q + kvh * a.dim + d] = a.k[row + kvh * a.dim + d];
                 }
-            for (int d = tid; d < a.vdim; d += 128) to[2 * n_q + head * a.vdim + d] = a.v[row + head * a.vdim + d];
+            for (int d = tid; d < a.vdim; d += kDeltaBlockThreads) to[2 * n_q + head * a.vdim + d] = a.v[row + head * a.vdim + d];
         }
     }
 }
@@ -422,7 +448,7 @@ int launch_delta(const DeltaArgs& a, cudaStream_t st, unsigned long long* n_kern
     auto go = [&](auto kernel) {
         const size_t smem = 4 * (size_t)kDeltaStages * (16 * L.dp + 8 * kDeltaCols + kDeltaCoef);
         if (int rc = allow_smem(kernel, smem)) return rc;
-        kernel<<<grid, 128, smem, st>>>(L);
+        kernel<<<grid, kDeltaBlockThreads, smem, st>>>(L);
         return (int)cudaGetLastError();
     };
     const int rc = L.dp == 64 ? go(delta_block_kernel<1>) : L.dp == 128 ? go(delta_block_kernel<2>) : go(delta_block_kernel<4>);

@@ -49,13 +49,26 @@ __device__ __forceinline__ void latent_row(const LatentLaunch& L, const float* s
 }
 
 // ---- decode --------------------------------------------------------------------------------------------------------------
+// The new tokens' cache rows, sequences `first`, `first` + `step`, .. below `end`.
+template <typename T>
+__device__ __forceinline__ void append_rows(const LatentLaunch& L, int first, int end, int step, float* scratch) {
+    const LatentAttnArgs& a = L.a;
+    for (int m = first; m < end; m += step) {
+        const int pos = a.pos[m];
+        const size_t slot = pos % a.ring;
+        latent_row<T>(L, a.dkv + (size_t)m * a.ld, pos, static_cast<T*>(a.ring_c) + (size_t)m * a.ring_c_stride + slot * L.ld_c,
+                      static_cast<T*>(a.ring_r) + (size_t)m * a.ring_r_stride + slot * L.rot8, scratch);
+    }
+}
+
 // 128 columns of the latent for one head and up to MR sequences: 16 threads over the columns, 16 slices of the head's rows.
 // One more head index, when the layer owns its cache, appends the new tokens' rows to the rings.
 template <typename T, int MR>
 __global__ void __launch_bounds__(kLtThreads) latent_absorb_kernel(const LatentLaunch L) {
     extern __shared__ float sm[];
     const LatentAttnArgs& a = L.a;
-    const int h = blockIdx.y, tid = threadIdx.x, cc = (tid & 15) * 8, ds = tid >> 4, c0 = blockIdx.x * 128 + cc, m0 = blockIdx.z * MR, nm = min(MR, a.M - m0);
+    const int h = blockIdx.y, tid = threadIdx.x, cc = (tid & 15) * 8, ds = tid >> 4, c0 = blockIdx.x * 128 + cc;
+    const int m0 = blockIdx.z * MR, nm = min(MR, a.M - m0);
     const bool product = h < a.heads, live = product && c0 < L.ld_c;
     const bf16* w = static_cast<const bf16*>(a.w_kv) + (size_t)(product ? h : 0) * L.dim8 * L.ld_c + c0;
     constexpr int kPre = 8;
@@ -66,17 +79,11 @@ __global__ void __launch_bounds__(kLtThreads) latent_absorb_kernel(const LatentL
     pdl_wait();
     pdl_launch_dependents();
     if (!product) {
-        if (blockIdx.x > 0) return;
-        for (int m = m0; m < m0 + nm; ++m) {
-            const int pos = a.pos[m];
-            const size_t slot = pos % a.ring;
-            latent_row<T>(L, a.dkv + (size_t)m * a.ld, pos, static_cast<T*>(a.ring_c) + (size_t)m * a.ring_c_stride + slot * L.ld_c,
-                          static_cast<T*>(a.ring_r) + (size_t)m * a.ring_r_stride + slot * L.rot8, sm);
-        }
+        append_rows<T>(L, m0 + blockIdx.x, m0 + nm, gridDim.x, sm);
         return;
     }
     float* s_q = sm;                                     // [MR][dim8]
-    float* s_part = sm + MR * L.dim8;                    // [16][MR][128]
+    float* s_part = sm + MR * L.dim8;                    // [8][MR][128]
     for (int i = tid; i < MR * L.dim8; i += kLtThreads) {
         const int m = i / L.dim8, d = i - m * L.dim8;
         s_q[i] = m < nm && d < a.dim ? a.q[(size_t)(m0 + m) * a.ld + (size_t)h * (a.dim + a.rot) + d] : 0.0f;
@@ -100,18 +107,78 @@ __global__ void __launch_bounds__(kLtThreads) latent_absorb_kernel(const LatentL
         for (int d = ds + 16 * kPre; d < a.dim; d += 16) step(ld_stream_u4(w + (size_t)d * L.ld_c), d);
     }
 #pragma unroll
-    for (int m = 0; m < MR; ++m)
+    for (int m = 0; m < MR; ++m) {                       // the two slices of a warp meet in its lower half
 #pragma unroll
-        for (int j = 0; j < 8; ++j) s_part[(ds * MR + m) * 128 + cc + j] = acc[m][j];
+        for (int j = 0; j < 8; ++j) acc[m][j] += __shfl_xor_sync(0xffffffffu, acc[m][j], 16);
+        if ((ds & 1) == 0) {
+            float4* p = reinterpret_cast<float4*>(s_part + ((ds >> 1) * MR + m) * 128 + cc);
+            p[0] = make_float4(acc[m][0], acc[m][1], acc[m][2], acc[m][3]);
+            p[1] = make_float4(acc[m][4], acc[m][5], acc[m][6], acc[m][7]);
+        }
+    }
     __syncthreads();
     for (int i = tid; i < nm * 128; i += kLtThreads) {
         const int m = i >> 7, c = i & 127;
         if (blockIdx.x * 128 + c >= L.ld_c) continue;
         float t = 0.0f;
 #pragma unroll
-        for (int s = 0; s < 16; ++s) t += s_part[(s * MR + m) * 128 + c];
+        for (int s = 0; s < 8; ++s) t += s_part[(s * MR + m) * 128 + c];
         a.q_abs[((size_t)(m0 + m) * a.heads + h) * L.ld_c + blockIdx.x * 128 + c] = t;
     }
+}
+
+// The same for many sequences with bf16 arithmetic, on tensor cores: 64 sequences x 128 columns of one head per CTA, a warp
+// 16 x 64 of them. The head's rows are in shared memory before the wait.
+constexpr int kLaM = 64, kLaN = 128, kLaW = kLaN + 8, kLaMinRows = 12;
+
+__global__ void __launch_bounds__(kLtThreads) latent_absorb_mma_kernel(const LatentLaunch L) {
+    extern __shared__ __align__(16) unsigned char smem[];
+    const LatentAttnArgs& a = L.a;
+    const int h = blockIdx.y, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, c0 = blockIdx.x * kLaN, m0 = blockIdx.z * kLaM, m_end = min(a.M, m0 + kLaM);
+    const int dp = (a.dim + 15) & ~15, qs = dp + 8;
+    bf16 *s_w = reinterpret_cast<bf16*>(smem), *s_q = s_w + dp * kLaW;       // [dp][136], [64][qs]
+    if (h < a.heads) {
+        const bf16* w = static_cast<const bf16*>(a.w_kv) + (size_t)h * L.dim8 * L.ld_c + c0;
+        for (int i = tid; i < dp * (kLaN / 8); i += kLtThreads) {
+            const int d = i / (kLaN / 8), c = (i - d * (kLaN / 8)) * 8;
+            if (d < a.dim && c0 + c < L.ld_c) cp16(s_w + d * kLaW + c, w + (size_t)d * L.ld_c + c);
+            else *reinterpret_cast<uint4*>(s_w + d * kLaW + c) = make_uint4(0, 0, 0, 0);
+        }
+        asm volatile("cp.async.commit_group;" ::: "memory");
+    }
+    pdl_wait();
+    pdl_launch_dependents();
+    if (h >= a.heads) {
+        append_rows<bf16>(L, m0 + blockIdx.x + gridDim.x * (h - a.heads), m_end, gridDim.x * (gridDim.y - a.heads), reinterpret_cast<float*>(smem));
+        return;
+    }
+    for (int m = warp; m < kLaM; m += kLtThreads / 32)
+        for (int d = lane; d < dp; d += 32)
+            s_q[m * qs + d] = __float2bfloat16_rn(m0 + m < m_end && d < a.dim ? a.q[(size_t)(m0 + m) * a.ld + (size_t)h * (a.dim + a.rot) + d] : 0.0f);
+    asm volatile("cp.async.wait_group 0;" ::: "memory");
+    __syncthreads();
+    const int rt = (warp & 3) * 16, ch = (warp >> 2) * 64, g = lane >> 2, t4 = lane & 3;
+    const uint32_t aq = smem_addr(s_q) + 2 * ((rt + (lane & 15)) * qs + (lane >> 4) * 8);
+    const uint32_t bw = smem_addr(s_w) + 2 * (((lane & 7) + ((lane >> 3) & 1) * 8) * kLaW + ch + (lane >> 4) * 8);
+    float acc[8][4] = {};
+    for (int k = 0; k < dp; k += 16) {
+        uint32_t q[4];
+        ldsm4(q, aq + 2 * k);
+#pragma unroll
+        for (int n = 0; n < 4; ++n) {
+            uint32_t b[4];
+            ldsm4t(b, bw + 2 * (k * kLaW + n * 16));
+            mma_bf16(acc[2 * n], q, b[0], b[1]);
+            mma_bf16(acc[2 * n + 1], q, b[2], b[3]);
+        }
+    }
+#pragma unroll
+    for (int n = 0; n < 8; ++n)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int m = m0 + rt + g + e * 8, c = c0 + ch + n * 8 + t4 * 2;
+            if (m < m_end && c < L.ld_c) *reinterpret_cast<float2*>(a.q_abs + ((size_t)m * a.heads + h) * L.ld_c + c) = make_float2(acc[n][2 * e], acc[n][2 * e + 1]);
+        }
 }
 
 // element d of a head's query against a cache row: the absorbed part, then the rotated part, times the scale
@@ -207,6 +274,7 @@ __global__ void __launch_bounds__(kLtThreads) latent_decode_kernel(const LatentL
 // elements, whose query fragments stay in its registers; softmax: a warp per head; sums: 16-column blocks over the warps.
 // The weights enter the second product as the sum of two bf16 values, so that rounding them costs nothing visible.
 constexpr int kLmThreads = 512;
+constexpr float kLog2e = 1.4426950408889634f;             // scores here are in powers of two
 
 struct LatentSmem {
     int ks;                                              // elements of a padded row
@@ -230,7 +298,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_decode_mma_kernel(const 
     cg::cluster_group cluster = cg::this_cluster();
     const int rank = (int)cluster.block_rank(), n_rank = (int)cluster.num_blocks();
     const int h0 = blockIdx.y * kLtHeads, seq = blockIdx.z, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, g = lane >> 2, t4 = lane & 3;
-    const int ks = o.ks, ldk = ks - 8, n_chunk = (L.ld_c + L.rot8) / 8, c_chunk = L.ld_c / 8, n_step = ldk / 32;
+    const int ks = o.ks, ldk = ks - 8, n_step = ldk / 32;
     const int kg = warp & 7, half = warp >> 3, p0 = half ? PH : 0, n_p = min(PH, n_step - p0);      // this warp's keys and steps
     bf16 *s_k = reinterpret_cast<bf16*>(smem + o.k), *s_q = s_k + kLtTile * ks, *s_p = reinterpret_cast<bf16*>(smem + o.p);
     float* s_s = reinterpret_cast<float*>(smem + o.s);
@@ -244,22 +312,46 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_decode_mma_kernel(const 
     const bf16* rr = static_cast<const bf16*>(a.ring_r) + (size_t)seq * a.ring_r_stride;
     const int per = (n_keys + n_rank - 1) / n_rank, j0 = min(n_keys, rank * per), j1 = min(n_keys, j0 + per);
     const int n_tiles = (j1 - j0 + kLtTile - 1) / kLtTile, slot0 = (first + j0) % a.ring;
+    const uint32_t c_bytes = 2 * L.ld_c, r_bytes = 2 * L.rot8, sk = smem_addr(s_k);
+    const char *rc8 = reinterpret_cast<const char*>(rc) + lane * 16, *rr8 = reinterpret_cast<const char*>(rr) + lane * 16;
+    auto copy = [](uint32_t dst, const char* src) { asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"(dst), "l"(src) : "memory"); };
     auto fetch = [&](int tile) {                         // a warp takes whole rows; rows past the end repeat the last one
-        bf16* dst = s_k + (tile & 1) * kLtTile * ks;
 #pragma unroll
         for (int i = 0; i < kLtTile * 32 / kLmThreads; ++i) {
-            const int r = warp + i * (kLmThreads / 32), k = slot0 + min(tile * kLtTile + r, j1 - j0 - 1);
-            const size_t slot = k >= a.ring ? k - a.ring : k;
-            for (int c = lane; c < n_chunk; c += 32)
-                cp16(dst + r * ks + c * 8, c < c_chunk ? rc + slot * L.ld_c + c * 8 : rr + slot * L.rot8 + (c - c_chunk) * 8);
+            const int r = warp + i * (kLmThreads / 32);
+            int slot = slot0 + min(tile * kLtTile + r, j1 - j0 - 1);
+            if (slot >= a.ring) slot -= a.ring;
+            const uint32_t dst = sk + 2 * ((tile & 1) * kLtTile + r) * ks + lane * 16;
+            const char* src = rc8 + (size_t)slot * c_bytes;
+            for (uint32_t c = 0; c + lane * 16 < c_bytes; c += 512) copy(dst + c, src + c);
+            if (lane * 16 < r_bytes) copy(dst + c_bytes, rr8 + (size_t)slot * r_bytes);
         }
         asm volatile("cp.async.commit_group;" ::: "memory");
     };
     if (n_tiles > 0) fetch(0);
-    for (int i = tid; i < kLtHeads * ldk; i += kLmThreads) {
-        const int h = i / ldk, d = i - h * ldk;
-        s_q[h * ks + d] = __float2bfloat16_rn(latent_query(L, seq, h0 + h, d, pos));
+    // the queries: absorbed part four elements at a time, rotated part a pair at a time, padding
+    const float scale = a.scale * kLog2e;
+    const int c4 = L.ld_c / 4, pairs = a.rot / 2, pad = ldk - L.ld_c - a.rot;
+#pragma unroll 4
+    for (int i = tid; i < kLtHeads * c4; i += kLmThreads) {
+        const int h = i / c4, d = (i - h * c4) * 4;
+        const float4 v = h0 + h < a.heads ? *reinterpret_cast<const float4*>(a.q_abs + ((size_t)seq * a.heads + h0 + h) * L.ld_c + d) : make_float4(0, 0, 0, 0);
+        const __nv_bfloat162 lo = __floats2bfloat162_rn(v.x * scale, v.y * scale), hi = __floats2bfloat162_rn(v.z * scale, v.w * scale);
+        *reinterpret_cast<uint2*>(s_q + h * ks + d) = make_uint2(reinterpret_cast<const uint32_t&>(lo), reinterpret_cast<const uint32_t&>(hi));
     }
+    for (int i = tid; i < kLtHeads * pairs; i += kLmThreads) {
+        const int h = i / pairs, f = i - h * pairs;
+        float u = 0.0f, v = 0.0f, cs, sn;
+        if (h0 + h < a.heads) {
+            const float* x = a.q + (size_t)seq * a.ld + (size_t)(h0 + h) * (a.dim + a.rot) + a.dim;
+            u = x[f];
+            v = x[pairs + f];
+        }
+        rotation(a.freq[f], pos, cs, sn);
+        s_q[h * ks + L.ld_c + f] = __float2bfloat16_rn((u * cs - v * sn) * scale);
+        s_q[h * ks + L.ld_c + pairs + f] = __float2bfloat16_rn((v * cs + u * sn) * scale);
+    }
+    for (int i = tid; i < kLtHeads * pad; i += kLmThreads) s_q[(i / pad) * ks + ldk - pad + i % pad] = __float2bfloat16_rn(0.0f);
     __syncthreads();
     uint32_t q[PH][2][4];
     const uint32_t aq = smem_addr(s_q) + 2 * ((lane & 15) * ks + (lane >> 4) * 8), ap = smem_addr(s_p) + 2 * ((lane & 15) * 72 + (lane >> 4) * 8);
@@ -297,7 +389,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_decode_mma_kernel(const 
             const int left = j1 - j0 - tile * kLtTile;   // keys of this tile
             const float *s0 = s_s + warp * 68, *s1 = s_s + (kLtHeads + warp) * 68;
             const float v0 = lane < left ? s0[lane] + s1[lane] : -INFINITY, v1 = lane + 32 < left ? s0[lane + 32] + s1[lane + 32] : -INFINITY;
-            const float mn = fmaxf(m, warp_max(fmaxf(v0, v1))), f = expf(m - mn), e0 = expf(v0 - mn), e1 = expf(v1 - mn);
+            const float mn = fmaxf(m, warp_max(fmaxf(v0, v1))), f = exp2f(m - mn), e0 = exp2f(v0 - mn), e1 = exp2f(v1 - mn);
             l = l * f + warp_sum(e0 + e1);
             m = mn;
             const bf16 b0 = __float2bfloat16_rn(e0), b1 = __float2bfloat16_rn(e1);
@@ -345,7 +437,7 @@ __global__ void __launch_bounds__(kLmThreads, 1) latent_decode_mma_kernel(const 
 #pragma unroll
             for (int e = 0; e < 4; ++e) s_acc[(g + (e >> 1) * 8) * L.ld_c + pair * 16 + x * 8 + t4 * 2 + (e & 1)] = acc[i][x][e];
     }
-    if (lane == 0) { s_ml[warp] = m; s_ml[kLtHeads + warp] = l; }
+    if (lane == 0) { s_ml[warp] = m / kLog2e; s_ml[kLtHeads + warp] = l; }
     latent_merge<bf16>(L, cluster, seq, h0, kLtHeads, s_acc, s_ml);
 }
 
@@ -405,12 +497,16 @@ __global__ void __launch_bounds__(128) latent_ring_kernel(const LatentLaunch L, 
 template <typename T>
 static int latent_decode(const LatentLaunch& L, cudaStream_t st, unsigned long long* n_kernels) {
     const LatentAttnArgs& a = L.a;
-    auto absorb = [&](auto kernel, int mr) {
-        const size_t smem = 4 * ((size_t)mr * L.dim8 + 16 * mr * 128);
+    auto absorb = [&](auto kernel, int rows, size_t smem, int append) {
         if (int rc = allow_smem(kernel, smem)) return rc;
-        return launch_kernel(kernel, dim3((L.ld_c + 127) / 128, a.heads + (a.dkv ? 1 : 0), (a.M + mr - 1) / mr), dim3(kLtThreads), smem, st, a.use_pdl, 1, L);
+        return launch_kernel(kernel, dim3((L.ld_c + 127) / 128, a.heads + (a.dkv ? append : 0), (a.M + rows - 1) / rows), dim3(kLtThreads), smem, st, a.use_pdl, 1, L);
     };
-    if (int rc = a.M == 1 ? absorb(latent_absorb_kernel<T, 1>, 1) : absorb(latent_absorb_kernel<T, kLtAbsorbRows>, kLtAbsorbRows)) return rc;
+    auto fma_smem = [&](int rows) { return 4 * ((size_t)rows * L.dim8 + 8 * rows * 128); };
+    const int dp = round_up(a.dim, 16);
+    const int rc0 = a.M == 1                           ? absorb(latent_absorb_kernel<T, 1>, 1, fma_smem(1), 1)
+                    : sizeof(T) == 4 || a.M < kLaMinRows ? absorb(latent_absorb_kernel<T, kLtAbsorbRows>, kLtAbsorbRows, fma_smem(kLtAbsorbRows), 1)
+                                                         : absorb(latent_absorb_mma_kernel, kLaM, 2 * ((size_t)dp * kLaW + kLaM * (dp + 8)), 4);
+    if (rc0) return rc0;
     const LatentSmem o(L.ld_c, L.rot8);
     const bool mma = sizeof(T) == 2 && L.ld_c <= 512 && o.bytes <= 220 * 1024;
     const int per_cta = mma ? kLtHeads : kLtFmaHeads, tiles = (a.heads + per_cta - 1) / per_cta;

@@ -7,32 +7,29 @@ namespace tz {
 
 constexpr int kRouteThreads = 1024, kRouteSmallPairs = 1024;
 
-// A warp chooses for row m; s: [E] scratch of the warp.
-__device__ __forceinline__ void choose(const RouteArgs& a, int m, float* s) {
+// A warp chooses for row m; s: [E] scratch of the warp. Choice scores are kept as integers in the order of the floats, 0 for
+// an expert that is taken (what a score that is not a number becomes may be any other value).
+__device__ __forceinline__ unsigned ordered(float v) {
+    const unsigned b = __float_as_uint(v);
+    return max(b ^ ((b >> 31) ? 0xffffffffu : 0x80000000u), 1u);
+}
+
+__device__ __forceinline__ void choose(const RouteArgs& a, int m, unsigned* s) {
     const int lane = threadIdx.x & 31;
     const float* z = a.logits + (size_t)m * a.ld;
-    for (int e = lane; e < a.experts; e += 32) s[e] = sigmoid_f(z[e]) + (a.correction ? a.correction[e] : 0.0f);
+    for (int e = lane; e < a.experts; e += 32) s[e] = ordered(sigmoid_f(z[e]) + (a.correction ? a.correction[e] : 0.0f));
     __syncwarp();
     for (int j = 0; j < a.top; ++j) {
-        float best = -INFINITY;
+        unsigned best = 0;
         int at = 0x7fffffff;
         for (int e = lane; e < a.experts; e += 32)
-            if (s[e] > best || (s[e] == best && e < at)) { best = s[e]; at = e; }
-#pragma unroll
-        for (int x = 16; x > 0; x >>= 1) {
-            const float v = __shfl_xor_sync(0xffffffffu, best, x);
-            const int i = __shfl_xor_sync(0xffffffffu, at, x);
-            if (v > best || (v == best && i < at)) { best = v; at = i; }
-        }
-        if (at >= a.experts) {                            // not-a-number scores: any expert not taken yet
-            at = 0;
-            for (int e = a.experts - 1; e >= 0; --e)
-                if (s[e] != -INFINITY) at = e;
-        }
+            if (s[e] > best) { best = s[e]; at = e; }
+        const unsigned top = __reduce_max_sync(0xffffffffu, best);
+        at = (int)__reduce_min_sync(0xffffffffu, best == top ? (unsigned)at : 0x7fffffffu);      // equal scores: the lower index
         if (lane == 0) {
             a.chosen[(size_t)m * a.top + j] = at;
             a.weight[(size_t)m * a.top + j] = sigmoid_f(z[at]);
-            s[at] = -INFINITY;
+            s[at] = 0;
         }
         __syncwarp();
     }
@@ -66,7 +63,7 @@ __device__ __forceinline__ void place_pairs(const RouteArgs& a, int e, const int
 }
 
 __global__ void __launch_bounds__(kRouteThreads) route_small_kernel(const RouteArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ unsigned sm[];
     __shared__ int s_chosen[kRouteSmallPairs];
     const int warp = threadIdx.x >> 5, nw = blockDim.x >> 5, n = a.M * a.top;
     pdl_wait();
@@ -79,7 +76,7 @@ __global__ void __launch_bounds__(kRouteThreads) route_small_kernel(const RouteA
 }
 
 __global__ void __launch_bounds__(256) route_choose_kernel(const RouteArgs a) {
-    extern __shared__ float sm[];
+    extern __shared__ unsigned sm[];
     const int m = blockIdx.x * 8 + (threadIdx.x >> 5);
     if (m < a.M) choose(a, m, sm + (size_t)(threadIdx.x >> 5) * a.experts);
 }

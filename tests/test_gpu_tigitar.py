@@ -340,6 +340,34 @@ def test_latent_attention(f32, heads, dim, rot, vdim, rank, window):
 
 
 @pytest.mark.parametrize("f32", [0, 1])
+@pytest.mark.parametrize("B,heads,dim,rot,vdim,rank,window", [(2, 3, 20, 4, 16, 72, 5), (15, 4, 100, 10, 24, 130, 40), (70, 2, 128, 64, 128, 512, 33)])
+def test_latent_attention_of_sequences_side_by_side(f32, B, heads, dim, rot, vdim, rank, window):
+    """Decode rows of several sequences at different positions, each against its own history."""
+    rng = np.random.default_rng(B)
+    one = Latent(f32, heads, dim, rot, vdim, rank, window, rng)
+    xs = [(as_f32(rng.standard_normal((n + 2, heads * (dim + rot)))), as_f32(rng.standard_normal((n + 2, rank + rot)))) for n in rng.integers(0, 3 * window, B)]
+    rc, rr = (torch.zeros((B,) + tuple(t.shape), dtype=DT[f32], device="cuda") for t in (one.rc, one.rr))
+    for s, (q, dkv) in enumerate(xs):
+        one.pos = 0
+        one.rc.zero_(), one.rr.zero_()
+        if len(q) > 2:
+            one.run(q[:-2], dkv[:-2], decode=0)
+        rc[s], rr[s] = one.rc, one.rr
+    want = np.stack([one.want(q, dkv)[-2:] for q, dkv in xs])
+    got = []
+    for i in range(2):
+        x = dev(np.stack([np.concatenate([q[len(q) - 2 + i], dkv[len(q) - 2 + i]]) for q, dkv in xs]))
+        out = torch.zeros((B, heads * one.v8), dtype=DT[f32], device="cuda")
+        kernels.latent_attention(q=x, dkv=x[:, heads * (dim + rot):], ld=x.shape[1], norm=dev(one.norm), eps=1e-5, freq=one.freq, heads=heads, dim=dim, rot=rot, vdim=vdim, rank=rank,
+                                 scale=one.scale, window=window, w_kv=one.w, ring_c=rc, ring_r=rr, ring=window, ring_c_stride=rc[0].numel(), ring_r_stride=rr[0].numel(),
+                                 pos=torch.tensor([len(q) - 2 + i for q, _ in xs], dtype=torch.int32, device="cuda"), M=B, decode=1, out=out, ld_out=heads * one.v8,
+                                 q_abs=torch.zeros((B, heads, one.ld), device="cuda"), lat=torch.zeros((heads, B, one.ld), dtype=DT[f32], device="cuda"), workspace=one.ws,
+                                 workspace_bytes=one.ws.numel(), f32=f32)
+        got.append(host(out).reshape(B, heads, one.v8)[:, :, :vdim].reshape(B, -1))
+    assert rel(np.stack(got, axis=1), want) < (3e-6 if f32 else 8e-3)
+
+
+@pytest.mark.parametrize("f32", [0, 1])
 @pytest.mark.parametrize("windows", [(9, 40), (40, 9), (70, 70), (1, 130)])
 def test_a_borrowed_latent_cache(f32, windows):
     """A second set of heads with a window of its own reads the rows that the first one left; the ring serves the wider window."""

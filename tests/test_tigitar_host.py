@@ -54,7 +54,7 @@ def test_kernel_calls_reject_bad_arguments_without_a_device():
     assert lib.tenzo_cuda_latent_attention(C.byref(b), None) == -1
     r = abi.RouteArgs(M=1, experts=2, top=3)
     assert lib.tenzo_cuda_route(C.byref(r), None) == -1
-    assert lib.tenzo_cuda_delta_rule_work_floats(9, 4, 2, 33, 17) == 2 * 2 * 16 * 64 + 2 * 4 * 8 * 32 + 2 * 4 * 144 + 9 * 4 * 17
+    assert lib.tenzo_cuda_delta_rule_work_floats(9, 4, 2, 33, 17) == 2 * 2 * 16 * 64 + 2 * 4 * 8 * 24 + 2 * 4 * 144 + 9 * 4 * 17
 
 
 def test_oracle_is_causal(tmp_path):
