@@ -36,7 +36,7 @@ TENZO_API tenzo_engine_t tenzo_ext_create_engine(const tenzo_config_t* config, c
 TENZO_API int tenzo_ext_batch(tenzo_engine_t engine);
 
 /* Models by folder: config.json names the architecture, the rest of the folder is what that family loads - "Sozopel"
- * (hybrid decoder): model.safetensors; "BitNet": weights.bin + model.mlir, with the fields of tenzo_config_t in
+ * and "Tigitar" (hybrid decoders): model.safetensors; "BitNet": weights.bin + model.mlir, with the fields of tenzo_config_t in
  * config.json. `compute` is the arithmetic of activations and matrix products: TENZO_COMPUTE_BF16 (bf16 operands, 32-bit
  * accumulation) or TENZO_COMPUTE_F32 (32-bit throughout); BitNet has its own integer arithmetic and takes only the
  * default. opt->batch, use_graph and use_pdl apply to every family. NULL on failure, see tenzo_ext_last_error(). */
